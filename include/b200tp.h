@@ -32,6 +32,9 @@ enum {
   B2_ERR_UNSUPPORTED = 6
 };
 
+enum { B2_DT_BF16 = 0, B2_DT_F32 = 1 };               /* element type of activations, weights and KV cache where a call takes one */
+enum { B2_ACT_NONE = 0, B2_ACT_SILU = 1, B2_ACT_RELU = 2 };
+
 #define B2_HANDLE_BYTES 64 /* one exported symmetric-memory handle */
 
 typedef struct b2_ctx b2_ctx;
@@ -133,7 +136,9 @@ int b2_gemm(b2_ctx* ctx, const void* A, int64_t lda, const void* W, int64_t ldw,
  * qkv[M, (nq + 2 nkv) head_dim] = A W^T (+ bias); then, per token and head:
  * q and k heads are RMS-normalised (weights may both be NULL) and rotated,
  * k and v heads are also written to the paged cache (k_cache may be NULL).
- * Arguments as b2_gemm and b2_qk_norm_rope_store.  For up to 64 tokens and
+ * Arguments as b2_gemm and b2_qk_norm_rope_store; cos_sin = NULL leaves the
+ * heads unrotated (positions may then be NULL, and a normalised head is rounded
+ * once instead of after each factor).  For up to 64 tokens and
  * head_dim 128 everything happens in the GEMM's epilogue (one launch);
  * otherwise the projection and the head kernel run as two launches. */
 int b2_qkv_fused(b2_ctx* ctx, const void* A, int64_t lda, const void* W, int64_t ldw, const void* bias, void* qkv,
@@ -150,6 +155,23 @@ int b2_qkv_fused(b2_ctx* ctx, const void* A, int64_t lda, const void* W, int64_t
  * bf16, then the product).  The [M, 2 I] intermediate never reaches HBM. */
 int b2_gemm_silu_mul(b2_ctx* ctx, const void* A, int64_t lda, const void* W_pairs, int64_t ldw, void* out, int64_t ldo,
                      int M, int I, int K, void* stream);
+
+/* The same with the activation named: out = act(A gate_j^T) * (A up_j^T), act = B2_ACT_SILU or B2_ACT_RELU. */
+int b2_gemm_act_mul(b2_ctx* ctx, const void* A, int64_t lda, const void* W_pairs, int64_t ldw, void* out, int64_t ldo,
+                    int M, int I, int K, int act, void* stream);
+
+/* b2_gemm whose first silu_cols output features (a multiple of 8) leave the
+ * kernel as silu(x); the activation is applied to the fp32 accumulator.  Merged
+ * projections of which only some sections are activated. */
+int b2_gemm_silu_cols(b2_ctx* ctx, const void* A, int64_t lda, const void* W, int64_t ldw, void* C, int64_t ldc, int M,
+                      int N, int K, int silu_cols, void* stream);
+
+/* The matrix product in true 32-bit (fp32 operands, CUDA cores), for models run
+ * in fp32: C[M, N] = A[M, K] W[N, K]^T; pair_act != B2_ACT_NONE stores
+ * act(even row) * odd row per row pair of W into C[M, N / 2]; otherwise the
+ * first silu_cols features are activated.  K a multiple of 8, N even. */
+int b2_gemm_f32(const float* A, int64_t lda, const float* W, int64_t ldw, float* C, int64_t ldc, int M, int N, int K,
+                int pair_act, int silu_cols, void* stream);
 
 /* ---- the same GEMM for callers that cannot allocate device memory.  It has
  *      no counterpart in the reference. ----------------------------------------
@@ -379,6 +401,77 @@ int b2_qk_norm_rope_store(void* qkv, int64_t ld_qkv, int M, int nq, int nkv, int
                           const void* q_norm_w, const void* k_norm_w, float eps,
                           const int64_t* positions, const float* cos_sin,
                           void* k_cache, void* v_cache, const int32_t* slot_mapping, void* stream);
+
+/* ---- mechanisms of designs the reference does not have ----------------------
+ * dtype (B2_DT_*) is the element type of activations and caches.  "_pad" sizes
+ * are multiples of 8: a head of qk_dim elements occupies qk_pad, of which the
+ * rest is zero (zero rows of the projection's weight), so that every head starts
+ * on a vector boundary for any size. */
+
+/* Residual streams in fp32, everything between two sublayers in one launch.
+ * x [M, streams, dim_pad] fp32 holds S copies of the residual.
+ *   ids != NULL:  every copy = table[ids] * embed_scale        (start of the model)
+ *   y != NULL:    x_t <- sum_s mix[s, t] x_s + mult w_out[t] y  (mix row-major [from][to])
+ *   u = sum_s w_in[s] x_s                                      (w_in NULL = all ones)
+ *   normed = u / sqrt(mean(u^2) + eps) * norm_w, the mean over `dim` elements
+ * x_out (may be x_in, NULL = not stored) receives the copies; normed may be
+ * NULL.  Coefficients and norm weight are fp32; rows of y / normed have strides
+ * ldy / ldn. */
+int b2_stream_step(int dtype, float* x_out, const float* x_in, const int64_t* ids, const void* table, int64_t ld_table,
+                   int64_t vocab, float embed_scale, const void* y, int64_t ldy, const float* mix, const float* w_out,
+                   float mult, const float* w_in, const float* norm_w, float eps, void* normed, int64_t ldn, int M,
+                   int streams, int dim, int dim_pad, void* stream);
+
+/* q/k head RMSNorm without rotation (weights may both be NULL) in place on rows
+ * [nq q heads | nkv k heads | nkv v heads], and the scatter of K and V into the
+ * paged cache (k_cache may be NULL; slot -1 stores nothing).  q/k heads have
+ * qk_dim, v heads v_dim elements. */
+int b2_qk_norm_store(int dtype, void* qkv, int64_t ld_qkv, int M, int nq, int nkv, int qk_dim, int qk_pad, int v_dim,
+                     int v_pad, const void* q_norm_w, const void* k_norm_w, float eps, void* k_cache, void* v_cache,
+                     const int32_t* slot_mapping, void* stream);
+
+/* Attention over the paged cache (k_cache [slots, nkv, qk_pad], v_cache
+ * [slots, nkv, v_pad]; block_tables int32 [B, bt_stride], block_size slots per
+ * block), this step's keys included.  Sequence b has kv_len[b] keys; its query
+ * rows are cu_q[b] .. cu_q[b+1] (its last positions), or the single row b when
+ * cu_q is NULL (decode).  Position i sees j when j <= i and (i - j < window or
+ * j < keep_first).  score = (q . k) scale, then softcap tanh(score / softcap)
+ * when softcap > 0; the softmax's denominator also contains exp(sink[head])
+ * when sink (fp32) is given.  q heads start every qk_pad elements of a row of q,
+ * outputs every v_pad of a row of out.  max_q / max_kv bound the step (host
+ * values; max_kv sizes the split of a decode step).  kv_len 0 marks a padded
+ * row of a decode graph (its output is zero).
+ * workspace: fp32 scratch of b2_attention_workspace bytes, zero before the
+ * first call and left zero where it has to be; one call at a time.
+ * form: 0 = the library chooses, 1 = the kernel for any size. */
+int64_t b2_attention_workspace(int dtype, int B, int max_q, int max_kv, int nq, int nkv, int qk_pad, int v_pad, int window,
+                               int keep_first);
+int b2_attention(int dtype, const void* q, int64_t ldq, void* out, int64_t ldo, const void* k_cache, const void* v_cache,
+                 const int32_t* block_tables, int64_t bt_stride, int block_size, const int32_t* cu_q,
+                 const int32_t* kv_len, int B, int max_q, int max_kv, int nq, int nkv, int qk_pad, int v_pad,
+                 float scale, float softcap, int window, int keep_first, const float* sink, void* workspace,
+                 int64_t workspace_bytes, int form, void* stream);
+
+/* Linear attention with a constant decay per head:
+ *   S_t = decay[h] S_(t-1) + k_t v_t^T,  o_t = S_t^T q_t
+ * qkv rows are [heads q | heads k | heads v | ...], activations applied; o
+ * [M, heads v_pad] fp32; state fp32 [slots, heads, qk_pad, v_pad], slots[b] the
+ * sequence's slot (-1 = padded row).  A sequence whose step starts at position 0
+ * (kv_len[b] equals its rows) starts from a zero state whatever its slot holds.
+ * decay_powers: fp32 [heads, 65], decay^0 .. decay^64.
+ * workspace: scratch of b2_linear_attn_workspace bytes (prefill; no contents
+ * are kept between calls).
+ * form: 0 = the library chooses, 1 = the kernel for any size. */
+int64_t b2_linear_attn_workspace(int dtype, int B, int max_q, int total_q, int heads, int qk_pad, int v_pad);
+int b2_linear_attn(int dtype, const void* qkv, int64_t ld_qkv, float* o, int64_t ldo, float* state, const int32_t* slots,
+                   const int32_t* cu_q, const int32_t* kv_len, const float* decay, const float* decay_powers, int B,
+                   int max_q, int total_q, int heads, int qk_pad, int v_pad, void* workspace, int64_t workspace_bytes,
+                   int form, void* stream);
+
+/* out = o / sqrt(mean(o^2) + eps) * w * sigmoid(gate) per row: o fp32, w fp32,
+ * the mean over `dim` of dim_pad elements (the rest of o is zero). */
+int b2_gated_norm(int dtype, const float* o, int64_t ldo, const void* gate, int64_t ldg, const float* w, float eps, int M,
+                  int dim, int dim_pad, void* out, int64_t ld_out, void* stream);
 
 /* Greedy pick: out[i] = argmax_j logits[i, j] (first index on ties), int64.
  * The reference's Sampler (nanovllm/layers/sampler.py:7-12) at temperature -> 0. */

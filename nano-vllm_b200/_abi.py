@@ -21,6 +21,8 @@ lib = C.CDLL(LIB_PATH)
 
 OK, ERR_ARG, ERR_SHAPE, ERR_CUDA, ERR_STATE, ERR_TIMEOUT, ERR_UNSUPPORTED = range(7)
 HANDLE_BYTES = 64
+DT_BF16, DT_F32 = 0, 1
+ACT_NONE, ACT_SILU, ACT_RELU = range(3)
 FORM_AUTO, FORM_ONESHOT, FORM_OWNER, FORM_TWOSHOT = range(4)
 OPT_ROWPAR_FORM, OPT_OWNER_MAX_TOKENS, OPT_TWOSHOT_MIN_TOKENS, OPT_WHOLE_TILES, OPT_OWNER_MIN_TOKENS = 1, 2, 3, 4, 5
 _ERR_NAMES = {1: "bad argument", 2: "shape outside what the context was created for", 3: "CUDA error",
@@ -58,6 +60,14 @@ SIGNATURES = {
     "b2_gemm": [_p, _p, _i64, _p, _i64, _p, _p, _i64, _i, _i, _i, _p],
     "b2_qkv_fused": [_p, _p, _i64, _p, _i64, _p, _p, _i64, _i, _i, _i, _i, _i, _p, _p, _f, _p, _p, _p, _p, _p, _p],
     "b2_gemm_silu_mul": [_p, _p, _i64, _p, _i64, _p, _i64, _i, _i, _i, _p],
+    "b2_gemm_act_mul": [_p, _p, _i64, _p, _i64, _p, _i64, _i, _i, _i, _i, _p],
+    "b2_gemm_silu_cols": [_p, _p, _i64, _p, _i64, _p, _i64, _i, _i, _i, _i, _p],
+    "b2_gemm_f32": [_p, _i64, _p, _i64, _p, _i64, _i, _i, _i, _i, _i, _p],
+    "b2_stream_step": [_i, _p, _p, _p, _p, _i64, _i64, _f, _p, _i64, _p, _p, _f, _p, _p, _f, _p, _i64, _i, _i, _i, _i, _p],
+    "b2_qk_norm_store": [_i, _p, _i64, _i, _i, _i, _i, _i, _i, _i, _p, _p, _f, _p, _p, _p, _p],
+    "b2_attention": [_i, _p, _i64, _p, _i64, _p, _p, _p, _i64, _i, _p, _p, _i, _i, _i, _i, _i, _i, _i, _f, _f, _i, _i, _p, _p, _i64, _i, _p],
+    "b2_linear_attn": [_i, _p, _i64, _p, _i64, _p, _p, _p, _p, _p, _p, _i, _i, _i, _i, _i, _i, _p, _i64, _i, _p],
+    "b2_gated_norm": [_i, _p, _i64, _p, _i64, _p, _f, _i, _i, _i, _p, _i64, _p],
     "b2_gemm_static_scratch": [_p, _i64, _p, _i64, _p, _p, _i64, _i, _i, _i, _p],
     "b2_rowpar_fused": [_p, _p, _i64, _p, _i64, _p, _i, _i, _i, _p, _p, _f, _p, _p, _p],
     "b2_ctx_set_option": [_p, _i, _i64],
@@ -91,12 +101,16 @@ for _name, _args in SIGNATURES.items():
     _fn = getattr(lib, _name)
     _fn.argtypes = _args
     _fn.restype = _i
+for _name, _args in {"b2_attention_workspace": [_i] * 10, "b2_linear_attn_workspace": [_i] * 7}.items():
+    _fn = getattr(lib, _name)
+    _fn.argtypes = _args
+    _fn.restype = _i64
 lib.b2_last_error.restype = C.c_char_p
 lib.b2_last_error.argtypes = []
 lib.b2_launch_count.restype = _i64
 lib.b2_launch_count.argtypes = []
 
-EXPORTED = list(SIGNATURES) + ["b2_last_error", "b2_launch_count"]
+EXPORTED = list(SIGNATURES) + ["b2_attention_workspace", "b2_linear_attn_workspace", "b2_last_error", "b2_launch_count"]
 
 
 def check(rc: int, what: str) -> None:

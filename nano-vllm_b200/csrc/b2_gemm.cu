@@ -97,7 +97,8 @@ struct GemmArgs {
   uint16_t* k_cache;
   uint16_t* v_cache;
   const int32_t* slots;
-  int silu_pairs;  // 1: features come in (gate, up) pairs; store silu(gate) * up, one value per pair, at column feature / 2
+  int pair_act;   // B2_ACT_*: features come in (gate, up) pairs; store act(gate) * up, one value per pair, at column feature / 2
+  int silu_cols;  // features below this one leave the kernel as silu(x), the others as they are
   // stream-K combine
   float* ws;
   int* counters;
@@ -284,11 +285,15 @@ __host__ __device__ __forceinline__ int owned_rows3(int M, int world, int rank) 
 __device__ __forceinline__ float silu_mul(float gate, float up) {
   return b2::bf16_round(gate / (1.0f + expf(-gate))) * up;
 }
-// 8 bf16 = 4 (gate, up) pairs -> 4 bf16
-__device__ __forceinline__ uint2 silu_mul_pairs(const uint4& w) {
-  return make_uint2(b2::pack_bf16(silu_mul(b2::bf16_lo(w.x), b2::bf16_hi(w.x)), silu_mul(b2::bf16_lo(w.y), b2::bf16_hi(w.y))),
-                    b2::pack_bf16(silu_mul(b2::bf16_lo(w.z), b2::bf16_hi(w.z)), silu_mul(b2::bf16_lo(w.w), b2::bf16_hi(w.w))));
+__device__ __forceinline__ float act_mul(int act, float gate, float up) {
+  return act == B2_ACT_RELU ? fmaxf(gate, 0.f) * up : silu_mul(gate, up);
 }
+// 8 bf16 = 4 (gate, up) pairs -> 4 bf16
+__device__ __forceinline__ uint2 act_mul_pairs(int act, const uint4& w) {
+  return make_uint2(b2::pack_bf16(act_mul(act, b2::bf16_lo(w.x), b2::bf16_hi(w.x)), act_mul(act, b2::bf16_lo(w.y), b2::bf16_hi(w.y))),
+                    b2::pack_bf16(act_mul(act, b2::bf16_lo(w.z), b2::bf16_hi(w.z)), act_mul(act, b2::bf16_lo(w.w), b2::bf16_hi(w.w))));
+}
+__device__ __forceinline__ float silu_f32(float x) { return x / (1.0f + expf(-x)); }
 
 // NC columns (tokens token0 ..) of one feature per lane, features = consecutive lanes.
 // Lanes 2i and 2i+1 hold features f and f+1 of the same tokens.  They swap
@@ -302,6 +307,10 @@ __device__ __forceinline__ void emit_feature_lanes(const GemmArgs& a, float (&v)
 #pragma unroll
     for (int j = 0; j < NC; ++j) v[j] += b;
   }
+  if (EPI == EPI_STORE && feature < a.silu_cols) {
+#pragma unroll
+    for (int j = 0; j < NC; ++j) v[j] = silu_f32(v[j]);
+  }
   const int fbase = feature & ~1;
   const bool odd = lane & 1;
 #pragma unroll
@@ -312,8 +321,8 @@ __device__ __forceinline__ void emit_feature_lanes(const GemmArgs& a, float (&v)
     uint32_t w = odd ? b2::pack_bf16(recv, v[j + 1]) : b2::pack_bf16(v[j], recv);
     if (token < a.M && fbase < a.N) {
       if (EPI == EPI_STORE) {
-        if (a.silu_pairs) {  // w = (gate, up) of feature pair fbase / 2
-          const float act = silu_mul(b2::bf16_lo(w), b2::bf16_hi(w));
+        if (a.pair_act) {  // w = (gate, up) of feature pair fbase / 2
+          const float act = act_mul(a.pair_act, b2::bf16_lo(w), b2::bf16_hi(w));
           a.C[token * a.ldc + (fbase >> 1)] = static_cast<uint16_t>(b2::pack_bf16(act, 0.f) & 0xFFFF);
         } else {
           *reinterpret_cast<uint32_t*>(a.C + token * a.ldc + fbase) = w;
@@ -357,6 +366,10 @@ __device__ __forceinline__ void stage_row_chunk(const GemmArgs& a, unsigned char
       f[0] += b2::bf16_lo(bv.x); f[1] += b2::bf16_hi(bv.x); f[2] += b2::bf16_lo(bv.y); f[3] += b2::bf16_hi(bv.y);
       f[4] += b2::bf16_lo(bv.z); f[5] += b2::bf16_hi(bv.z); f[6] += b2::bf16_lo(bv.w); f[7] += b2::bf16_hi(bv.w);
     }
+    if (feature < a.silu_cols) {  // silu_cols is a multiple of 8
+#pragma unroll
+      for (int e = 0; e < 8; ++e) f[e] = silu_f32(f[e]);
+    }
     uint4 w = make_uint4(b2::pack_bf16(f[0], f[1]), b2::pack_bf16(f[2], f[3]), b2::pack_bf16(f[4], f[5]), b2::pack_bf16(f[6], f[7]));
     if (scrub) {
       w.x = b2::scrub_sentinel(w.x); w.y = b2::scrub_sentinel(w.y);
@@ -380,7 +393,7 @@ __device__ __forceinline__ void flush_rows(const GemmArgs& a, unsigned char* wbu
     if (piece < npieces && token < a.M && feature < a.N) {
       const uint4 w = *reinterpret_cast<const uint4*>(wbuf + row * STAGE_ROW_BYTES + ((piece ^ (row & 15)) << 4));
       if (EPI == EPI_STORE) {
-        if (a.silu_pairs) *reinterpret_cast<uint2*>(a.C + token * a.ldc + (feature >> 1)) = silu_mul_pairs(w);
+        if (a.pair_act) *reinterpret_cast<uint2*>(a.C + token * a.ldc + (feature >> 1)) = act_mul_pairs(a.pair_act, w);
         else *reinterpret_cast<uint4*>(a.C + token * a.ldc + feature) = w;
       } else if (EPI == EPI_PUSH2) {
         int lrow;
@@ -1207,7 +1220,7 @@ gemm_cluster_kernel(const __grid_constant__ CUtensorMap tmP, const __grid_consta
     b2::pdl_wait();
     if (is_push(EPI)) parity = *reinterpret_cast<volatile unsigned int*>(&a.dstate->rowpar_seq) & 1u;
     if (EPI == EPI_STORE && a.qkv_fused) {
-      const bool rotated = tile < a.nq + a.nkv;
+      const bool rotated = a.cos_sin != nullptr && tile < a.nq + a.nkv;
 #pragma unroll
       for (int i = 0; i < PRE_ROWS; ++i) {
         const int lt = (warp - 2) + 4 * i;
@@ -1266,6 +1279,9 @@ gemm_cluster_kernel(const __grid_constant__ CUtensorMap tmP, const __grid_consta
         const float4 t = *reinterpret_cast<const float4*>(red_buf + ((src * GL + gl) * BM + f) * 16);
         sum.x += t.x; sum.y += t.y; sum.z += t.z; sum.w += t.w;
       }
+      if (EPI == EPI_STORE && feature < a.silu_cols) {
+        sum.x = silu_f32(sum.x); sum.y = silu_f32(sum.y); sum.z = silu_f32(sum.z); sum.w = silu_f32(sum.w);
+      }
       const uint32_t lo = b2::pack_bf16(sum.x, sum.y), hi = b2::pack_bf16(sum.z, sum.w);
       out16[(gl * 4 + 0) * BM + f] = static_cast<uint16_t>(lo & 0xFFFF);
       out16[(gl * 4 + 1) * BM + f] = static_cast<uint16_t>(lo >> 16);
@@ -1304,9 +1320,12 @@ gemm_cluster_kernel(const __grid_constant__ CUtensorMap tmP, const __grid_consta
           cs4[0] = pre_cs[i][0]; cs4[1] = pre_cs[i][1]; cs4[2] = pre_cs[i][2]; cs4[3] = pre_cs[i][3];
         } else {  // more rows than were prefetched (no K split: the CTA owns all 64 tokens)
           slot = (a.k_cache != nullptr && !is_q) ? __ldg(a.slots + token) : -1;
-          const float* cs = a.cos_sin + __ldg(a.positions + token) * 128;
-          cs4[0] = __ldg(cs + lane * 2); cs4[1] = __ldg(cs + lane * 2 + 1);
-          cs4[2] = __ldg(cs + 64 + lane * 2); cs4[3] = __ldg(cs + 64 + lane * 2 + 1);
+          cs4[0] = cs4[1] = cs4[2] = cs4[3] = 0.f;
+          if (a.cos_sin != nullptr) {
+            const float* cs = a.cos_sin + __ldg(a.positions + token) * 128;
+            cs4[0] = __ldg(cs + lane * 2); cs4[1] = __ldg(cs + lane * 2 + 1);
+            cs4[2] = __ldg(cs + 64 + lane * 2); cs4[3] = __ldg(cs + 64 + lane * 2 + 1);
+          }
         }
         if (is_q || is_k) {
           float x1[2] = {b2::bf16_lo(lo), b2::bf16_hi(lo)}, x2[2] = {b2::bf16_lo(hi), b2::bf16_hi(hi)};
@@ -1317,11 +1336,17 @@ gemm_cluster_kernel(const __grid_constant__ CUtensorMap tmP, const __grid_consta
             const float rstd = rsqrtf(ss / 128.0f + a.qk_eps);
 #pragma unroll
             for (int e = 0; e < 2; ++e) {
-              x1[e] = b2::bf16_round(b2::bf16_round(x1[e] * rstd) * nw1[e]);
-              x2[e] = b2::bf16_round(b2::bf16_round(x2[e] * rstd) * nw2[e]);
+              if (a.cos_sin != nullptr) {
+                x1[e] = b2::bf16_round(b2::bf16_round(x1[e] * rstd) * nw1[e]);
+                x2[e] = b2::bf16_round(b2::bf16_round(x2[e] * rstd) * nw2[e]);
+              } else {  // heads without rotation: the normalised value is rounded once, at the store
+                x1[e] = x1[e] * rstd * nw1[e];
+                x2[e] = x2[e] * rstd * nw2[e];
+              }
             }
           }
-          float y1[2], y2[2];
+          float y1[2] = {x1[0], x1[1]}, y2[2] = {x2[0], x2[1]};
+          if (a.cos_sin != nullptr)
 #pragma unroll
           for (int e = 0; e < 2; ++e) {
             y1[e] = __fsub_rn(__fmul_rn(x1[e], cs4[e]), __fmul_rn(x2[e], cs4[2 + e]));
@@ -1349,7 +1374,7 @@ gemm_cluster_kernel(const __grid_constant__ CUtensorMap tmP, const __grid_consta
       if (token < a.M && feat < a.N) {
         uint4 w = *reinterpret_cast<const uint4*>(out_buf + lt * (BM * 2) + piece * 16);
         if (EPI == EPI_STORE) {
-          if (a.silu_pairs) *reinterpret_cast<uint2*>(a.C + token * a.ldc + (feat >> 1)) = silu_mul_pairs(w);
+          if (a.pair_act) *reinterpret_cast<uint2*>(a.C + token * a.ldc + (feat >> 1)) = act_mul_pairs(a.pair_act, w);
           else *reinterpret_cast<uint4*>(a.C + token * a.ldc + feat) = w;
         } else if (EPI == EPI_PUSH3) {
           w.x = b2::scrub_sentinel(w.x); w.y = b2::scrub_sentinel(w.y);
@@ -2121,6 +2146,21 @@ int b2_gemm(b2_ctx* ctx, const void* A, int64_t lda, const void* W, int64_t ldw,
   return launch_gemm<EPI_STORE>(ctx, A, lda, W, ldw, M, N, K, args, 0, static_cast<cudaStream_t>(stream));
 }
 
+int b2_gemm_silu_cols(b2_ctx* ctx, const void* A, int64_t lda, const void* W, int64_t ldw, void* C, int64_t ldc, int M, int N, int K,
+                      int silu_cols, void* stream) {
+  if (ctx == nullptr) return B2_ERR_ARG;
+  int rc = check_operands(A, lda, W, ldw, M, N, K);
+  if (rc != B2_OK) return rc;
+  if (silu_cols < 0 || silu_cols > N || silu_cols % 8 != 0) return B2_ERR_ARG;
+  if (M == 0) return B2_OK;
+  if (!C || !aligned16(C) || ldc % 8 != 0 || ldc < N) return B2_ERR_ARG;
+  GemmArgs args{};
+  args.C = static_cast<uint16_t*>(C);
+  args.ldc = ldc;
+  args.silu_cols = silu_cols;
+  return launch_gemm<EPI_STORE>(ctx, A, lda, W, ldw, M, N, K, args, 0, static_cast<cudaStream_t>(stream));
+}
+
 int b2_qkv_fused(b2_ctx* ctx, const void* A, int64_t lda, const void* W, int64_t ldw, const void* bias, void* qkv, int64_t ld_qkv, int M,
                  int nq, int nkv, int head_dim, int K, const void* q_norm_w, const void* k_norm_w, float eps, const int64_t* positions,
                  const float* cos_sin, void* k_cache, void* v_cache, const int32_t* slot_mapping, void* stream) {
@@ -2129,7 +2169,7 @@ int b2_qkv_fused(b2_ctx* ctx, const void* A, int64_t lda, const void* W, int64_t
   int rc = check_operands(A, lda, W, ldw, M, N, K);
   if (rc != B2_OK) return rc;
   if (M == 0) return B2_OK;
-  if (!qkv || !aligned16(qkv) || ld_qkv % 8 != 0 || ld_qkv < N || !positions || !cos_sin) return B2_ERR_ARG;
+  if (!qkv || !aligned16(qkv) || ld_qkv % 8 != 0 || ld_qkv < N || (cos_sin != nullptr && !positions)) return B2_ERR_ARG;
   if ((q_norm_w == nullptr) != (k_norm_w == nullptr)) return B2_ERR_ARG;
   if (k_cache != nullptr && (!v_cache || !slot_mapping)) return B2_ERR_ARG;
   if (bias != nullptr && !aligned16(bias)) return B2_ERR_ARG;
@@ -2154,13 +2194,23 @@ int b2_qkv_fused(b2_ctx* ctx, const void* A, int64_t lda, const void* W, int64_t
   if (rc != B2_OK) return rc;
   if (args.qkv_fused && g_last_gemm_path == 1) return B2_OK;
   // many tokens (or 64-wide heads): the projection ran on the stream-K kernel; finish the heads in a second launch
+  if (cos_sin == nullptr) {
+    uint16_t* q = static_cast<uint16_t*>(qkv);
+    return b2_qk_norm_store(B2_DT_BF16, q, ld_qkv, M, nq, nkv, head_dim, head_dim, head_dim, head_dim, q_norm_w, k_norm_w, eps, k_cache, v_cache,
+                            slot_mapping, stream);
+  }
   return b2_qk_norm_rope_store(qkv, ld_qkv, M, nq, nkv, head_dim, q_norm_w, k_norm_w, eps, positions, cos_sin, k_cache, v_cache, slot_mapping,
                                stream);
 }
 
 int b2_gemm_silu_mul(b2_ctx* ctx, const void* A, int64_t lda, const void* W_pairs, int64_t ldw, void* out, int64_t ldo, int M, int I, int K,
                      void* stream) {
-  if (ctx == nullptr) return B2_ERR_ARG;
+  return b2_gemm_act_mul(ctx, A, lda, W_pairs, ldw, out, ldo, M, I, K, B2_ACT_SILU, stream);
+}
+
+int b2_gemm_act_mul(b2_ctx* ctx, const void* A, int64_t lda, const void* W_pairs, int64_t ldw, void* out, int64_t ldo, int M, int I, int K,
+                    int act, void* stream) {
+  if (ctx == nullptr || (act != B2_ACT_SILU && act != B2_ACT_RELU)) return B2_ERR_ARG;
   if (I <= 0 || I % 8 != 0) return B2_ERR_ARG;
   int rc = check_operands(A, lda, W_pairs, ldw, M, 2 * I, K);
   if (rc != B2_OK) return rc;
@@ -2169,7 +2219,7 @@ int b2_gemm_silu_mul(b2_ctx* ctx, const void* A, int64_t lda, const void* W_pair
   GemmArgs args{};
   args.C = static_cast<uint16_t*>(out);
   args.ldc = ldo;
-  args.silu_pairs = 1;
+  args.pair_act = act;
   return launch_gemm<EPI_STORE>(ctx, A, lda, W_pairs, ldw, M, 2 * I, K, args, 0, static_cast<cudaStream_t>(stream));
 }
 

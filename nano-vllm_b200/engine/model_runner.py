@@ -16,30 +16,11 @@ import torch
 import torch.distributed as dist
 
 from ..layers.sampler import Sampler
-from ..models.qwen3 import Qwen3ForCausalLM
+from ..models.registry import ModelConfig, build_model
 from ..runtime import get_runtime, init_runtime, shutdown_runtime
 from ..utils.context import reset_context, set_context
 
 FUSED_SAMPLER_MAX_ROWS = 256  # b2_lm_head_sample takes one token tile of the feature-lane layout
-
-
-@dataclass
-class ModelConfig:
-    """The fields of a HF Qwen3 config the model reads (nanovllm/models/qwen3.py:127-143,167-171,199-203)."""
-    hidden_size: int
-    num_attention_heads: int
-    num_key_value_heads: int
-    head_dim: int
-    intermediate_size: int
-    num_hidden_layers: int
-    vocab_size: int
-    rms_norm_eps: float = 1e-6
-    rope_theta: float = 1e6
-    max_position_embeddings: int = 40960
-    tie_word_embeddings: bool = False
-    attention_bias: bool = False
-    hidden_act: str = "silu"
-    rope_scaling: dict | None = None
 
 
 QWEN3_0_6B = dict(hidden_size=1024, num_attention_heads=16, num_key_value_heads=8, head_dim=128, intermediate_size=3072,
@@ -53,10 +34,12 @@ QWEN3_32B = dict(hidden_size=5120, num_attention_heads=64, num_key_value_heads=8
 @dataclass
 class Seq:
     """Minimal per-request state: the token ids so far, the KV blocks they
-    occupy and how many leading tokens are already in the cache."""
+    occupy, how many leading tokens are already in the cache and the slot of
+    their recurrent state."""
     token_ids: list[int]
     block_table: list[int] = field(default_factory=list)
     num_cached_tokens: int = 0
+    state_slot: int = -1  # recurrent-state slot, for models that have one
 
     def __len__(self):
         return len(self.token_ids)
@@ -79,7 +62,7 @@ class ModelRunner:
     def __init__(self, config: ModelConfig, *, max_num_seqs: int = 512, max_model_len: int = 4096, max_num_batched_tokens: int = 16384,
                  kvcache_block_size: int = 256, num_kvcache_blocks: int | None = None, gpu_memory_utilization: float = 0.9,
                  enforce_eager: bool = False, oneshot_tokens: int = 1024, timeout_ms: int = 5000, seed: int = 0,
-                 full_weights: dict | None = None, fused_sampler: bool | None = None, sample_seed: int = 0):
+                 full_weights: dict | None = None, fused_sampler: bool | None = None, sample_seed: int = 0, dtype: torch.dtype = torch.bfloat16):
         assert dist.is_initialized(), "create the process group first (world size 1 included), as the reference does"
         self.config = config
         self.rank, self.world = dist.get_rank(), dist.get_world_size()
@@ -89,19 +72,24 @@ class ModelRunner:
         # LM head and sampler in one pass (no [B, vocab] logits, no gather): the default at every world size
         if fused_sampler is None:
             fused_sampler = True
-        self.fused_sampler = fused_sampler
         self.sample_seed = sample_seed
         self.device = torch.device("cuda", torch.cuda.current_device())
         # symmetric buffers exist before the layers are built, so graph capture sees fixed addresses
         self.runtime = init_runtime(max_tokens=max_num_batched_tokens, hidden=config.hidden_size, oneshot_tokens=oneshot_tokens,
-                                    vocab=config.vocab_size, max_seqs=max_num_seqs, timeout_ms=timeout_ms)
+                                    vocab=config.logits_size, max_seqs=max_num_seqs, timeout_ms=timeout_ms)
         prev_dtype = torch.get_default_dtype()
-        torch.set_default_dtype(torch.bfloat16)
+        torch.set_default_dtype(dtype)
         torch.set_default_device(self.device)
         try:
-            self.model = Qwen3ForCausalLM(config)
+            self.model = build_model(config)
+            if dtype != torch.bfloat16 and not getattr(self.model, "runs_in_fp32", False):
+                raise ValueError(f"{config.architecture} runs in bf16 only")
+            self.dtype = dtype
+            self.fused_sampler = fused_sampler and getattr(self.model, "fused_sampling", True)
             if full_weights is not None:
                 self.model.load_full_weights(full_weights)
+            elif hasattr(self.model, "random_init_"):
+                self.model.random_init_(seed)
             else:
                 random_init_(self.model, seed, self.rank)
             self.sampler = Sampler()
@@ -122,23 +110,32 @@ class ModelRunner:
 
     # ---- KV cache (reference :103-121) -------------------------------------
     def _allocate_kv_cache(self, num_blocks: int | None, utilization: float):
-        c = self.config
-        self.num_kv_heads = c.num_key_value_heads // self.world
-        block_bytes = 2 * c.num_hidden_layers * self.block_size * self.num_kv_heads * c.head_dim * 2
+        """Paged K/V for every layer run that attends and, first, a fixed-size state slot per sequence for every run that
+        recurs; what the model asks for is in kv_layers() / state_layers()."""
+        kv, states = self.model.kv_layers(), self.model.state_layers()
+        self.num_state_slots = self.max_num_seqs if states else 0
+        for s in states:
+            s.state = torch.zeros(self.num_state_slots, *s.shape, dtype=torch.float32, device=self.device)
+        itemsize = torch.tensor([], dtype=self.dtype).element_size()
+        block_bytes = sum(self.block_size * l.num_kv_heads * (l.k_dim + l.v_dim) for l in kv) * itemsize
         if num_blocks is None:
             free, total = torch.cuda.mem_get_info()
             budget = int(total * utilization) - (total - free)
-            # activations of the largest prefill step: a few [tokens, widest layer output] bf16 tensors
-            widest = max(2 * c.intermediate_size // self.world, c.hidden_size, (c.num_attention_heads + 2 * c.num_key_value_heads) * c.head_dim // self.world)
-            budget -= 6 * self.max_num_batched_tokens * widest * 2
-            num_blocks = budget // block_bytes
+            # activations of the largest prefill step: a few [tokens, widest layer output] tensors
+            budget -= 6 * self.max_num_batched_tokens * self.model.activation_width() * itemsize
+            num_blocks = budget // block_bytes if block_bytes else -(-self.max_num_seqs * self.max_model_len // self.block_size)
         assert num_blocks > 0, "no memory left for the KV cache"
         self.num_kvcache_blocks = int(num_blocks)
-        self.kv_cache = torch.zeros(2, c.num_hidden_layers, self.num_kvcache_blocks, self.block_size, self.num_kv_heads, c.head_dim,
-                                    dtype=torch.bfloat16, device=self.device)
-        for i, layer in enumerate(self.model.model.layers):
-            layer.self_attn.attn.k_cache = self.kv_cache[0, i]
-            layer.self_attn.attn.v_cache = self.kv_cache[1, i]
+        shapes = {(l.num_kv_heads, l.k_dim, l.v_dim) for l in kv}
+        if len(shapes) == 1 and kv[0].k_dim == kv[0].v_dim:  # one tensor when all layers are alike, as the reference lays it out
+            self.kv_cache = torch.zeros(2, len(kv), self.num_kvcache_blocks, self.block_size, kv[0].num_kv_heads, kv[0].k_dim, dtype=self.dtype,
+                                        device=self.device)
+            for i, l in enumerate(kv):
+                l.k_cache, l.v_cache = self.kv_cache[0, i], self.kv_cache[1, i]
+        else:
+            for l in kv:
+                l.k_cache, l.v_cache = (torch.zeros(self.num_kvcache_blocks, self.block_size, l.num_kv_heads, d, dtype=self.dtype, device=self.device)
+                                        for d in (l.k_dim, l.v_dim))
 
     # ---- batch -> tensors -----------------------------------------------------
     def _h2d(self, values, dtype):
@@ -147,6 +144,12 @@ class ModelRunner:
     def _block_tables(self, seqs: list[Seq]):
         width = max(len(s.block_table) for s in seqs)
         return self._h2d([s.block_table + [-1] * (width - len(s.block_table)) for s in seqs], torch.int32)
+
+    def _state_slots(self, seqs: list[Seq]):
+        if not self.num_state_slots:
+            return None
+        assert all(0 <= s.state_slot < self.num_state_slots for s in seqs), "every sequence needs a state slot"
+        return self._h2d([s.state_slot for s in seqs], torch.int32)
 
     def prepare_prefill(self, seqs: list[Seq], num_new: list[int] | None = None):
         """Tokens [num_cached, num_cached + new) of each sequence are computed;
@@ -164,10 +167,12 @@ class ModelRunner:
             max_q, max_k = max(max_q, end - start), max(max_k, end)
             if s.block_table:
                 slots.extend(s.block_table[p // bs] * bs + p % bs for p in range(start, end))
-        block_tables = self._block_tables(seqs) if cu_k[-1] > cu_q[-1] else None
+        paged = getattr(self.model, "paged_prefill", False)
+        block_tables = self._block_tables(seqs) if paged or cu_k[-1] > cu_q[-1] else None
+        kv_len = self._h2d([b - a for a, b in zip(cu_k[:-1], cu_k[1:])], torch.int32) if paged else None
         ids_t, pos_t = self._h2d(ids, torch.int64), self._h2d(pos, torch.int64)
         set_context(True, self._h2d(cu_q, torch.int32), self._h2d(cu_k, torch.int32), max_q, max_k,
-                    self._h2d(slots, torch.int32) if slots else None, None, block_tables)
+                    self._h2d(slots, torch.int32) if slots else None, kv_len, block_tables, self._state_slots(seqs))
         return ids_t, pos_t
 
     def prepare_decode(self, seqs: list[Seq]):
@@ -178,7 +183,7 @@ class ModelRunner:
         slots = [s.block_table[(len(s) - 1) // bs] * bs + (len(s) - 1) % bs for s in seqs]
         lens = [len(s) for s in seqs]
         set_context(False, slot_mapping=self._h2d(slots, torch.int32), context_lens=self._h2d(lens, torch.int32),
-                    block_tables=self._block_tables(seqs))
+                    block_tables=self._block_tables(seqs), state_slots=self._state_slots(seqs))
         return self._h2d(ids, torch.int64), self._h2d(pos, torch.int64)
 
     # ---- forward ---------------------------------------------------------------
@@ -202,6 +207,9 @@ class ModelRunner:
         gv["context_lens"].zero_()
         gv["context_lens"][:n] = ctx.context_lens
         gv["block_tables"][:n, :ctx.block_tables.size(1)] = ctx.block_tables
+        if ctx.state_slots is not None:
+            gv["state_slots"].fill_(-1)
+            gv["state_slots"][:n] = ctx.state_slots
         self._bt_rows = {}  # the graph's table no longer matches what _decode_graph_step last staged
         self.graphs[bs].replay()
         return gv["outputs"][:n]
@@ -213,7 +221,7 @@ class ModelRunner:
         if getattr(self, "_stage", None) is None:
             gv = self.graph_vars
             self._stage = {k: torch.zeros(gv[k].shape, dtype=gv[k].dtype, pin_memory=True) for k in
-                           ("input_ids", "positions", "slot_mapping", "context_lens", "block_tables")}
+                           ("input_ids", "positions", "slot_mapping", "context_lens", "block_tables", "state_slots") if k in gv}
             self._stage_np = {k: v.numpy() for k, v in self._stage.items()}
             self._bt_rows = {}  # row of the staged block table -> the blocks last copied into the graph's table for it
         return self._stage, self._stage_np
@@ -246,7 +254,12 @@ class ModelRunner:
                 rows[i] = key
                 dirty = True
         gv = self.graph_vars
-        for k in ("input_ids", "positions", "slot_mapping", "context_lens"):
+        staged = ["input_ids", "positions", "slot_mapping", "context_lens"]
+        if self.num_state_slots:
+            np_["state_slots"][:n] = [s.state_slot for s in seqs]
+            np_["state_slots"][n:bs] = -1
+            staged.append("state_slots")
+        for k in staged:
             gv[k][:bs].copy_(stage[k][:bs], non_blocking=True)
         if dirty:
             gv["block_tables"][:n, :width].copy_(stage["block_tables"][:n, :width], non_blocking=True)
@@ -254,15 +267,31 @@ class ModelRunner:
         set_context(False)  # the LM head only needs to know this is not a prefill step
         return gv["outputs"][:n]
 
+    def _step_hidden(self, seqs: list[Seq], is_prefill: bool, num_new: list[int] | None):
+        if not is_prefill and not self.enforce_eager and len(seqs) <= self.graph_bs[-1]:
+            return self._decode_graph_step(seqs)
+        ids, pos = self.prepare_prefill(seqs, num_new) if is_prefill else self.prepare_decode(seqs)
+        return self.run_hidden(ids, pos, is_prefill)
+
+    @torch.inference_mode()
+    def step_logits(self, seqs: list[Seq], is_prefill: bool, num_new: list[int] | None = None, rows: list[int] = ()) -> torch.Tensor:
+        """The forward pass of step() without sampling: fp32 logits [len(rows), vocab] on the host for the given rows of
+        the step's tokens (in batch order)."""
+        hidden = self._step_hidden(seqs, is_prefill, num_new)
+        out = torch.empty(len(rows), self.config.vocab_size, dtype=torch.float32)
+        for a in range(0, len(rows), self.max_num_seqs):  # the logits buffer holds max_num_seqs rows
+            part = rows[a:a + self.max_num_seqs]
+            out[a:a + len(part)] = self.model.logits_of_rows(hidden, self._h2d(list(part), torch.int32)).float().cpu()
+        torch.cuda.synchronize()
+        reset_context()
+        self.runtime.check_status()
+        return out
+
     @torch.inference_mode()
     def step(self, seqs: list[Seq], is_prefill: bool, temperatures: list[float] | None = None, num_new: list[int] | None = None):
         """One forward pass + sampling on rank 0; the chosen token ids are
         returned on every rank.  temperatures=None means greedy (argmax)."""
-        if not is_prefill and not self.enforce_eager and len(seqs) <= self.graph_bs[-1]:
-            hidden = self._decode_graph_step(seqs)
-        else:
-            ids, pos = self.prepare_prefill(seqs, num_new) if is_prefill else self.prepare_decode(seqs)
-            hidden = self.run_hidden(ids, pos, is_prefill)
+        hidden = self._step_hidden(seqs, is_prefill, num_new)
         if getattr(self, "_picked", None) is None or self._picked.numel() < len(seqs):
             self._picked = torch.zeros(max(len(seqs), self.max_num_seqs), dtype=torch.int64, device=self.device)
         picked = self._picked[:len(seqs)]  # one buffer for every step: rank 0's sampler fills it, the broadcast hands it to the others
@@ -297,13 +326,16 @@ class ModelRunner:
             slot_mapping=torch.full((max_bs,), -1, dtype=torch.int32, device=dev),
             context_lens=torch.zeros(max_bs, dtype=torch.int32, device=dev),
             block_tables=torch.zeros(max_bs, max_blocks, dtype=torch.int32, device=dev),
-            outputs=torch.zeros(max_bs, c.hidden_size, dtype=torch.bfloat16, device=dev),
+            outputs=torch.zeros(max_bs, c.hidden_size, dtype=self.dtype, device=dev),
         )
+        if self.num_state_slots:
+            gv["state_slots"] = torch.full((max_bs,), -1, dtype=torch.int32, device=dev)
+        self.graph_vars = gv
         self.graph_bs = [b for b in (1, 2, 4, 8) if b <= max_bs] + list(range(16, max_bs + 1, 16))
         self.graph_pool = None
         for bs in reversed(self.graph_bs):
             graph = torch.cuda.CUDAGraph()
-            set_context(False, slot_mapping=gv["slot_mapping"][:bs], context_lens=gv["context_lens"][:bs], block_tables=gv["block_tables"][:bs])
+            self._graph_context(bs)
             gv["outputs"][:bs] = self.model(gv["input_ids"][:bs], gv["positions"][:bs])  # warm-up (also runs the collectives once)
             with torch.cuda.graph(graph, self.graph_pool):
                 gv["outputs"][:bs] = self.model(gv["input_ids"][:bs], gv["positions"][:bs])
@@ -312,7 +344,12 @@ class ModelRunner:
             self.graphs[bs] = graph
             torch.cuda.synchronize()
             reset_context()
-        self.graph_vars = gv
+
+    def _graph_context(self, bs: int) -> None:
+        """The step context over the graphs' input buffers."""
+        gv = self.graph_vars
+        set_context(False, slot_mapping=gv["slot_mapping"][:bs], context_lens=gv["context_lens"][:bs], block_tables=gv["block_tables"][:bs],
+                    state_slots=gv["state_slots"][:bs] if self.num_state_slots else None)
 
 
 class ResidentDecoder:
@@ -332,6 +369,8 @@ class ResidentDecoder:
         gv = runner.graph_vars
         gv["slot_mapping"].fill_(-1)
         gv["context_lens"].zero_()
+        if runner.num_state_slots:
+            gv["state_slots"].fill_(-1)
         before = ops._abi.launch_count()
         self._body()  # warm-up: also creates the logits view outside the capture
         self.kernels_per_step = ops._abi.launch_count() - before
@@ -346,7 +385,7 @@ class ResidentDecoder:
     @torch.inference_mode()
     def _body(self):
         r, bs, gv = self.r, self.bs, self.r.graph_vars
-        set_context(False, slot_mapping=gv["slot_mapping"][:bs], context_lens=gv["context_lens"][:bs], block_tables=gv["block_tables"][:bs])
+        r._graph_context(bs)
         hidden = r.model(gv["input_ids"][:bs], gv["positions"][:bs])
         if r.fused_sampler and bs <= FUSED_SAMPLER_MAX_ROWS:
             r.model.sample_tokens(hidden, None, r.sample_seed, out=self.tokens)  # greedy: rank 0 gets the picks
@@ -373,6 +412,8 @@ class ResidentDecoder:
         gv["positions"][:n] = r._h2d([len(s) - 1 for s in seqs], torch.int64)
         gv["context_lens"][:n] = r._h2d([len(s) for s in seqs], torch.int32)
         gv["slot_mapping"][:n] = r._h2d([s.block_table[(len(s) - 1) // bs] * bs + (len(s) - 1) % bs for s in seqs], torch.int32)
+        if r.num_state_slots:
+            gv["state_slots"][:n] = r._state_slots(seqs)
         r._bt_rows = {}  # the graph's table is rewritten here: _decode_graph_step must stage its rows again
         gv["block_tables"][:n].fill_(-1)  # columns past a sequence's own blocks: no room (the advance kernel freezes such a row)
         gv["block_tables"][:n, :width] = r._h2d([s.block_table + [-1] * (width - len(s.block_table)) for s in seqs], torch.int32)

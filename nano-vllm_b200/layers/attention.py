@@ -14,6 +14,7 @@ from torch import nn
 
 from .. import ops
 from ..utils.context import get_context
+from .linear import HeadsLinear, MergeHeadsLinear, pad8
 
 try:  # the attention library is outside this path; it is only called, never re-implemented
     from flash_attn import flash_attn_varlen_func, flash_attn_with_kvcache
@@ -63,6 +64,7 @@ class Attention(nn.Module):
     def __init__(self, num_heads, head_dim, scale, num_kv_heads):
         super().__init__()
         self.num_heads, self.head_dim, self.scale, self.num_kv_heads = num_heads, head_dim, scale, num_kv_heads
+        self.k_dim = self.v_dim = head_dim
         self.k_cache = self.v_cache = torch.tensor([])
 
     def attend(self, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor) -> torch.Tensor:
@@ -101,3 +103,49 @@ class Attention(nn.Module):
         if self.k_cache.numel() and self.v_cache.numel():
             store_kvcache(k, v, self.k_cache, self.v_cache, get_context().slot_mapping)
         return self.attend(q, k, v)
+
+
+class PagedKV:
+    """One layer run's K and V in the paged cache, bound by the runner; K and V heads may differ in size."""
+
+    def __init__(self, num_kv_heads: int, k_dim: int, v_dim: int):
+        self.num_kv_heads, self.k_dim, self.v_dim = num_kv_heads, k_dim, v_dim
+        self.k_cache = self.v_cache = torch.tensor([])
+
+
+class WindowAttention(nn.Module):
+    """Grouped-query attention without rotation: q/k head norm, soft-capped scores, a sliding window that keeps the first
+    tokens, a learned sink per head in the softmax's denominator.  Always reads K and V from the paged cache."""
+
+    def __init__(self, hidden_size: int, num_heads: int, num_kv_heads: int, dim: int, vdim: int, scale: float, softcap: float, window: int,
+                 keep_first: int, eps: float) -> None:
+        super().__init__()
+        if num_heads % num_kv_heads:
+            raise ValueError(f"{num_heads} query heads do not divide over {num_kv_heads} key/value heads")
+        self.num_heads, self.num_kv_heads, self.dim, self.vdim = num_heads, num_kv_heads, dim, vdim
+        self.qk_pad, self.v_pad = pad8(dim), pad8(vdim)
+        self.scale, self.softcap, self.window, self.keep_first, self.eps = scale, softcap, window, keep_first, eps
+        self.qkv_proj = HeadsLinear(hidden_size, [(num_heads, dim), (num_kv_heads, dim), (num_kv_heads, vdim)])
+        self.o_proj = MergeHeadsLinear(num_heads, vdim, hidden_size)
+        self.q_norm = nn.Parameter(torch.zeros(self.qk_pad), requires_grad=False)
+        self.k_norm = nn.Parameter(torch.zeros(self.qk_pad), requires_grad=False)
+        self.sink = nn.Parameter(torch.zeros(num_heads, dtype=torch.float32), requires_grad=False)
+        for p in (self.q_norm, self.k_norm):
+            p.weight_loader = self._load_norm
+
+    def _load_norm(self, param: nn.Parameter, loaded_weight: torch.Tensor):
+        param.data[:self.dim].copy_(loaded_weight)
+
+    def forward(self, x: torch.Tensor, cache: PagedKV) -> torch.Tensor:
+        ctx = get_context()
+        if x.dtype == torch.bfloat16 and self.dim == self.vdim == 128:  # one launch for decode-sized batches
+            qkv = ops.qkv_fused(x, self.qkv_proj.weight, None, self.num_heads, self.num_kv_heads, 128, self.q_norm, self.k_norm, self.eps,
+                                None, None, cache.k_cache, cache.v_cache, ctx.slot_mapping)
+        else:
+            qkv = self.qkv_proj(x)
+            ops.qk_norm_store(qkv, self.num_heads, self.num_kv_heads, self.dim, self.qk_pad, self.vdim, self.v_pad, self.q_norm, self.k_norm,
+                              self.eps, cache.k_cache, cache.v_cache, ctx.slot_mapping)
+        o = ops.window_attention(qkv, self.num_heads, cache.k_cache, cache.v_cache, ctx.block_tables, ctx.cu_seqlens_q if ctx.is_prefill else None,
+                                 ctx.context_lens, ctx.max_seqlen_q if ctx.is_prefill else 1, ctx.max_seqlen_k if ctx.is_prefill else 2 ** 31 - 1,
+                                 self.scale, self.softcap, self.window, self.keep_first, self.sink)
+        return self.o_proj(o)

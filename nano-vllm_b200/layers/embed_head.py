@@ -13,7 +13,7 @@ from torch import nn
 
 from .. import ops
 from ..utils.context import get_context
-from .linear import _tp_rank_world
+from .linear import _tp_rank_world, pad8
 
 
 class VocabParallelEmbedding(nn.Module):
@@ -51,5 +51,40 @@ class ParallelLMHead(VocabParallelEmbedding):
         """forward() followed by Sampler.forward (nanovllm/layers/sampler.py:7-12; greedy when temperatures is
         None) without materialising the logits: every rank scans its vocabulary slice in the GEMM epilogue and
         only the best (score, id) per row reaches rank 0.  Returns int64 token ids, valid on rank 0."""
+        ctx = get_context()
+        return ops.lm_head_sample(x, self.weight, ctx.last_token_index if ctx.is_prefill else None, temperatures, seed, out)
+
+
+class TiedEmbedding(nn.Module):
+    """One table [vocab, width] that serves as embedding (read by the first stream launch) and as LM head.  Stored padded
+    to multiples of 8 in both directions; the padded vocabulary entries never leave this class."""
+
+    def __init__(self, num_embeddings: int, embedding_dim: int):
+        super().__init__()
+        self.num_embeddings, self.embedding_dim = num_embeddings, embedding_dim
+        self.weight = nn.Parameter(torch.zeros(pad8(num_embeddings), pad8(embedding_dim)), requires_grad=False)
+        self.weight.weight_loader = self.weight_loader
+
+    @property
+    def fused_sampling(self) -> bool:
+        """The LM head fused with the sampler scans every stored entry, so it needs a vocabulary without padding."""
+        return self.weight.dtype == torch.bfloat16 and self.weight.shape[0] == self.num_embeddings
+
+    def weight_loader(self, param: nn.Parameter, loaded_weight: torch.Tensor):
+        param.data[:self.num_embeddings, :self.embedding_dim].copy_(loaded_weight)
+
+    def logits(self, x: torch.Tensor, rows: torch.Tensor | None) -> torch.Tensor:
+        """Logits of the rows of x picked by int32 `rows` (None: all).  bf16 results are a view of the runtime's buffer."""
+        if x.dtype == torch.float32:
+            y = ops.gemm(x if rows is None else x[rows.long()], self.weight)
+        else:
+            y = ops.lm_head(x, self.weight, rows)
+        return y[:, :self.num_embeddings]
+
+    def head(self, x: torch.Tensor) -> torch.Tensor:
+        ctx = get_context()
+        return self.logits(x, ctx.last_token_index if ctx.is_prefill else None)
+
+    def head_sample(self, x: torch.Tensor, temperatures: torch.Tensor | None, seed: int, out: torch.Tensor | None = None):
         ctx = get_context()
         return ops.lm_head_sample(x, self.weight, ctx.last_token_index if ctx.is_prefill else None, temperatures, seed, out)

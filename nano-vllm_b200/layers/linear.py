@@ -186,3 +186,47 @@ class RowParallelLinear(LinearBase):
 
     def forward_fused(self, x: torch.Tensor, residual: torch.Tensor, norm) -> tuple[torch.Tensor, torch.Tensor]:
         return ops.rowpar_fused(x, self.weight, self.bias, residual, norm.weight, norm.eps)
+
+
+def pad8(n: int) -> int:
+    """Sizes are stored in multiples of 8 elements, so that every row and every head starts on a 16-byte boundary."""
+    return (n + 7) // 8 * 8
+
+
+class HeadsLinear(nn.Module):
+    """Several head-structured projections of one input, stacked along the output dimension: section (heads, dim)
+    takes heads * pad8(dim) rows, the rows that pad a head are zero.  The first `silu_sections` sections leave the
+    product activated.  A checkpoint tensor [heads * dim, in] is loaded by section number."""
+
+    def __init__(self, input_size: int, sections: list[tuple[int, int]], silu_sections: int = 0):
+        super().__init__()
+        self.input_size, self.sections = input_size, list(sections)
+        self.widths = [h * pad8(d) for h, d in sections]
+        self.silu_cols = sum(self.widths[:silu_sections])
+        self.weight = nn.Parameter(torch.zeros(sum(self.widths), pad8(input_size)), requires_grad=False)
+        self.weight.weight_loader = self.weight_loader
+
+    def weight_loader(self, param: nn.Parameter, loaded_weight: torch.Tensor, shard_id: int):
+        heads, dim = self.sections[shard_id]
+        rows = param.data.narrow(0, sum(self.widths[:shard_id]), self.widths[shard_id])
+        rows.view(heads, pad8(dim), -1)[:, :dim, :self.input_size].copy_(loaded_weight.view(heads, dim, self.input_size))
+
+    def forward(self, x: torch.Tensor) -> torch.Tensor:
+        return ops.gemm(x, self.weight, silu_cols=self.silu_cols)
+
+
+class MergeHeadsLinear(nn.Module):
+    """Projection of concatenated heads [tokens, heads * pad8(dim)] back to the model's width (weight columns that meet
+    a head's padding are zero)."""
+
+    def __init__(self, heads: int, dim: int, output_size: int):
+        super().__init__()
+        self.heads, self.dim, self.output_size = heads, dim, output_size
+        self.weight = nn.Parameter(torch.zeros(pad8(output_size), heads * pad8(dim)), requires_grad=False)
+        self.weight.weight_loader = self.weight_loader
+
+    def weight_loader(self, param: nn.Parameter, loaded_weight: torch.Tensor):
+        param.data.view(-1, self.heads, pad8(self.dim))[:self.output_size, :, :self.dim].copy_(loaded_weight.view(self.output_size, self.heads, self.dim))
+
+    def forward(self, x: torch.Tensor) -> torch.Tensor:
+        return ops.gemm(x, self.weight)

@@ -17,4 +17,4 @@ class Sampler(nn.Module):
 
     @staticmethod
     def greedy(logits: torch.Tensor) -> torch.Tensor:
-        return ops.argmax(logits)
+        return ops.argmax(logits) if logits.dtype == torch.bfloat16 else logits.argmax(dim=-1)

@@ -144,16 +144,31 @@ class Qwen3ForCausalLM(nn.Module):
 
     def __init__(self, config) -> None:
         super().__init__()
+        self.config = config
         self.model = Qwen3Model(config)
         self.lm_head = ParallelLMHead(config.vocab_size, config.hidden_size)
         if config.tie_word_embeddings:
             self.lm_head.weight.data = self.model.embed_tokens.weight.data
+
+    def kv_layers(self) -> list[Attention]:
+        return [l.self_attn.attn for l in self.model.layers]
+
+    def state_layers(self) -> list:
+        return []
+
+    def activation_width(self) -> int:
+        """Elements per token of the widest layer output on this rank."""
+        c, (_, tp) = self.config, _tp_rank_world()
+        return max(2 * c.intermediate_size // tp, c.hidden_size, (c.num_attention_heads + 2 * c.num_key_value_heads) * c.head_dim // tp)
 
     def forward(self, input_ids: torch.Tensor, positions: torch.Tensor) -> torch.Tensor:
         return self.model(input_ids, positions)
 
     def compute_logits(self, hidden_states: torch.Tensor):
         return self.lm_head(hidden_states)
+
+    def logits_of_rows(self, hidden_states: torch.Tensor, rows: torch.Tensor):
+        return ops.lm_head(hidden_states, self.lm_head.weight, rows)
 
     def sample_tokens(self, hidden_states: torch.Tensor, temperatures: torch.Tensor | None, seed: int, out: torch.Tensor | None = None):
         """compute_logits + the sampler in one pass (token ids valid on rank 0); see ParallelLMHead.forward_sample."""

@@ -30,8 +30,39 @@ def _as2d(t: torch.Tensor) -> torch.Tensor:
     return t.reshape(-1, t.shape[-1])
 
 
-def gemm(x: torch.Tensor, w: torch.Tensor, bias: torch.Tensor | None = None) -> torch.Tensor:
-    """x[..., K] @ w[N, K]^T (+ bias)."""
+def _dt(t: torch.Tensor) -> int:
+    """The library's element-type code of a tensor."""
+    if t.dtype == torch.bfloat16:
+        return _abi.DT_BF16
+    if t.dtype == torch.float32:
+        return _abi.DT_F32
+    raise TypeError(f"expected bf16 or fp32, got {t.dtype}")
+
+
+def _ptr(t: torch.Tensor | None):
+    return None if t is None else t.data_ptr()
+
+
+def _gemm_f32(x: torch.Tensor, w: torch.Tensor, pair_act: int = _abi.ACT_NONE, silu_cols: int = 0) -> torch.Tensor:
+    """The fp32 form of gemm / gemm_act_mul: true 32-bit products."""
+    x2 = _as2d(x)
+    if x2.stride(-1) != 1 or x2.stride(0) % 4 or x2.data_ptr() % 16:
+        x2 = x2.contiguous()
+    M, K = x2.shape
+    N = w.shape[0]
+    if w.dtype != torch.float32 or w.shape[1] != K:
+        raise ValueError(f"fp32 gemm: input has {K} features, weight is {tuple(w.shape)} {w.dtype}")
+    out = torch.empty(M, N // 2 if pair_act else N, dtype=torch.float32, device=x.device)
+    _abi.check(_lib.b2_gemm_f32(x2.data_ptr(), x2.stride(0), w.data_ptr(), w.stride(0), out.data_ptr(), out.stride(0), M, N, K, pair_act,
+                                silu_cols, _stream()), "b2_gemm_f32")
+    return out.view(*x.shape[:-1], out.shape[1])
+
+
+def gemm(x: torch.Tensor, w: torch.Tensor, bias: torch.Tensor | None = None, silu_cols: int = 0) -> torch.Tensor:
+    """x[..., K] @ w[N, K]^T (+ bias); the first silu_cols output features leave as silu(x)."""
+    if x.dtype == torch.float32:
+        assert bias is None
+        return _gemm_f32(x, w, silu_cols=silu_cols)
     lead = x.shape[:-1]
     x2 = _as2d(_bf16_rows(x, "gemm input"))
     if x2.stride(0) % 8 != 0 or x2.data_ptr() % 16 != 0:
@@ -42,23 +73,27 @@ def gemm(x: torch.Tensor, w: torch.Tensor, bias: torch.Tensor | None = None) -> 
     if w.dim() != 2 or w.shape[1] != K:
         raise ValueError(f"gemm: input has {K} features, weight is {tuple(w.shape)}")
     out = torch.empty(M, N, dtype=torch.bfloat16, device=x.device)
-    if M:
+    if M and silu_cols:
+        assert bias is None
+        _abi.check(_lib.b2_gemm_silu_cols(get_runtime().ctx, x2.data_ptr(), x2.stride(0), w.data_ptr(), w.stride(0), out.data_ptr(), out.stride(0),
+                                          M, N, K, silu_cols, _stream()), "b2_gemm_silu_cols")
+    elif M:
         _abi.check(_lib.b2_gemm(get_runtime().ctx, x2.data_ptr(), x2.stride(0), w.data_ptr(), w.stride(0),
                                 bias.data_ptr() if bias is not None else None, out.data_ptr(), out.stride(0), M, N, K, _stream()), "b2_gemm")
     return out.view(*lead, N)
 
 
 def qkv_fused(x: torch.Tensor, w: torch.Tensor, bias, nq: int, nkv: int, head_dim: int, q_norm_w, k_norm_w, eps: float,
-              positions: torch.Tensor, cos_sin: torch.Tensor, k_cache, v_cache, slot_mapping) -> torch.Tensor:
+              positions: torch.Tensor | None, cos_sin: torch.Tensor | None, k_cache, v_cache, slot_mapping) -> torch.Tensor:
     """qkv projection + q/k head norm + RoPE + KV scatter; returns the [M, (nq + 2 nkv) head_dim] tensor with q and k
-    already normalised and rotated."""
+    already normalised and rotated (cos_sin None: not rotated)."""
     x2 = _as2d(_bf16_rows(x, "qkv input"))
     if x2.stride(0) % 8 != 0 or x2.data_ptr() % 16 != 0:
         x2 = x2.contiguous()
     M, K = x2.shape
     N = w.shape[0]
     assert N == (nq + 2 * nkv) * head_dim and w.shape[1] == K
-    assert positions.dtype == torch.int64 and cos_sin.dtype == torch.float32 and cos_sin.is_contiguous()
+    assert cos_sin is None or (positions.dtype == torch.int64 and cos_sin.dtype == torch.float32 and cos_sin.is_contiguous())
     have_cache = k_cache is not None and k_cache.numel() > 0
     if have_cache:
         assert k_cache.stride(1) == nkv * head_dim and slot_mapping.dtype == torch.int32
@@ -67,7 +102,7 @@ def qkv_fused(x: torch.Tensor, w: torch.Tensor, bias, nq: int, nkv: int, head_di
         _abi.check(_lib.b2_qkv_fused(get_runtime().ctx, x2.data_ptr(), x2.stride(0), w.data_ptr(), w.stride(0),
                                      bias.data_ptr() if bias is not None else None, out.data_ptr(), out.stride(0), M, nq, nkv, head_dim, K,
                                      q_norm_w.data_ptr() if q_norm_w is not None else None, k_norm_w.data_ptr() if k_norm_w is not None else None,
-                                     float(eps), positions.data_ptr(), cos_sin.data_ptr(), k_cache.data_ptr() if have_cache else None,
+                                     float(eps), _ptr(positions), _ptr(cos_sin), k_cache.data_ptr() if have_cache else None,
                                      v_cache.data_ptr() if have_cache else None, slot_mapping.data_ptr() if have_cache else None, _stream()),
                    "b2_qkv_fused")
     return out
@@ -75,18 +110,25 @@ def qkv_fused(x: torch.Tensor, w: torch.Tensor, bias, nq: int, nkv: int, head_di
 
 def gemm_silu_mul(x: torch.Tensor, w_pairs: torch.Tensor) -> torch.Tensor:
     """silu(x @ gate^T) * (x @ up^T) where w_pairs interleaves gate and up rows (gate_0, up_0, gate_1, ...)."""
+    return gemm_act_mul(x, w_pairs, _abi.ACT_SILU)
+
+
+def gemm_act_mul(x: torch.Tensor, w_pairs: torch.Tensor, act: int) -> torch.Tensor:
+    """act(x @ gate^T) * (x @ up^T), act one of _abi.ACT_SILU / ACT_RELU."""
+    if x.dtype == torch.float32:
+        return _gemm_f32(x, w_pairs, pair_act=act)
     lead = x.shape[:-1]
-    x2 = _as2d(_bf16_rows(x, "gemm_silu_mul input"))
+    x2 = _as2d(_bf16_rows(x, "gemm_act_mul input"))
     if x2.stride(0) % 8 != 0 or x2.data_ptr() % 16 != 0:
         x2 = x2.contiguous()
     M, K = x2.shape
     I = w_pairs.shape[0] // 2
     if w_pairs.shape[1] != K or w_pairs.shape[0] % 2:
-        raise ValueError(f"gemm_silu_mul: input has {K} features, paired weight is {tuple(w_pairs.shape)}")
+        raise ValueError(f"gemm_act_mul: input has {K} features, paired weight is {tuple(w_pairs.shape)}")
     out = torch.empty(M, I, dtype=torch.bfloat16, device=x.device)
     if M:
-        _abi.check(_lib.b2_gemm_silu_mul(get_runtime().ctx, x2.data_ptr(), x2.stride(0), w_pairs.data_ptr(), w_pairs.stride(0),
-                                         out.data_ptr(), out.stride(0), M, I, K, _stream()), "b2_gemm_silu_mul")
+        _abi.check(_lib.b2_gemm_act_mul(get_runtime().ctx, x2.data_ptr(), x2.stride(0), w_pairs.data_ptr(), w_pairs.stride(0),
+                                        out.data_ptr(), out.stride(0), M, I, K, act, _stream()), "b2_gemm_act_mul")
     return out.view(*lead, I)
 
 
@@ -280,6 +322,101 @@ def lm_head_sample(h: torch.Tensor, w: torch.Tensor, row_index: torch.Tensor | N
                                       w.data_ptr(), w.stride(0), B, Vr, H, temperatures.data_ptr() if temperatures is not None else None,
                                       int(seed) & 0xFFFFFFFFFFFFFFFF, out.data_ptr(), _stream()), "b2_lm_head_sample")
     return out[:B]
+
+
+def stream_step(x: torch.Tensor, y: torch.Tensor | None, mix, w_out, mult: float, w_in, norm_w: torch.Tensor, eps: float, dim: int,
+                store: bool = True, embed: tuple | None = None, dtype: torch.dtype | None = None) -> torch.Tensor:
+    """Everything between two sublayers on the fp32 residual streams x [M, S, D] (updated in place unless store is
+    False): x <- mix^T x + mult w_out y, then RMSNorm(sum_s w_in[s] x_s) * norm_w, which is returned.  w_in None = all
+    ones.  embed = (ids, table, scale) fills x from the embedding table instead of reading it."""
+    M, S, D = x.shape
+    assert x.dtype == torch.float32 and x.is_contiguous()
+    if y is not None:
+        assert y.shape == (M, D) and y.stride(1) == 1 and mix.dtype == torch.float32 and w_out.dtype == torch.float32
+    assert norm_w.dtype == torch.float32 and norm_w.numel() == D and (w_in is None or w_in.dtype == torch.float32)
+    ids, table, scale = embed if embed is not None else (None, None, 1.0)
+    dtype = y.dtype if y is not None else table.dtype if table is not None else dtype
+    normed = torch.empty(M, D, dtype=dtype, device=x.device)
+    _abi.check(_lib.b2_stream_step(_dt(normed), x.data_ptr() if store else None, None if embed is not None else x.data_ptr(), _ptr(ids), _ptr(table),
+                                   table.stride(0) if table is not None else 0, table.shape[0] if table is not None else 0, float(scale),
+                                   _ptr(y), y.stride(0) if y is not None else 0, _ptr(mix) if y is not None else None,
+                                   _ptr(w_out) if y is not None else None, float(mult), _ptr(w_in), norm_w.data_ptr(), float(eps),
+                                   normed.data_ptr(), D, M, S, dim, D, _stream()), "b2_stream_step")
+    return normed
+
+
+def qk_norm_store(qkv: torch.Tensor, nq: int, nkv: int, qk_dim: int, qk_pad: int, v_dim: int, v_pad: int, q_norm_w, k_norm_w, eps: float,
+                  k_cache, v_cache, slot_mapping) -> None:
+    """q/k head RMSNorm (no rotation) in place on [q heads | k heads | v heads] rows and the scatter into the paged cache."""
+    assert qkv.dim() == 2 and qkv.stride(1) == 1
+    have_cache = k_cache is not None and k_cache.numel() > 0
+    if have_cache:
+        assert k_cache.dtype == qkv.dtype and k_cache.stride(1) == nkv * qk_pad and v_cache.stride(1) == nkv * v_pad and slot_mapping.dtype == torch.int32
+    _abi.check(_lib.b2_qk_norm_store(_dt(qkv), qkv.data_ptr(), qkv.stride(0), qkv.shape[0], nq, nkv, qk_dim, qk_pad, v_dim, v_pad, _ptr(q_norm_w),
+                                     _ptr(k_norm_w), float(eps), _ptr(k_cache) if have_cache else None, _ptr(v_cache) if have_cache else None,
+                                     _ptr(slot_mapping) if have_cache else None, _stream()), "b2_qk_norm_store")
+
+
+_WORKSPACES: dict = {}
+
+
+def _workspace(kind: str, nbytes: int, device) -> torch.Tensor | None:
+    """Scratch shared by the calls of one kind (stream-ordered); grows, never shrinks.  Starts as zeros.  A larger buffer
+    replaces the old one, which stays alive because a captured graph may hold its address."""
+    if nbytes <= 0:
+        return None
+    held = _WORKSPACES.setdefault((kind, device), [])
+    if not held or held[-1].numel() < nbytes:
+        held.append(torch.zeros(nbytes, dtype=torch.uint8, device=device))
+    return held[-1]
+
+
+def window_attention(q: torch.Tensor, out_heads: int, k_cache: torch.Tensor, v_cache: torch.Tensor, block_tables: torch.Tensor, cu_q, kv_len,
+                     max_q: int, max_kv: int, scale: float, softcap: float, window: int, keep_first: int, sink, form: int = 0) -> torch.Tensor:
+    """Attention of q [M, >= nq * qk_pad] over the paged cache [blocks, block_size, nkv, dim]; cu_q None = decode (one row
+    per sequence).  Returns [M, nq * v_pad]."""
+    nkv, qk_pad, v_pad = k_cache.shape[2], k_cache.shape[3], v_cache.shape[3]
+    M, B = q.shape[0], kv_len.numel() if cu_q is None else cu_q.numel() - 1
+    assert q.stride(1) == 1 and q.dtype == k_cache.dtype and k_cache.is_contiguous() and v_cache.is_contiguous()
+    assert block_tables.dtype == torch.int32 and kv_len.dtype == torch.int32 and (sink is None or sink.dtype == torch.float32)
+    out = torch.empty(M, out_heads * v_pad, dtype=q.dtype, device=q.device)
+    max_kv = min(max_kv, block_tables.shape[1] * k_cache.shape[1])
+    window = min(window, 2 ** 31 - 1)
+    nbytes = _lib.b2_attention_workspace(_dt(q), B, max_q, max_kv, out_heads, nkv, qk_pad, v_pad, window, keep_first)
+    ws = _workspace("attention", nbytes, q.device)
+    _abi.check(_lib.b2_attention(_dt(q), q.data_ptr(), q.stride(0), out.data_ptr(), out.stride(0), k_cache.data_ptr(), v_cache.data_ptr(),
+                                 block_tables.data_ptr(), block_tables.stride(0), k_cache.shape[1], _ptr(cu_q), kv_len.data_ptr(), B, max_q, max_kv,
+                                 out_heads, nkv, qk_pad, v_pad, float(scale), float(softcap), window, keep_first, _ptr(sink), _ptr(ws),
+                                 ws.numel() if ws is not None else 0, form, _stream()), "b2_attention")
+    return out
+
+
+def linear_attn(qkv: torch.Tensor, heads: int, qk_pad: int, v_pad: int, state: torch.Tensor, slots: torch.Tensor, cu_q, kv_len: torch.Tensor,
+                max_q: int, decay: torch.Tensor, decay_powers: torch.Tensor, form: int = 0) -> torch.Tensor:
+    """Decayed linear attention on rows [q heads | k heads | v heads | ...]; returns o [M, heads * v_pad] in fp32 and leaves
+    the new state in `state` [slots, heads, qk_pad, v_pad]."""
+    assert qkv.dim() == 2 and qkv.stride(1) == 1 and qkv.shape[1] >= heads * (2 * qk_pad + v_pad)
+    assert state.dtype == torch.float32 and state.is_contiguous() and state.shape[1:] == (heads, qk_pad, v_pad)
+    assert slots.dtype == torch.int32 and kv_len.dtype == torch.int32
+    assert decay.dtype == torch.float32 and decay_powers.shape == (heads, 65) and decay_powers.is_contiguous()
+    M, B = qkv.shape[0], slots.numel()
+    o = torch.empty(M, heads * v_pad, dtype=torch.float32, device=qkv.device)
+    nbytes = _lib.b2_linear_attn_workspace(_dt(qkv), B, max_q, M, heads, qk_pad, v_pad) if cu_q is not None else 0
+    ws = _workspace("linear_attn", nbytes, qkv.device)
+    _abi.check(_lib.b2_linear_attn(_dt(qkv), qkv.data_ptr(), qkv.stride(0), o.data_ptr(), o.stride(0), state.data_ptr(), slots.data_ptr(), _ptr(cu_q),
+                                   kv_len.data_ptr(), decay.data_ptr(), decay_powers.data_ptr(), B, max_q, M, heads, qk_pad, v_pad, _ptr(ws),
+                                   ws.numel() if ws is not None else 0, form, _stream()), "b2_linear_attn")
+    return o
+
+
+def gated_norm(o: torch.Tensor, gate: torch.Tensor, w: torch.Tensor, eps: float, dim: int) -> torch.Tensor:
+    """o / rms(o) * w * sigmoid(gate) per row, in the gate's dtype; o and w fp32, the mean over `dim` elements."""
+    M, pad = o.shape
+    assert o.dtype == torch.float32 and w.dtype == torch.float32 and gate.shape == (M, pad) and gate.stride(1) == 1
+    out = torch.empty(M, pad, dtype=gate.dtype, device=o.device)
+    _abi.check(_lib.b2_gated_norm(_dt(gate), o.data_ptr(), o.stride(0), gate.data_ptr(), gate.stride(0), w.data_ptr(), float(eps), M, dim, pad,
+                                  out.data_ptr(), out.stride(0), _stream()), "b2_gated_norm")
+    return out
 
 
 def argmax(logits: torch.Tensor, out: torch.Tensor | None = None) -> torch.Tensor:
