@@ -4,10 +4,13 @@
 // switch those parts off.
 //
 //   qk_norm_store_kernel   q/k head RMSNorm and the scatter of K and V into the cache
+//   attn_prefill_kernel    bf16, head sizes up to 128: 64 rows x 64 keys on the tensor cores
+//   attn_decode_kernel     the same for one query row per sequence, keys split over warps and CTAs
 //   attn_any_kernel        any head size, bf16 or fp32, prefill and decode (one warp per query head)
 #include <algorithm>
 #include <climits>
 
+#include "b2_mma.cuh"
 #include "b2_vec.cuh"
 
 namespace {
@@ -188,6 +191,458 @@ __global__ void __launch_bounds__(128) attn_any_kernel(const AttnArgs a, int row
     if (lane + 32 * i < a.v_pad) out[lane + 32 * i] = b2::from_float<T>(acc[i] * inv);
 }
 
+// ---------------------------------------------------------------------------
+// Tensor-core kernels, bf16, head sizes up to 128.  The query heads that share a key/value head are rows of one tile
+// (row = token * rep + head), so K and V are read once per group.  Scores, softmax and weights are fp32; the weights
+// enter the product with V as a sum of two bf16 numbers.
+// ---------------------------------------------------------------------------
+constexpr int BN = 64;  // keys per tile
+
+// The key tiles a range of positions [pmin, pmax] looks at: those of the kept first tokens, then those of the window.
+struct KeyTiles {
+  int n_first, win0, total;
+  __device__ __forceinline__ KeyTiles(int pmin, int pmax, int window, int keep_first) {
+    const int lo = pmin - window + 1;
+    win0 = (lo > 0 ? lo : 0) / BN;
+    const int kept = min(keep_first, pmax + 1);
+    n_first = min((kept + BN - 1) / BN, win0);
+    total = n_first + pmax / BN - win0 + 1;
+  }
+  __device__ __forceinline__ int at(int i) const { return i < n_first ? i : win0 + (i - n_first); }
+};
+
+__device__ __forceinline__ float fast_exp2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+// cap * tanh(s / cap), tanh(x) = 1 - 2 / (1 + e^2x); its Taylor series where that would cancel
+__device__ __forceinline__ float soft_cap(float s, float cap, float inv_cap) {
+  const float x = s * inv_cap;
+  const float e = fast_exp2(x * 2.885390081777927f);  // 2 log2(e)
+  const float t = 1.0f - __fdividef(2.0f, e + 1.0f);
+  const float x2 = x * x;
+  const float series = x * (1.0f + x2 * (-0.33333333333f + x2 * 0.13333333333f));
+  return cap * (fabsf(x) < 0.125f ? series : (e > 1e30f ? 1.0f : t));
+}
+
+constexpr float LOG2E = 1.4426950408889634f;
+
+template <int DQ, int DV>
+__device__ __forceinline__ void load_kv_tile(const AttnArgs& a, const int32_t* bt, int bs_shift, int g, int tile, int last, uint32_t sk, uint32_t sv) {
+  constexpr int QP = DQ / 8, VP = DV / 8;
+  const uint16_t* kc = static_cast<const uint16_t*>(a.k_cache);
+  const uint16_t* vc = static_cast<const uint16_t*>(a.v_cache);
+#pragma unroll
+  for (int i = 0; i < BN * QP / 128; ++i) {
+    const int idx = threadIdx.x + i * 128, r = idx / QP, p = idx % QP, j = tile * BN + r;
+    const bool ok = j <= last && p * 8 < a.qk_pad;
+    int64_t slot = 0;
+    if (ok) slot = bs_shift >= 0 ? (static_cast<int64_t>(__ldg(bt + (j >> bs_shift))) << bs_shift) + (j & ((1 << bs_shift) - 1))
+                                 : static_cast<int64_t>(__ldg(bt + j / a.block_size)) * a.block_size + j % a.block_size;
+    b2::cp_async16(b2::tile_addr<DQ>(sk, r, p), kc + (slot * a.nkv + g) * a.qk_pad + (ok ? p * 8 : 0), ok);
+  }
+#pragma unroll
+  for (int i = 0; i < BN * VP / 128; ++i) {
+    const int idx = threadIdx.x + i * 128, r = idx / VP, p = idx % VP, j = tile * BN + r;
+    const bool ok = j <= last && p * 8 < a.v_pad;
+    int64_t slot = 0;
+    if (ok) slot = bs_shift >= 0 ? (static_cast<int64_t>(__ldg(bt + (j >> bs_shift))) << bs_shift) + (j & ((1 << bs_shift) - 1))
+                                 : static_cast<int64_t>(__ldg(bt + j / a.block_size)) * a.block_size + j % a.block_size;
+    b2::cp_async16(b2::tile_addr<DV>(sv, r, p), vc + (slot * a.nkv + g) * a.v_pad + (ok ? p * 8 : 0), ok);
+  }
+}
+
+// One tile's scores of a warp: NT 8-key column tiles starting at key j0.  Scales, caps, masks (when `masked`), folds
+// into the running maximum m and sum l, and leaves the weights in s.  Returns the factors for the old outputs.
+template <int NT>
+__device__ __forceinline__ void softmax_tile(const AttnArgs& a, float (&s)[NT][4], int j0, const int (&pos)[2], bool masked, float inv_cap,
+                                             float (&m)[2], float (&l)[2], float (&corr)[2], int lane) {
+  float mx[2] = {-INFINITY, -INFINITY};
+#pragma unroll
+  for (int n = 0; n < NT; ++n)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      float v = s[n][e] * a.scale;
+      if (a.softcap > 0.f) v = soft_cap(v, a.softcap, inv_cap);
+      if (masked && !visible(pos[e >> 1], j0 + n * 8 + (lane & 3) * 2 + (e & 1), a.window, a.keep_first)) v = -INFINITY;
+      s[n][e] = v;
+      mx[e >> 1] = fmaxf(mx[e >> 1], v);
+    }
+#pragma unroll
+  for (int h = 0; h < 2; ++h) {
+    mx[h] = fmaxf(mx[h], __shfl_xor_sync(0xffffffffu, mx[h], 1));
+    mx[h] = fmaxf(mx[h], __shfl_xor_sync(0xffffffffu, mx[h], 2));
+    const float m_new = fmaxf(m[h], mx[h]);
+    corr[h] = m_new == -INFINITY ? 1.0f : fast_exp2((m[h] - m_new) * LOG2E);
+    m[h] = m_new;
+  }
+  float sum[2] = {0.f, 0.f};
+#pragma unroll
+  for (int n = 0; n < NT; ++n)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const float p = m[e >> 1] == -INFINITY ? 0.f : fast_exp2((s[n][e] - m[e >> 1]) * LOG2E);
+      s[n][e] = p;
+      sum[e >> 1] += p;
+    }
+#pragma unroll
+  for (int h = 0; h < 2; ++h) l[h] = l[h] * corr[h] + sum[h];  // this lane's part; summed over the row's four lanes at the end
+}
+
+template <int DQ, int DV>
+struct CfgTile {
+  static constexpr int STAGE = BN * (DQ + DV) * 2;
+  static constexpr int SMEM_PREFILL = 64 * DQ * 2 + 2 * STAGE + 128;
+  static constexpr int DEC_STAGES = 3;
+  static constexpr int SMEM_DECODE = 16 * DQ * 2 + DEC_STAGES * STAGE + 128;
+};
+
+// Prefill: 64 rows (token, head of the group) per CTA, 16 per warp; the four warps share the key tiles.
+template <int DQ, int DV>
+__global__ void __launch_bounds__(128, 2) attn_prefill_kernel(const AttnArgs a, int rep, int bs_shift) {
+  extern __shared__ unsigned char smem_raw[];
+  const uint32_t base = (b2::smem_u32(smem_raw) + 127) & ~127u;
+  const uint32_t sq = base, skv = base + 64 * DQ * 2;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  b2::pdl_launch_dependents();
+  b2::pdl_wait();
+  const int b = blockIdx.z, g = blockIdx.y;
+  const int row0 = a.cu_q[b];
+  const int n_q = a.cu_q[b + 1] - row0;
+  const int rows = n_q * rep;
+  const int tile0 = (static_cast<int>(gridDim.x) - 1 - static_cast<int>(blockIdx.x)) * 64;  // the longest rows first
+  if (tile0 >= rows) return;
+  const int klen = a.kv_len[b];
+  const int first_pos = klen - n_q;
+  const int32_t* bt = a.block_tables + b * a.bt_stride;
+  const int pmin = first_pos + tile0 / rep, pmax = first_pos + min(tile0 + 63, rows - 1) / rep;
+  const KeyTiles tiles(pmin, pmax, a.window, a.keep_first);
+  const float inv_cap = a.softcap > 0.f ? 1.0f / a.softcap : 0.f;
+  const uint16_t* q = static_cast<const uint16_t*>(a.q);
+#pragma unroll
+  for (int i = 0; i < 64 * (DQ / 8) / 128; ++i) {
+    const int idx = threadIdx.x + i * 128, r = idx / (DQ / 8), p = idx % (DQ / 8);
+    const int gr = tile0 + r;
+    const bool ok = gr < rows && p * 8 < a.qk_pad;
+    const int tok = ok ? gr / rep : 0, hh = ok ? gr - tok * rep : 0;
+    b2::cp_async16(b2::tile_addr<DQ>(sq, r, p), q + (row0 + tok) * a.ldq + static_cast<int64_t>(g * rep + hh) * a.qk_pad + (ok ? p * 8 : 0), ok);
+  }
+  load_kv_tile<DQ, DV>(a, bt, bs_shift, g, tiles.at(0), pmax, skv, skv + BN * DQ * 2);
+  b2::cp_async_commit();
+  int pos[2];
+#pragma unroll
+  for (int h = 0; h < 2; ++h) pos[h] = first_pos + min(tile0 + warp * 16 + (lane >> 2) + h * 8, rows - 1) / rep;
+  const int wpmin = first_pos + min(tile0 + warp * 16, rows - 1) / rep;
+  const int wpmax = first_pos + min(tile0 + warp * 16 + 15, rows - 1) / rep;
+  float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
+  float o[DV / 8][4];
+#pragma unroll
+  for (int n = 0; n < DV / 8; ++n)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) o[n][e] = 0.f;
+  for (int it = 0; it < tiles.total; ++it) {
+    const uint32_t sk = skv + (it & 1) * CfgTile<DQ, DV>::STAGE, sv = sk + BN * DQ * 2;
+    b2::cp_async_wait<0>();
+    __syncthreads();  // this tile has landed for everyone, and everyone has left the stage that is filled next
+    if (it + 1 < tiles.total) {
+      const uint32_t nk = skv + ((it + 1) & 1) * CfgTile<DQ, DV>::STAGE;
+      load_kv_tile<DQ, DV>(a, bt, bs_shift, g, tiles.at(it + 1), pmax, nk, nk + BN * DQ * 2);
+    }
+    b2::cp_async_commit();
+    const int j0 = tiles.at(it) * BN;
+    float s[BN / 8][4];
+#pragma unroll
+    for (int n = 0; n < BN / 8; ++n)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) s[n][e] = 0.f;
+#pragma unroll
+    for (int k = 0; k < DQ / 16; ++k) {
+      uint32_t qa[4];
+      b2::frag_a<DQ>(sq, warp * 16, k * 16, lane, qa);
+#pragma unroll
+      for (int n = 0; n < BN / 16; ++n) {
+        uint32_t kb[4];
+        b2::frag_b<DQ>(sk, n * 16, k * 16, lane, kb);
+        b2::mma16816(s[2 * n], qa, kb[0], kb[1]);
+        b2::mma16816(s[2 * n + 1], qa, kb[2], kb[3]);
+      }
+    }
+    const bool all_seen = j0 + BN - 1 <= wpmin && (wpmax - j0 < a.window || j0 + BN - 1 < a.keep_first);
+    float corr[2];
+    softmax_tile<BN / 8>(a, s, j0, pos, !all_seen, inv_cap, m, l, corr, lane);
+#pragma unroll
+    for (int n = 0; n < DV / 8; ++n) {
+      o[n][0] *= corr[0]; o[n][1] *= corr[0]; o[n][2] *= corr[1]; o[n][3] *= corr[1];
+    }
+#pragma unroll
+    for (int k = 0; k < BN / 16; ++k) {
+      uint32_t hi[4], lo[4];
+      b2::split_bf16(s[2 * k][0], s[2 * k][1], hi[0], lo[0]);
+      b2::split_bf16(s[2 * k][2], s[2 * k][3], hi[1], lo[1]);
+      b2::split_bf16(s[2 * k + 1][0], s[2 * k + 1][1], hi[2], lo[2]);
+      b2::split_bf16(s[2 * k + 1][2], s[2 * k + 1][3], hi[3], lo[3]);
+#pragma unroll
+      for (int n = 0; n < DV / 16; ++n) {
+        uint32_t vb[4];
+        b2::frag_b_t<DV>(sv, n * 16, k * 16, lane, vb);
+        b2::mma16816(o[2 * n], hi, vb[0], vb[1]);
+        b2::mma16816(o[2 * n + 1], hi, vb[2], vb[3]);
+        b2::mma16816(o[2 * n], lo, vb[0], vb[1]);
+        b2::mma16816(o[2 * n + 1], lo, vb[2], vb[3]);
+      }
+    }
+  }
+  uint16_t* out = static_cast<uint16_t*>(a.out);
+#pragma unroll
+  for (int h = 0; h < 2; ++h) {
+    l[h] += __shfl_xor_sync(0xffffffffu, l[h], 1);
+    l[h] += __shfl_xor_sync(0xffffffffu, l[h], 2);
+    const int gr = tile0 + warp * 16 + (lane >> 2) + h * 8;
+    if (gr >= rows) continue;
+    const int tok = gr / rep, head = g * rep + (gr - tok * rep);
+    float f = 1.0f;
+    if (a.sink != nullptr) {
+      const float sk = a.sink[head], m_new = fmaxf(m[h], sk);
+      f = fast_exp2((m[h] - m_new) * LOG2E);
+      l[h] = l[h] * f + fast_exp2((sk - m_new) * LOG2E);
+    }
+    f /= l[h];
+    uint16_t* dst = out + (row0 + tok) * a.ldo + static_cast<int64_t>(head) * a.v_pad;
+#pragma unroll
+    for (int n = 0; n < DV / 8; ++n) {
+      const int c = n * 8 + (lane & 3) * 2;
+      if (c < a.v_pad) *reinterpret_cast<uint32_t*>(dst + c) = b2::pack_bf16(o[n][2 * h] * f, o[n][2 * h + 1] * f);
+    }
+  }
+}
+
+// Decode: up to 16 query heads of one key/value head are the rows; the keys of a tile are dealt to the four warps and
+// the tiles to `splits` CTAs, whose partial results the last one to arrive combines.
+constexpr int DEC_MAX_SPLITS = 64;
+constexpr int DEC_MAX_GROUPS = 65536;  // arrival counters at the front of the workspace
+
+template <int DQ, int DV>
+__global__ void __launch_bounds__(128) attn_decode_kernel(const AttnArgs a, int rep, int row_tiles, int bs_shift, int splits, int* counters,
+                                                          float* part) {
+  extern __shared__ unsigned char smem_raw[];
+  __shared__ float s_ml[4][16][2];
+  __shared__ float s_fin[16][2];
+  __shared__ int s_last;
+  constexpr int STAGES = CfgTile<DQ, DV>::DEC_STAGES;
+  const uint32_t base = (b2::smem_u32(smem_raw) + 127) & ~127u;
+  const uint32_t sq = base, skv = base + 16 * DQ * 2;
+  float* o_buf = reinterpret_cast<float*>(smem_raw + (skv - b2::smem_u32(smem_raw)));  // [4][16][DV], after the last tile
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  b2::pdl_launch_dependents();
+  b2::pdl_wait();
+  const int b = blockIdx.z, g = blockIdx.y / row_tiles, h0 = (blockIdx.y % row_tiles) * 16, split = blockIdx.x;
+  const int nrows = min(16, rep - h0);
+  const int klen = a.kv_len[b];
+  uint16_t* out = static_cast<uint16_t*>(a.out) + b * a.ldo + static_cast<int64_t>(g * rep + h0) * a.v_pad;
+  if (klen <= 0) {  // padded row of a decode graph
+    if (split == 0)
+      for (int i = threadIdx.x; i < nrows * a.v_pad; i += 128) out[i] = 0;
+    return;
+  }
+  const int p = klen - 1;
+  const int32_t* bt = a.block_tables + b * a.bt_stride;
+  const KeyTiles tiles(p, p, a.window, a.keep_first);
+  const int per = (tiles.total + splits - 1) / splits;
+  const int t0 = split * per, t1 = min(tiles.total, t0 + per);
+  const float inv_cap = a.softcap > 0.f ? 1.0f / a.softcap : 0.f;
+  const uint16_t* q = static_cast<const uint16_t*>(a.q) + b * a.ldq + static_cast<int64_t>(g * rep + h0) * a.qk_pad;
+  for (int idx = threadIdx.x; idx < 16 * (DQ / 8); idx += 128) {
+    const int r = idx / (DQ / 8), pc = idx % (DQ / 8);
+    const bool ok = r < nrows && pc * 8 < a.qk_pad;
+    b2::cp_async16(b2::tile_addr<DQ>(sq, r, pc), q + (ok ? r * a.qk_pad + pc * 8 : 0), ok);
+  }
+#pragma unroll
+  for (int i = 0; i < STAGES - 1; ++i) {
+    if (t0 + i < t1) {
+      const uint32_t sk = skv + i * CfgTile<DQ, DV>::STAGE;
+      load_kv_tile<DQ, DV>(a, bt, bs_shift, g, tiles.at(t0 + i), p, sk, sk + BN * DQ * 2);
+    }
+    b2::cp_async_commit();
+  }
+  const int pos[2] = {p, p};
+  float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
+  float o[DV / 8][4];
+#pragma unroll
+  for (int n = 0; n < DV / 8; ++n)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) o[n][e] = 0.f;
+  for (int t = t0; t < t1; ++t) {
+    const uint32_t sk = skv + ((t - t0) % STAGES) * CfgTile<DQ, DV>::STAGE, sv = sk + BN * DQ * 2;
+    b2::cp_async_wait<STAGES - 2>();
+    __syncthreads();
+    if (t + STAGES - 1 < t1) {
+      const uint32_t nk = skv + ((t - t0 + STAGES - 1) % STAGES) * CfgTile<DQ, DV>::STAGE;
+      load_kv_tile<DQ, DV>(a, bt, bs_shift, g, tiles.at(t + STAGES - 1), p, nk, nk + BN * DQ * 2);
+    }
+    b2::cp_async_commit();
+    const int j0 = tiles.at(t) * BN + warp * 16;  // this warp's 16 keys
+    float s[2][4] = {};
+#pragma unroll
+    for (int k = 0; k < DQ / 16; ++k) {
+      uint32_t qa[4], kb[4];
+      b2::frag_a<DQ>(sq, 0, k * 16, lane, qa);
+      b2::frag_b<DQ>(sk, warp * 16, k * 16, lane, kb);
+      b2::mma16816(s[0], qa, kb[0], kb[1]);
+      b2::mma16816(s[1], qa, kb[2], kb[3]);
+    }
+    float corr[2];
+    softmax_tile<2>(a, s, j0, pos, true, inv_cap, m, l, corr, lane);
+#pragma unroll
+    for (int n = 0; n < DV / 8; ++n) {
+      o[n][0] *= corr[0]; o[n][1] *= corr[0]; o[n][2] *= corr[1]; o[n][3] *= corr[1];
+    }
+    uint32_t hi[4], lo[4];
+    b2::split_bf16(s[0][0], s[0][1], hi[0], lo[0]);
+    b2::split_bf16(s[0][2], s[0][3], hi[1], lo[1]);
+    b2::split_bf16(s[1][0], s[1][1], hi[2], lo[2]);
+    b2::split_bf16(s[1][2], s[1][3], hi[3], lo[3]);
+#pragma unroll
+    for (int n = 0; n < DV / 16; ++n) {
+      uint32_t vb[4];
+      b2::frag_b_t<DV>(sv, n * 16, warp * 16, lane, vb);
+      b2::mma16816(o[2 * n], hi, vb[0], vb[1]);
+      b2::mma16816(o[2 * n + 1], hi, vb[2], vb[3]);
+      b2::mma16816(o[2 * n], lo, vb[0], vb[1]);
+      b2::mma16816(o[2 * n + 1], lo, vb[2], vb[3]);
+    }
+  }
+  b2::cp_async_wait<0>();
+  __syncthreads();  // the stages become the combine buffer
+#pragma unroll
+  for (int h = 0; h < 2; ++h) {
+    l[h] += __shfl_xor_sync(0xffffffffu, l[h], 1);
+    l[h] += __shfl_xor_sync(0xffffffffu, l[h], 2);
+    const int r = (lane >> 2) + h * 8;
+    if ((lane & 3) == 0) {
+      s_ml[warp][r][0] = m[h];
+      s_ml[warp][r][1] = l[h];
+    }
+#pragma unroll
+    for (int n = 0; n < DV / 8; ++n)
+      *reinterpret_cast<float2*>(o_buf + (warp * 16 + r) * DV + n * 8 + (lane & 3) * 2) = make_float2(o[n][2 * h], o[n][2 * h + 1]);
+  }
+  __syncthreads();
+  const int group = (b * a.nkv + g) * row_tiles + blockIdx.y % row_tiles;
+  float* my = part + (static_cast<int64_t>(group) * splits + split) * 16 * (DV + 2);
+  for (int idx = threadIdx.x; idx < nrows * DV; idx += 128) {
+    const int r = idx / DV, c = idx % DV;
+    float mt = -INFINITY;
+#pragma unroll
+    for (int w = 0; w < 4; ++w) mt = fmaxf(mt, s_ml[w][r][0]);
+    float lt = 0.f, ot = 0.f;
+#pragma unroll
+    for (int w = 0; w < 4; ++w) {
+      const float f = s_ml[w][r][0] == -INFINITY ? 0.f : fast_exp2((s_ml[w][r][0] - mt) * LOG2E);
+      lt += f * s_ml[w][r][1];
+      ot += f * o_buf[(w * 16 + r) * DV + c];
+    }
+    if (splits == 1) {
+      if (a.sink != nullptr) {
+        const float sk = a.sink[g * rep + h0 + r], m_new = fmaxf(mt, sk);
+        const float f = fast_exp2((mt - m_new) * LOG2E);
+        lt = lt * f + fast_exp2((sk - m_new) * LOG2E);
+        ot *= f;
+      }
+      if (c < a.v_pad) out[r * a.v_pad + c] = b2::from_float<uint16_t>(ot / lt);
+    } else {
+      my[32 + r * DV + c] = ot;
+      if (c == 0) {
+        my[r] = mt;
+        my[16 + r] = lt;
+      }
+    }
+  }
+  if (splits == 1) return;
+  __threadfence();
+  __syncthreads();
+  if (threadIdx.x == 0) s_last = atomicAdd(counters + group, 1) == splits - 1;
+  __syncthreads();
+  if (!s_last) return;
+  if (threadIdx.x == 0) counters[group] = 0;
+  __threadfence();
+  const float* all = part + static_cast<int64_t>(group) * splits * 16 * (DV + 2);
+  if (threadIdx.x < nrows) {  // the rows' maximum over the splits, and the denominator
+    const int r = threadIdx.x;
+    float mt = a.sink != nullptr ? a.sink[g * rep + h0 + r] : -INFINITY;
+    for (int s = 0; s < splits; ++s) mt = fmaxf(mt, b2::ld_cg_f32(all + static_cast<int64_t>(s) * 16 * (DV + 2) + r));
+    float lt = a.sink != nullptr ? fast_exp2((a.sink[g * rep + h0 + r] - mt) * LOG2E) : 0.f;
+    for (int s = 0; s < splits; ++s) {
+      const float* ps = all + static_cast<int64_t>(s) * 16 * (DV + 2);
+      const float ms = b2::ld_cg_f32(ps + r);
+      if (ms > -INFINITY) lt += fast_exp2((ms - mt) * LOG2E) * b2::ld_cg_f32(ps + 16 + r);
+    }
+    s_fin[r][0] = mt;
+    s_fin[r][1] = 1.0f / lt;
+  }
+  __syncthreads();
+  for (int idx = threadIdx.x; idx < nrows * DV; idx += 128) {
+    const int r = idx / DV, c = idx % DV;
+    float ot = 0.f;
+    for (int s = 0; s < splits; ++s) {
+      const float* ps = all + static_cast<int64_t>(s) * 16 * (DV + 2);
+      const float ms = b2::ld_cg_f32(ps + r);
+      if (ms > -INFINITY) ot += fast_exp2((ms - s_fin[r][0]) * LOG2E) * b2::ld_cg_f32(ps + 32 + r * DV + c);
+    }
+    if (c < a.v_pad) out[r * a.v_pad + c] = b2::from_float<uint16_t>(ot * s_fin[r][1]);
+  }
+}
+
+int log2_exact(int n) {
+  for (int s = 0; s < 31; ++s)
+    if ((1 << s) == n) return s;
+  return -1;
+}
+
+bool tiled_form(int dtype, int qk_pad, int v_pad) { return dtype == B2_DT_BF16 && qk_pad <= 128 && v_pad <= 128; }
+
+// CTAs a decode step's keys are dealt to, per (sequence, key/value head, 16 query heads)
+int decode_splits(int B, int max_kv, int nq, int nkv, int window, int keep_first) {
+  const int64_t groups = static_cast<int64_t>(B) * nkv * ((nq / nkv + 15) / 16);
+  const int64_t all = (static_cast<int64_t>(max_kv) + BN - 1) / BN;
+  const int64_t seen = (static_cast<int64_t>(keep_first) + BN - 1) / BN + (static_cast<int64_t>(window) + BN - 2) / BN + 1;
+  const int64_t tiles = std::max<int64_t>(1, std::min(all, seen));
+  // two CTAs per SM fit; a CTA should have at least two tiles
+  const int64_t want = (2 * 148 + groups - 1) / groups;
+  return static_cast<int>(std::max<int64_t>(1, std::min({want, tiles / 2, static_cast<int64_t>(DEC_MAX_SPLITS)})));
+}
+
+template <int DQ, int DV>
+int launch_tiled(const AttnArgs& a, int max_q, int max_kv, void* ws, int64_t ws_bytes, cudaStream_t s) {
+  using C = CfgTile<DQ, DV>;
+  const int rep = a.nq / a.nkv, shift = log2_exact(a.block_size);
+  if (a.cu_q != nullptr) {
+    static bool set = false;
+    if (!set) {
+      B2_CUDA(cudaFuncSetAttribute(attn_prefill_kernel<DQ, DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, C::SMEM_PREFILL));
+      set = true;
+    }
+    const int64_t tiles = (static_cast<int64_t>(max_q) * rep + 63) / 64;
+    B2_CUDA(b2_launch(attn_prefill_kernel<DQ, DV>, dim3(static_cast<unsigned>(tiles), a.nkv, a.B), dim3(128), C::SMEM_PREFILL, s, a, rep, shift));
+    return B2_OK;
+  }
+  static bool set = false;
+  if (!set) {
+    B2_CUDA(cudaFuncSetAttribute(attn_decode_kernel<DQ, DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, C::SMEM_DECODE));
+    set = true;
+  }
+  const int row_tiles = (rep + 15) / 16;
+  const int64_t groups = static_cast<int64_t>(a.B) * a.nkv * row_tiles;
+  int splits = decode_splits(a.B, max_kv, a.nq, a.nkv, a.window, a.keep_first);
+  const int64_t need = DEC_MAX_GROUPS * 4ll + groups * splits * 16 * (DV + 2) * 4;
+  if (groups > DEC_MAX_GROUPS) splits = 1;
+  if (splits > 1 && (ws == nullptr || ws_bytes < need)) return b2::set_error(B2_ERR_SHAPE, "b2_attention: workspace of %lld bytes, %lld needed",
+                                                                             static_cast<long long>(ws_bytes), static_cast<long long>(need));
+  B2_CUDA(b2_launch(attn_decode_kernel<DQ, DV>, dim3(splits, a.nkv * row_tiles, a.B), dim3(128), C::SMEM_DECODE, s, a, rep, row_tiles, shift, splits,
+                    static_cast<int*>(ws), reinterpret_cast<float*>(static_cast<unsigned char*>(ws) + DEC_MAX_GROUPS * 4ll)));
+  return B2_OK;
+}
+
 bool aligned16(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; }
 
 template <typename T>
@@ -243,7 +698,10 @@ int b2_qk_norm_store(int dtype, void* qkv, int64_t ld_qkv, int M, int nq, int nk
 }
 
 int64_t b2_attention_workspace(int dtype, int B, int max_q, int max_kv, int nq, int nkv, int qk_pad, int v_pad, int window, int keep_first) {
-  return 0;
+  if (max_q > 1 || B <= 0 || nkv <= 0 || nq < nkv || !tiled_form(dtype, qk_pad, v_pad)) return 0;
+  const int64_t groups = static_cast<int64_t>(B) * nkv * ((nq / nkv + 15) / 16);
+  const int splits = decode_splits(B, max_kv, nq, nkv, window, keep_first);
+  return splits > 1 ? DEC_MAX_GROUPS * 4ll + groups * splits * 16 * ((v_pad <= 64 ? 64 : 128) + 2) * 4 : 0;
 }
 
 int b2_attention(int dtype, const void* q, int64_t ldq, void* out, int64_t ldo, const void* k_cache, const void* v_cache,
@@ -264,7 +722,11 @@ int b2_attention(int dtype, const void* q, int64_t ldq, void* out, int64_t ldo, 
   a.scale = scale; a.softcap = softcap; a.sink = sink;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   if (dtype == B2_DT_F32) return launch_any<float>(a, max_q, s);
-  return launch_any<uint16_t>(a, max_q, s);
+  if (form == 1 || !tiled_form(dtype, qk_pad, v_pad)) return launch_any<uint16_t>(a, max_q, s);
+  if (qk_pad <= 64) return v_pad <= 64 ? launch_tiled<64, 64>(a, max_q, max_kv, workspace, workspace_bytes, s)
+                                       : launch_tiled<64, 128>(a, max_q, max_kv, workspace, workspace_bytes, s);
+  return v_pad <= 64 ? launch_tiled<128, 64>(a, max_q, max_kv, workspace, workspace_bytes, s)
+                     : launch_tiled<128, 128>(a, max_q, max_kv, workspace, workspace_bytes, s);
 }
 
 }  // extern "C"
