@@ -1,4 +1,4 @@
-"""The two other BASELINE workloads, behind `bench.py --workload cfg2|cfg5` (same JSON line as the default workload).
+"""The other workloads, behind `bench.py --workload cfg2|cfg5|vekerax` (the JSON line of the default workload).
 
 cfg2  the reference's own bench.py workload (bench.py:9-27): Qwen3-0.6B random-init bf16 on one GPU, 256 sequences,
       prompt ids uniform in [0, 10000], prompt and output lengths uniform in [100, 1024], temperature 0.6, ignore_eos;
@@ -8,6 +8,8 @@ cfg2  the reference's own bench.py workload (bench.py:9-27): Qwen3-0.6B random-i
 cfg5  long-context prefill of Qwen3-32B random-init bf16 at tensor-parallel size 8: 4 sequences of 32768 uniform-random
       tokens in 16384-token chunks (nanovllm/engine/scheduler.py:42-48: only the first waiting sequence is chunked), KV
       blocks taken from a random permutation of the free list; prefill tokens / second.
+vekerax  prefill and decode throughput of the Vekerax design beside Qwen3 with layers of the same size (random weights),
+      and the time and roofline fraction of each of its kernels beside the like kernel of Qwen3.
 """
 from __future__ import annotations
 
@@ -170,4 +172,258 @@ def run_cfg2(args, peaks, clock_sampler_cls) -> None:
                 "gpu_launches": _abi.launch_count(), "total_output_tokens": total, "seconds": seconds}
         print(json.dumps(line), flush=True)
     runner.exit()
+    dist.destroy_process_group()
+
+
+# ---------------------------------------------------------------------------------------------------------------------
+# vekerax: throughput of the Vekerax design beside Qwen3 with layers of the same size, and every kernel of the design
+# beside the kernel of Qwen3 that does the like work.
+# ---------------------------------------------------------------------------------------------------------------------
+VEKERAX_SIZES = {  # layer sizes of Qwen3-0.6B and Qwen3-8B; fewer layers and a smaller vocabulary, the same for both models
+    "width1024": dict(width=1024, ff=3072, heads=16, kv_heads=8, dim=128, layers=12, vocab=32768),
+    "width4096": dict(width=4096, ff=12288, heads=32, kv_heads=8, dim=128, layers=8, vocab=32768),
+}
+VEKERAX_WINDOW, VEKERAX_KEEP, VEKERAX_STREAMS = 1024, 4, 4
+
+
+def _vekerax_config(z: dict) -> dict:
+    attn = {"type": "attention", "mixer": {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": z["dim"], "vdim": z["dim"], "scale": z["dim"] ** -0.5,
+                                           "softcap": 30.0, "mask": {"size": VEKERAX_WINDOW, "keep_first": VEKERAX_KEEP}},
+            "mlp": {"kind": "dense", "ff": z["ff"]}}
+    light = {"type": "lightning", "mixer": {"heads": z["heads"], "dim": z["dim"], "vdim": z["dim"],
+                                            "decay": [1.0 - 2.0 ** (-2 - 6 * h / z["heads"]) for h in range(z["heads"])]},
+             "mlp": {"kind": "dense", "ff": z["ff"]}}
+    return {"architecture": "Vekerax", "embedding": {"scale": 1.0}, "layers": [attn, light] * (z["layers"] // 2), "norm": {"eps": 1e-6},
+            "residual_mult": 1.0, "streams": VEKERAX_STREAMS, "vocab": z["vocab"], "width": z["width"]}
+
+
+def _qwen_config(z: dict) -> dict:
+    return {"architectures": ["Qwen3ForCausalLM"], "hidden_size": z["width"], "num_attention_heads": z["heads"], "num_key_value_heads": z["kv_heads"],
+            "head_dim": z["dim"], "intermediate_size": z["ff"], "num_hidden_layers": z["layers"], "vocab_size": z["vocab"], "attention_bias": False}
+
+
+def _model_throughput(torch, cfg: dict, vocab: int, batch: int, prompt: int, steps: int, warmup: int) -> dict:
+    """Prefill tokens/s through step() (4 prompts a step) and decode tokens/s (device-resident and through step())."""
+    from nanovllm_b200.engine.llm_engine import ensure_process_group
+    from nanovllm_b200.engine.model_runner import ModelRunner, ResidentDecoder, Seq, sequential_block_tables
+    from nanovllm_b200.models.registry import config_from_dict
+    ensure_process_group()
+    max_len = -(-(prompt + steps + warmup + 8) // 256) * 256
+    runner = ModelRunner(config_from_dict(cfg), max_num_seqs=batch, max_model_len=max_len, max_num_batched_tokens=16384,
+                         num_kvcache_blocks=batch * max_len // 256)
+    g = torch.Generator().manual_seed(0)
+    prompts = torch.randint(0, vocab, (batch, prompt), generator=g).tolist()
+    tables = sequential_block_tables([max_len] * batch, 256)
+    seqs = [Seq(p, t, 0, i) for i, (p, t) in enumerate(zip(prompts, tables))]
+    per = max(1, min(batch, 8192 // prompt))
+
+    def prefill():
+        out = []
+        for a in range(0, batch, per):
+            out += runner.step(seqs[a:a + per], True)
+        return out
+
+    def timed(fn, n):
+        torch.cuda.synchronize()
+        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        e0.record()
+        for _ in range(n):
+            fn()
+        e1.record()
+        torch.cuda.synchronize()
+        return e0.elapsed_time(e1) / n
+
+    for _ in range(2):
+        first = prefill()
+    pre_ms = timed(prefill, 3)
+    for s, t in zip(seqs, first):
+        s.token_ids = s.token_ids[:prompt] + [t]
+    out = {"prefill_tok_s": batch * prompt / pre_ms * 1e3, "prefill_tokens_per_step": per * prompt}
+    rd = ResidentDecoder(runner, batch)
+    rd.load(seqs)
+    for _ in range(warmup):
+        rd.replay()
+    ms = timed(rd.replay, steps)
+    out.update(decode_tok_s=batch / ms * 1e3, decode_ms_per_step=ms, launches_per_decode_step=rd.kernels_per_step)
+
+    def step():
+        for s, t in zip(seqs, runner.step(seqs, False)):
+            s.token_ids.append(t)
+    for s in seqs:
+        s.token_ids = s.token_ids[:prompt + 1]
+    for _ in range(3):
+        step()
+    out["decode_tok_s_through_step"] = batch / timed(step, min(steps, max_len - prompt - 8)) * 1e3
+    runner.runtime.check_status()
+    runner.exit()
+    del rd, runner
+    import gc
+    gc.collect()
+    torch.cuda.empty_cache()
+    return out
+
+
+def _kernel_table(torch, z: dict, peaks: dict, batch: int, ctx_len: int) -> list[dict]:
+    """Microseconds and fraction of the roofline (measured copy bandwidth or burst bf16 throughput) of every kernel of the
+    design at this layer size, each next to the like kernel of Qwen3 on the same sizes.  Inputs rotate through more than L2."""
+    from flash_attn import flash_attn_varlen_func, flash_attn_with_kvcache
+    from nanovllm_b200 import _abi, ops
+    from nanovllm_b200.rowpar_microbench import time_in_graph
+    dev, bf, W, S = "cuda", torch.bfloat16, z["width"], VEKERAX_STREAMS
+    H, G, d, ff, win, keep = z["heads"], z["kv_heads"], z["dim"], z["ff"], VEKERAX_WINDOW, VEKERAX_KEEP
+    rows = []
+
+    def add(name, like, work, us, like_work, like_us, bound):
+        peak = peaks["hbm_gbs"] * 1e9 if bound == "hbm" else peaks["bf16_tflops"] * 1e12
+        f, g = work / (us * 1e-6) / peak, like_work / (like_us * 1e-6) / peak
+        rows.append({"kernel": name, "us": round(us, 2), "bound": bound, "frac": round(f, 3), "like": like, "like_us": round(like_us, 2),
+                     "like_frac": round(g, 3), "like_over_this": round(g / f, 2)})
+
+    def variants(make, nbytes):
+        return [make() for _ in range(max(2, min(48, int(4e8 / nbytes) + 1)))]
+
+    for M in (batch, 8192):
+        # residual: streams against add + RMSNorm
+        nb = M * W * (8 * S + 4)
+        vs = variants(lambda: (torch.randn(M, S, W, device=dev), torch.randn(M, W, device=dev).to(bf)), nb)
+        mix, so, si, nw = torch.eye(S, device=dev), torch.ones(S, device=dev), torch.ones(S, device=dev) / S, torch.ones(W, device=dev)
+        us = time_in_graph(lambda i: ops.stream_step(vs[i][0], vs[i][1], mix, so, 0.1, si, nw, 1e-6, W), len(vs), 4 * len(vs))
+        nl = M * W * 8
+        ls = variants(lambda: (torch.randn(M, W, device=dev).to(bf), torch.randn(M, W, device=dev).to(bf)), nl)
+        nwb = nw.to(bf)
+        lus = time_in_graph(lambda i: ops.add_rmsnorm(ls[i][0], ls[i][1], nwb, 1e-6), len(ls), 4 * len(ls))
+        add(f"stream_step M={M}", "add_rmsnorm", nb, us, nl, lus, "hbm")
+        del vs, ls
+        # gated norm against RMSNorm of the same row length
+        n = H * d
+        nb = M * n * 8
+        vs = variants(lambda: (torch.randn(M, n, device=dev), torch.randn(M, n, device=dev).to(bf)), nb)
+        w = torch.ones(n, device=dev)
+        us = time_in_graph(lambda i: ops.gated_norm(vs[i][0], vs[i][1], w, 1e-6, n), len(vs), 4 * len(vs))
+        ls = variants(lambda: torch.randn(M, n, device=dev).to(bf), M * n * 4)
+        wb = w.to(bf)
+        lus = time_in_graph(lambda i: ops.rmsnorm(ls[i], wb, 1e-6), len(ls), 4 * len(ls))
+        add(f"gated_norm M={M}", "rmsnorm", nb, us, M * n * 4, lus, "hbm")
+        del vs, ls
+        # projections: the same GEMM with other epilogues
+        def gemm_pair(name, like, mine, theirs, N, out_cols, K):
+            ws = [(torch.randn(N, K, device=dev) * 0.02).to(bf) for _ in range(max(2, min(12, int(3e8 / (N * K * 2)) + 1)))]
+            x = torch.randn(M, K, device=dev).to(bf)
+            us = time_in_graph(lambda i: mine(x, ws[i]), len(ws), 4 * len(ws))
+            lus = time_in_graph(lambda i: theirs(x, ws[i]), len(ws), 4 * len(ws))
+            if M > 1000:
+                add(f"{name} M={M}", like, 2.0 * M * N * K, us, 2.0 * M * N * K, lus, "tensor")
+            else:
+                nbytes = 2.0 * (N * K + M * K + M * out_cols)
+                add(f"{name} M={M}", like, nbytes, us, nbytes, lus, "hbm")
+        gemm_pair("gate_up + relu*mul", "gate_up + silu*mul", lambda x, w: ops.gemm_act_mul(x, w, _abi.ACT_RELU), ops.gemm_silu_mul, 2 * ff, ff, W)
+        gemm_pair("lightning q|k|v|g + silu", "gemm", lambda x, w: ops.gemm(x, w, silu_cols=3 * H * d), ops.gemm, 4 * H * d, 4 * H * d, W)
+        # o / down projection and what follows: GEMM, then the stream launch, against the fused row-parallel block
+        for nm, K in (("o_proj", H * d), ("down_proj", ff)):
+            ws = [(torch.randn(W, K, device=dev) * 0.02).to(bf) for _ in range(max(2, min(24, int(3e8 / (W * K * 2)) + 1)))]
+            x, xs, r = torch.randn(M, K, device=dev).to(bf), torch.randn(M, S, W, device=dev), torch.randn(M, W, device=dev).to(bf)
+            us = time_in_graph(lambda i: ops.stream_step(xs, ops.gemm(x, ws[i]), mix, so, 0.1, si, nw, 1e-6, W), len(ws), 4 * len(ws))
+            lus = time_in_graph(lambda i: ops.rowpar_fused(x, ws[i], None, r, nwb, 1e-6), len(ws), 4 * len(ws))
+            if M > 1000:
+                # time at the two rooflines: the product, then the bytes of the streams (the like block: residual and outputs)
+                roof = 2.0 * M * W * K / (peaks["bf16_tflops"] * 1e12) + M * W * (8.0 * S + 4) / (peaks["hbm_gbs"] * 1e9)
+                lroof = 2.0 * M * W * K / (peaks["bf16_tflops"] * 1e12) + M * W * 8.0 / (peaks["hbm_gbs"] * 1e9)
+            else:
+                roof = (2.0 * (W * K + M * K) + M * W * (8.0 * S + 4)) / (peaks["hbm_gbs"] * 1e9)
+                lroof = (2.0 * (W * K + M * K) + M * W * 8.0) / (peaks["hbm_gbs"] * 1e9)
+            rows.append({"kernel": f"{nm} + stream_step M={M}", "us": round(us, 2), "bound": "sum", "frac": round(roof * 1e6 / us, 3),
+                         "like": "rowpar_fused", "like_us": round(lus, 2), "like_frac": round(lroof * 1e6 / lus, 3),
+                         "like_over_this": round((lroof / lus) / (roof / us), 2)})
+            del ws, x, xs, r
+        # head norm and scatter after the projection (decode: inside the projection launch for both models)
+        N = (H + 2 * G) * d
+        kc = torch.zeros(64, 256, G, d, dtype=bf, device=dev)
+        vc = torch.zeros_like(kc)
+        slots = torch.randperm(64 * 256, device=dev)[:M].int()
+        pos = torch.arange(M, device=dev) % 2048
+        cs = torch.randn(2048, d, device=dev)
+        qw = torch.ones(d, device=dev).to(bf)
+        nb = M * d * (2 * H + 2 * H + 2 * G + 2 * G + 2 * G + 2 * G + 2 * G)  # q in and out, k in and out, v in, both to the cache
+        vs = variants(lambda: torch.randn(M, N, device=dev).to(bf), nb)
+        us = time_in_graph(lambda i: ops.qk_norm_store(vs[i], H, G, d, d, d, d, qw, qw, 1e-6, kc, vc, slots), len(vs), 4 * len(vs))
+        lus = time_in_graph(lambda i: ops.qk_norm_rope_store(vs[i], H, G, d, qw, qw, 1e-6, pos, cs, kc, vc, slots), len(vs), 4 * len(vs))
+        add(f"qk_norm_store M={M}", "qk_norm_rope_store", nb, us, nb, lus, "hbm")
+        del vs, kc, vc
+    # attention, prefill: sequences of 2048 in a batch of 8192, the same window for both
+    B, L = 4, 2048
+    M = B * L
+    kc = torch.randn(B * L // 256, 256, G, d, device=dev).to(bf)
+    vc = torch.randn_like(kc)
+    bt = torch.randperm(B * L // 256, device=dev).int().view(B, -1).contiguous()
+    cu = torch.arange(0, M + 1, L, device=dev, dtype=torch.int32)
+    kl = torch.full((B,), L, dtype=torch.int32, device=dev)
+    q = torch.randn(M, H * d, device=dev).to(bf)
+    sink = torch.zeros(H, device=dev)
+    seen = sum(min(i + 1, win) for i in range(L)) * B
+    flops = 4.0 * H * d * seen
+    k, v = torch.randn(M, G, d, device=dev).to(bf), torch.randn(M, G, d, device=dev).to(bf)
+    us = time_in_graph(lambda i: ops.window_attention(q, H, kc, vc, bt, cu, kl, L, L, d ** -0.5, 30.0, win, keep, sink), 4, 24)
+    lus = time_in_graph(lambda i: flash_attn_varlen_func(q.view(M, H, d), k, v, cu, cu, L, L, softmax_scale=d ** -0.5, causal=True, window_size=(win - 1, 0)), 4, 24)
+    add(f"window_attention prefill {B}x{L} window {win}", "flash-attn, same window, passed K/V", flops, us, flops, lus, "tensor")
+    # linear attention, prefill
+    D = torch.tensor([1.0 - 2.0 ** (-2 - 6 * h / H) for h in range(H)], dtype=torch.float64)
+    dec, pw = D.float().to(dev), (D.unsqueeze(1) ** torch.arange(65)).float().to(dev)
+    p = torch.randn(M, 4 * H * d, device=dev).to(bf)
+    state = torch.zeros(max(batch, B), H, d, d, device=dev)
+    sl = torch.arange(B, device=dev, dtype=torch.int32)
+    lin_flops = 2.0 * M * H * (2 * d * d + 64 * d)  # state in and out, and the causal half of two 64-wide products
+    us2 = time_in_graph(lambda i: ops.linear_attn(p, H, d, d, state, sl, cu, kl, L, dec, pw), 4, 24)
+    full = 4.0 * H * d * B * L * (L + 1) / 2
+    lus2 = time_in_graph(lambda i: flash_attn_varlen_func(q.view(M, H, d), k, v, cu, cu, L, L, softmax_scale=d ** -0.5, causal=True), 4, 24)
+    add(f"linear_attn prefill {B}x{L}", "flash-attn, full causal", lin_flops, us2, full, lus2, "tensor")
+    lin_bytes = M * H * d * (3 * 2 + 4.0)
+    rows[-1]["frac_of_hbm"] = round(lin_bytes / (us2 * 1e-6) / (peaks["hbm_gbs"] * 1e9), 3)
+    # decode
+    nblk = -(-ctx_len // 256)
+    n_layers = 6
+    kcs = [torch.randn(batch * nblk, 256, G, d, device=dev).to(bf) for _ in range(n_layers)]
+    vcs = [torch.randn(batch * nblk, 256, G, d, device=dev).to(bf) for _ in range(n_layers)]
+    bt = torch.randperm(batch * nblk, device=dev).int().view(batch, nblk).contiguous()
+    kl = torch.full((batch,), ctx_len, dtype=torch.int32, device=dev)
+    q = torch.randn(batch, H * d, device=dev).to(bf)
+    nb = 2.0 * batch * min(ctx_len, win) * G * d * 2
+    us = time_in_graph(lambda i: ops.window_attention(q, H, kcs[i], vcs[i], bt, None, kl, 1, nblk * 256, d ** -0.5, 30.0, win, keep, sink), n_layers, 10 * n_layers)
+    lus = time_in_graph(lambda i: flash_attn_with_kvcache(q.view(batch, 1, H, d), kcs[i], vcs[i], cache_seqlens=kl, block_table=bt, softmax_scale=d ** -0.5, causal=True),
+                        n_layers, 10 * n_layers)
+    add(f"window_attention decode {batch} x {ctx_len}", "flash-attn kvcache", nb, us, nb, lus, "hbm")
+    sts = [torch.zeros(batch, H, d, d, device=dev) for _ in range(4)]
+    sl = torch.arange(batch, device=dev, dtype=torch.int32)
+    p = torch.randn(batch, 4 * H * d, device=dev).to(bf)
+    us = time_in_graph(lambda i: ops.linear_attn(p, H, d, d, sts[i], sl, None, kl, 1, dec, pw), 4, 40)
+    add(f"linear_attn decode {batch}", "flash-attn kvcache", 8.0 * batch * H * d * d, us, nb, lus, "hbm")
+    return rows
+
+
+def run_vekerax(args, peaks, clock_sampler_cls) -> None:
+    torch, dist, rank, world, local = _setup(args)
+    assert world == 1, "Vekerax runs on one GPU"
+    from nanovllm_b200 import runtime as rt
+    K, W = min(args.steps, 128), max(3, args.warmup)
+    sizes = {}
+    with clock_sampler_cls(local) as clocks:
+        for name, z in VEKERAX_SIZES.items():
+            res = {}
+            for batch, prompt in ((64, 1024), (4, 4096)):
+                key = f"batch {batch}, prompts of {prompt}"
+                res[key] = {"vekerax": _model_throughput(torch, _vekerax_config(z), z["vocab"], batch, prompt, K, W),
+                            "qwen3": _model_throughput(torch, _qwen_config(z), z["vocab"], batch, prompt, K, W)}
+            rt.init_runtime(max_tokens=8192, hidden=z["width"], oneshot_tokens=1024)
+            with torch.inference_mode():
+                kernels = _kernel_table(torch, z, peaks, 64, 1024)
+            rt.shutdown_runtime()
+            torch.cuda.empty_cache()
+            sizes[name] = {"layer_sizes": z, "throughput": res, "kernels": kernels}
+    from nanovllm_b200 import _abi
+    head = sizes["width4096"]["throughput"]["batch 64, prompts of 1024"]["vekerax"]
+    print(json.dumps({"metric": "vekerax_decode_tokens_per_s", "value": head["decode_tok_s"], "unit": "tok/s", "n_gpus": 1, "steps": K, "warmup": W,
+                      "ms_per_step": head["decode_ms_per_step"], "higher_is_better": True, "scaling": "strong", "vs_baseline": None, "dtype": "bf16", "data": "synthetic",
+                      "config": {"workload": f"Vekerax and Qwen3 with the same layer sizes, random weights; {VEKERAX_STREAMS} streams, window {VEKERAX_WINDOW} + {VEKERAX_KEEP}, "
+                                             "attention and lightning layers in turn; value: width 4096, batch 64, 1024-token prompts, device-resident decode",
+                                 "l2": "weights, caches and rotated kernel inputs exceed the 126 MB L2"},
+                      "clocks": clocks.summary(), "gpu_launches": _abi.launch_count(), "sizes": sizes}), flush=True)
     dist.destroy_process_group()

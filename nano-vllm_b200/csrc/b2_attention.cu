@@ -216,65 +216,100 @@ __device__ __forceinline__ float fast_exp2(float x) {
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
 }
-// cap * tanh(s / cap), tanh(x) = 1 - 2 / (1 + e^2x); its Taylor series where that would cancel
-__device__ __forceinline__ float soft_cap(float s, float cap, float inv_cap) {
-  const float x = s * inv_cap;
-  const float e = fast_exp2(x * 2.885390081777927f);  // 2 log2(e)
-  const float t = 1.0f - __fdividef(2.0f, e + 1.0f);
-  const float x2 = x * x;
-  const float series = x * (1.0f + x2 * (-0.33333333333f + x2 * 0.13333333333f));
-  return cap * (fabsf(x) < 0.125f ? series : (e > 1e30f ? 1.0f : t));
+// Scores in units of log2: t = log2(e) * softcap(scale * s).  The three forms of the cap:
+enum { CAP_NONE = 0, CAP_SHORT = 1, CAP_FULL = 2 };
+struct ScoreScale {
+  float a, b, c;  // NONE: t = a s.  SHORT: t = c - b / (1 + 2^(a s)).  FULL: see score()
+};
+__host__ __device__ inline ScoreScale score_scale(int cap_form, float scale, float cap) {
+  constexpr float L = 1.4426950408889634f;
+  if (cap_form == CAP_NONE) return {scale * L, 0.f, 0.f};
+  return {2.0f * L * scale / cap, 2.0f * cap * L, cap * L};
+}
+// tanh(x) = 1 - 2 / (1 + e^2x) has an absolute error of about 1e-7, so the capped score is off by 1e-7 cap: below fp32
+// rounding of the scores themselves for caps up to a few hundred (SHORT).  FULL adds the Taylor series where the
+// difference would cancel, for any cap.
+template <int CAP>
+__device__ __forceinline__ float score(float s, const ScoreScale& k) {
+  if (CAP == CAP_NONE) return s * k.a;
+  const float z = s * k.a;  // 2 log2(e) x
+  const float t = fmaf(-k.b, __fdividef(1.0f, 1.0f + fast_exp2(fminf(z, 120.0f))), k.c);
+  if (CAP == CAP_SHORT) return t;
+  const float x = z * 0.34657359027997264f, x2 = x * x;
+  const float series = k.c * x * fmaf(x2, fmaf(x2, 0.13333333333f, -0.33333333333f), 1.0f);
+  return fabsf(x) < 0.125f ? series : t;
 }
 
 constexpr float LOG2E = 1.4426950408889634f;
 
+// The slot of key j of a sequence
+__device__ __forceinline__ int64_t slot_of(const AttnArgs& a, const int32_t* bt, int j) {
+  const int blk = j / a.block_size;
+  return static_cast<int64_t>(__ldg(bt + blk)) * a.block_size + (j - blk * a.block_size);
+}
+// One tile of one operand, D columns of which `pad` exist: 128 threads, 16 bytes per copy.  base = first row's address
+// when the tile lies in one block (`whole`), else every row is looked up.
+template <int D>
+__device__ __forceinline__ void load_rows(const AttnArgs& a, const uint16_t* cache, const int32_t* bt, bool whole, int64_t slot0, int g, int pad,
+                                          int tile, int last, uint32_t dst) {
+  constexpr int P = D / 8, STEP = 128 / P;
+  const int r0 = threadIdx.x / P, p = threadIdx.x % P;
+  const bool piece = p * 8 < pad;
+  const int64_t stride = static_cast<int64_t>(a.nkv) * pad;
+  const uint16_t* col = cache + static_cast<int64_t>(g) * pad + (piece ? p * 8 : 0);
+  if (whole) {
+    const uint16_t* src = col + (slot0 + r0) * stride;
+#pragma unroll
+    for (int i = 0; i < BN / STEP; ++i, src += STEP * stride) {
+      const int r = r0 + i * STEP;
+      const bool ok = piece && tile * BN + r <= last;
+      b2::cp_async16(b2::tile_addr<D>(dst, r, p), ok ? src : cache, ok);
+    }
+  } else {
+#pragma unroll
+    for (int i = 0; i < BN / STEP; ++i) {
+      const int r = r0 + i * STEP, j = tile * BN + r;
+      const bool ok = piece && j <= last;
+      b2::cp_async16(b2::tile_addr<D>(dst, r, p), ok ? col + slot_of(a, bt, j) * stride : cache, ok);
+    }
+  }
+}
 template <int DQ, int DV>
-__device__ __forceinline__ void load_kv_tile(const AttnArgs& a, const int32_t* bt, int bs_shift, int g, int tile, int last, uint32_t sk, uint32_t sv) {
-  constexpr int QP = DQ / 8, VP = DV / 8;
-  const uint16_t* kc = static_cast<const uint16_t*>(a.k_cache);
-  const uint16_t* vc = static_cast<const uint16_t*>(a.v_cache);
-#pragma unroll
-  for (int i = 0; i < BN * QP / 128; ++i) {
-    const int idx = threadIdx.x + i * 128, r = idx / QP, p = idx % QP, j = tile * BN + r;
-    const bool ok = j <= last && p * 8 < a.qk_pad;
-    int64_t slot = 0;
-    if (ok) slot = bs_shift >= 0 ? (static_cast<int64_t>(__ldg(bt + (j >> bs_shift))) << bs_shift) + (j & ((1 << bs_shift) - 1))
-                                 : static_cast<int64_t>(__ldg(bt + j / a.block_size)) * a.block_size + j % a.block_size;
-    b2::cp_async16(b2::tile_addr<DQ>(sk, r, p), kc + (slot * a.nkv + g) * a.qk_pad + (ok ? p * 8 : 0), ok);
-  }
-#pragma unroll
-  for (int i = 0; i < BN * VP / 128; ++i) {
-    const int idx = threadIdx.x + i * 128, r = idx / VP, p = idx % VP, j = tile * BN + r;
-    const bool ok = j <= last && p * 8 < a.v_pad;
-    int64_t slot = 0;
-    if (ok) slot = bs_shift >= 0 ? (static_cast<int64_t>(__ldg(bt + (j >> bs_shift))) << bs_shift) + (j & ((1 << bs_shift) - 1))
-                                 : static_cast<int64_t>(__ldg(bt + j / a.block_size)) * a.block_size + j % a.block_size;
-    b2::cp_async16(b2::tile_addr<DV>(sv, r, p), vc + (slot * a.nkv + g) * a.v_pad + (ok ? p * 8 : 0), ok);
-  }
+__device__ __forceinline__ void load_kv_tile(const AttnArgs& a, const int32_t* bt, bool whole, int g, int tile, int last, uint32_t sk, uint32_t sv) {
+  const int64_t slot0 = whole ? slot_of(a, bt, tile * BN) : 0;
+  load_rows<DQ>(a, static_cast<const uint16_t*>(a.k_cache), bt, whole, slot0, g, a.qk_pad, tile, last, sk);
+  load_rows<DV>(a, static_cast<const uint16_t*>(a.v_cache), bt, whole, slot0, g, a.v_pad, tile, last, sv);
 }
 
 // One tile's scores of a warp: NT 8-key column tiles starting at key j0.  Scales, caps, masks (when `masked`), folds
 // into the running maximum m and sum l, and leaves the weights in s.  Returns the factors for the old outputs.
-template <int NT>
-__device__ __forceinline__ void softmax_tile(const AttnArgs& a, float (&s)[NT][4], int j0, const int (&pos)[2], bool masked, float inv_cap,
+template <int NT, int CAP>
+__device__ __forceinline__ void softmax_tile(const AttnArgs& a, const ScoreScale& k, float (&s)[NT][4], int j0, const int (&pos)[2], bool masked,
                                              float (&m)[2], float (&l)[2], float (&corr)[2], int lane) {
   float mx[2] = {-INFINITY, -INFINITY};
 #pragma unroll
   for (int n = 0; n < NT; ++n)
 #pragma unroll
-    for (int e = 0; e < 4; ++e) {
-      float v = s[n][e] * a.scale;
-      if (a.softcap > 0.f) v = soft_cap(v, a.softcap, inv_cap);
-      if (masked && !visible(pos[e >> 1], j0 + n * 8 + (lane & 3) * 2 + (e & 1), a.window, a.keep_first)) v = -INFINITY;
-      s[n][e] = v;
-      mx[e >> 1] = fmaxf(mx[e >> 1], v);
-    }
+    for (int e = 0; e < 4; ++e) s[n][e] = score<CAP>(s[n][e], k);
+  if (masked) {
+#pragma unroll
+    for (int n = 0; n < NT; ++n)
+#pragma unroll
+      for (int e = 0; e < 4; ++e)
+        if (!visible(pos[e >> 1], j0 + n * 8 + (lane & 3) * 2 + (e & 1), a.window, a.keep_first)) s[n][e] = -INFINITY;
+  }
+#pragma unroll
+  for (int n = 0; n < NT; ++n)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) mx[e >> 1] = fmaxf(mx[e >> 1], s[n][e]);
+  float base[2];
 #pragma unroll
   for (int h = 0; h < 2; ++h) {
     mx[h] = fmaxf(mx[h], __shfl_xor_sync(0xffffffffu, mx[h], 1));
     mx[h] = fmaxf(mx[h], __shfl_xor_sync(0xffffffffu, mx[h], 2));
     const float m_new = fmaxf(m[h], mx[h]);
-    corr[h] = m_new == -INFINITY ? 1.0f : fast_exp2((m[h] - m_new) * LOG2E);
+    base[h] = m_new == -INFINITY ? 0.f : m_new;  // nothing visible yet: every weight is 2^-inf = 0
+    corr[h] = fast_exp2(m[h] - base[h]);
     m[h] = m_new;
   }
   float sum[2] = {0.f, 0.f};
@@ -282,12 +317,12 @@ __device__ __forceinline__ void softmax_tile(const AttnArgs& a, float (&s)[NT][4
   for (int n = 0; n < NT; ++n)
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
-      const float p = m[e >> 1] == -INFINITY ? 0.f : fast_exp2((s[n][e] - m[e >> 1]) * LOG2E);
+      const float p = fast_exp2(s[n][e] - base[e >> 1]);
       s[n][e] = p;
       sum[e >> 1] += p;
     }
 #pragma unroll
-  for (int h = 0; h < 2; ++h) l[h] = l[h] * corr[h] + sum[h];  // this lane's part; summed over the row's four lanes at the end
+  for (int h = 0; h < 2; ++h) l[h] = fmaf(l[h], corr[h], sum[h]);  // this lane's part; summed over the row's four lanes at the end
 }
 
 template <int DQ, int DV>
@@ -299,8 +334,8 @@ struct CfgTile {
 };
 
 // Prefill: 64 rows (token, head of the group) per CTA, 16 per warp; the four warps share the key tiles.
-template <int DQ, int DV>
-__global__ void __launch_bounds__(128, 2) attn_prefill_kernel(const AttnArgs a, int rep, int bs_shift) {
+template <int DQ, int DV, int CAP>
+__global__ void __launch_bounds__(128, 2) attn_prefill_kernel(const AttnArgs a, int rep, bool whole) {
   extern __shared__ unsigned char smem_raw[];
   const uint32_t base = (b2::smem_u32(smem_raw) + 127) & ~127u;
   const uint32_t sq = base, skv = base + 64 * DQ * 2;
@@ -318,7 +353,7 @@ __global__ void __launch_bounds__(128, 2) attn_prefill_kernel(const AttnArgs a, 
   const int32_t* bt = a.block_tables + b * a.bt_stride;
   const int pmin = first_pos + tile0 / rep, pmax = first_pos + min(tile0 + 63, rows - 1) / rep;
   const KeyTiles tiles(pmin, pmax, a.window, a.keep_first);
-  const float inv_cap = a.softcap > 0.f ? 1.0f / a.softcap : 0.f;
+  const ScoreScale sscale = score_scale(CAP, a.scale, a.softcap);
   const uint16_t* q = static_cast<const uint16_t*>(a.q);
 #pragma unroll
   for (int i = 0; i < 64 * (DQ / 8) / 128; ++i) {
@@ -328,7 +363,7 @@ __global__ void __launch_bounds__(128, 2) attn_prefill_kernel(const AttnArgs a, 
     const int tok = ok ? gr / rep : 0, hh = ok ? gr - tok * rep : 0;
     b2::cp_async16(b2::tile_addr<DQ>(sq, r, p), q + (row0 + tok) * a.ldq + static_cast<int64_t>(g * rep + hh) * a.qk_pad + (ok ? p * 8 : 0), ok);
   }
-  load_kv_tile<DQ, DV>(a, bt, bs_shift, g, tiles.at(0), pmax, skv, skv + BN * DQ * 2);
+  load_kv_tile<DQ, DV>(a, bt, whole, g, tiles.at(0), pmax, skv, skv + BN * DQ * 2);
   b2::cp_async_commit();
   int pos[2];
 #pragma unroll
@@ -347,7 +382,7 @@ __global__ void __launch_bounds__(128, 2) attn_prefill_kernel(const AttnArgs a, 
     __syncthreads();  // this tile has landed for everyone, and everyone has left the stage that is filled next
     if (it + 1 < tiles.total) {
       const uint32_t nk = skv + ((it + 1) & 1) * CfgTile<DQ, DV>::STAGE;
-      load_kv_tile<DQ, DV>(a, bt, bs_shift, g, tiles.at(it + 1), pmax, nk, nk + BN * DQ * 2);
+      load_kv_tile<DQ, DV>(a, bt, whole, g, tiles.at(it + 1), pmax, nk, nk + BN * DQ * 2);
     }
     b2::cp_async_commit();
     const int j0 = tiles.at(it) * BN;
@@ -370,7 +405,7 @@ __global__ void __launch_bounds__(128, 2) attn_prefill_kernel(const AttnArgs a, 
     }
     const bool all_seen = j0 + BN - 1 <= wpmin && (wpmax - j0 < a.window || j0 + BN - 1 < a.keep_first);
     float corr[2];
-    softmax_tile<BN / 8>(a, s, j0, pos, !all_seen, inv_cap, m, l, corr, lane);
+    softmax_tile<BN / 8, CAP>(a, sscale, s, j0, pos, !all_seen, m, l, corr, lane);
 #pragma unroll
     for (int n = 0; n < DV / 8; ++n) {
       o[n][0] *= corr[0]; o[n][1] *= corr[0]; o[n][2] *= corr[1]; o[n][3] *= corr[1];
@@ -403,9 +438,9 @@ __global__ void __launch_bounds__(128, 2) attn_prefill_kernel(const AttnArgs a, 
     const int tok = gr / rep, head = g * rep + (gr - tok * rep);
     float f = 1.0f;
     if (a.sink != nullptr) {
-      const float sk = a.sink[head], m_new = fmaxf(m[h], sk);
-      f = fast_exp2((m[h] - m_new) * LOG2E);
-      l[h] = l[h] * f + fast_exp2((sk - m_new) * LOG2E);
+      const float sk = a.sink[head] * LOG2E, m_new = fmaxf(m[h], sk);
+      f = fast_exp2(m[h] - m_new);
+      l[h] = l[h] * f + fast_exp2(sk - m_new);
     }
     f /= l[h];
     uint16_t* dst = out + (row0 + tok) * a.ldo + static_cast<int64_t>(head) * a.v_pad;
@@ -422,8 +457,8 @@ __global__ void __launch_bounds__(128, 2) attn_prefill_kernel(const AttnArgs a, 
 constexpr int DEC_MAX_SPLITS = 64;
 constexpr int DEC_MAX_GROUPS = 65536;  // arrival counters at the front of the workspace
 
-template <int DQ, int DV>
-__global__ void __launch_bounds__(128) attn_decode_kernel(const AttnArgs a, int rep, int row_tiles, int bs_shift, int splits, int* counters,
+template <int DQ, int DV, int CAP>
+__global__ void __launch_bounds__(128) attn_decode_kernel(const AttnArgs a, int rep, int row_tiles, bool whole, int splits, int* counters,
                                                           float* part) {
   extern __shared__ unsigned char smem_raw[];
   __shared__ float s_ml[4][16][2];
@@ -450,7 +485,7 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(const AttnArgs a, int 
   const KeyTiles tiles(p, p, a.window, a.keep_first);
   const int per = (tiles.total + splits - 1) / splits;
   const int t0 = split * per, t1 = min(tiles.total, t0 + per);
-  const float inv_cap = a.softcap > 0.f ? 1.0f / a.softcap : 0.f;
+  const ScoreScale sscale = score_scale(CAP, a.scale, a.softcap);
   const uint16_t* q = static_cast<const uint16_t*>(a.q) + b * a.ldq + static_cast<int64_t>(g * rep + h0) * a.qk_pad;
   for (int idx = threadIdx.x; idx < 16 * (DQ / 8); idx += 128) {
     const int r = idx / (DQ / 8), pc = idx % (DQ / 8);
@@ -461,7 +496,7 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(const AttnArgs a, int 
   for (int i = 0; i < STAGES - 1; ++i) {
     if (t0 + i < t1) {
       const uint32_t sk = skv + i * CfgTile<DQ, DV>::STAGE;
-      load_kv_tile<DQ, DV>(a, bt, bs_shift, g, tiles.at(t0 + i), p, sk, sk + BN * DQ * 2);
+      load_kv_tile<DQ, DV>(a, bt, whole, g, tiles.at(t0 + i), p, sk, sk + BN * DQ * 2);
     }
     b2::cp_async_commit();
   }
@@ -478,7 +513,7 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(const AttnArgs a, int 
     __syncthreads();
     if (t + STAGES - 1 < t1) {
       const uint32_t nk = skv + ((t - t0 + STAGES - 1) % STAGES) * CfgTile<DQ, DV>::STAGE;
-      load_kv_tile<DQ, DV>(a, bt, bs_shift, g, tiles.at(t + STAGES - 1), p, nk, nk + BN * DQ * 2);
+      load_kv_tile<DQ, DV>(a, bt, whole, g, tiles.at(t + STAGES - 1), p, nk, nk + BN * DQ * 2);
     }
     b2::cp_async_commit();
     const int j0 = tiles.at(t) * BN + warp * 16;  // this warp's 16 keys
@@ -492,7 +527,7 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(const AttnArgs a, int 
       b2::mma16816(s[1], qa, kb[2], kb[3]);
     }
     float corr[2];
-    softmax_tile<2>(a, s, j0, pos, true, inv_cap, m, l, corr, lane);
+    softmax_tile<2, CAP>(a, sscale, s, j0, pos, j0 + 15 > p || (p - j0 >= a.window && j0 + 15 >= a.keep_first), m, l, corr, lane);
 #pragma unroll
     for (int n = 0; n < DV / 8; ++n) {
       o[n][0] *= corr[0]; o[n][1] *= corr[0]; o[n][2] *= corr[1]; o[n][3] *= corr[1];
@@ -538,15 +573,15 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(const AttnArgs a, int 
     float lt = 0.f, ot = 0.f;
 #pragma unroll
     for (int w = 0; w < 4; ++w) {
-      const float f = s_ml[w][r][0] == -INFINITY ? 0.f : fast_exp2((s_ml[w][r][0] - mt) * LOG2E);
+      const float f = s_ml[w][r][0] == -INFINITY ? 0.f : fast_exp2(s_ml[w][r][0] - mt);
       lt += f * s_ml[w][r][1];
       ot += f * o_buf[(w * 16 + r) * DV + c];
     }
     if (splits == 1) {
       if (a.sink != nullptr) {
-        const float sk = a.sink[g * rep + h0 + r], m_new = fmaxf(mt, sk);
-        const float f = fast_exp2((mt - m_new) * LOG2E);
-        lt = lt * f + fast_exp2((sk - m_new) * LOG2E);
+        const float sk = a.sink[g * rep + h0 + r] * LOG2E, m_new = fmaxf(mt, sk);
+        const float f = fast_exp2(mt - m_new);
+        lt = lt * f + fast_exp2(sk - m_new);
         ot *= f;
       }
       if (c < a.v_pad) out[r * a.v_pad + c] = b2::from_float<uint16_t>(ot / lt);
@@ -569,13 +604,14 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(const AttnArgs a, int 
   const float* all = part + static_cast<int64_t>(group) * splits * 16 * (DV + 2);
   if (threadIdx.x < nrows) {  // the rows' maximum over the splits, and the denominator
     const int r = threadIdx.x;
-    float mt = a.sink != nullptr ? a.sink[g * rep + h0 + r] : -INFINITY;
+    const float sk = a.sink != nullptr ? a.sink[g * rep + h0 + r] * LOG2E : -INFINITY;
+    float mt = sk;
     for (int s = 0; s < splits; ++s) mt = fmaxf(mt, b2::ld_cg_f32(all + static_cast<int64_t>(s) * 16 * (DV + 2) + r));
-    float lt = a.sink != nullptr ? fast_exp2((a.sink[g * rep + h0 + r] - mt) * LOG2E) : 0.f;
+    float lt = fast_exp2(sk - mt);
     for (int s = 0; s < splits; ++s) {
       const float* ps = all + static_cast<int64_t>(s) * 16 * (DV + 2);
       const float ms = b2::ld_cg_f32(ps + r);
-      if (ms > -INFINITY) lt += fast_exp2((ms - mt) * LOG2E) * b2::ld_cg_f32(ps + 16 + r);
+      if (ms > -INFINITY) lt += fast_exp2(ms - mt) * b2::ld_cg_f32(ps + 16 + r);
     }
     s_fin[r][0] = mt;
     s_fin[r][1] = 1.0f / lt;
@@ -587,16 +623,10 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(const AttnArgs a, int 
     for (int s = 0; s < splits; ++s) {
       const float* ps = all + static_cast<int64_t>(s) * 16 * (DV + 2);
       const float ms = b2::ld_cg_f32(ps + r);
-      if (ms > -INFINITY) ot += fast_exp2((ms - s_fin[r][0]) * LOG2E) * b2::ld_cg_f32(ps + 32 + r * DV + c);
+      if (ms > -INFINITY) ot += fast_exp2(ms - s_fin[r][0]) * b2::ld_cg_f32(ps + 32 + r * DV + c);
     }
     if (c < a.v_pad) out[r * a.v_pad + c] = b2::from_float<uint16_t>(ot * s_fin[r][1]);
   }
-}
-
-int log2_exact(int n) {
-  for (int s = 0; s < 31; ++s)
-    if ((1 << s) == n) return s;
-  return -1;
 }
 
 bool tiled_form(int dtype, int qk_pad, int v_pad) { return dtype == B2_DT_BF16 && qk_pad <= 128 && v_pad <= 128; }
@@ -607,30 +637,25 @@ int decode_splits(int B, int max_kv, int nq, int nkv, int window, int keep_first
   const int64_t all = (static_cast<int64_t>(max_kv) + BN - 1) / BN;
   const int64_t seen = (static_cast<int64_t>(keep_first) + BN - 1) / BN + (static_cast<int64_t>(window) + BN - 2) / BN + 1;
   const int64_t tiles = std::max<int64_t>(1, std::min(all, seen));
-  // two CTAs per SM fit; a CTA should have at least two tiles
-  const int64_t want = (2 * 148 + groups - 1) / groups;
-  return static_cast<int>(std::max<int64_t>(1, std::min({want, tiles / 2, static_cast<int64_t>(DEC_MAX_SPLITS)})));
+  // two CTAs per SM fit: about four rounds of them, so that the last one is short; a CTA should have several tiles
+  const int64_t want = (4 * 2 * 148 + groups - 1) / groups;
+  return static_cast<int>(std::max<int64_t>(1, std::min({want, tiles / 4, static_cast<int64_t>(DEC_MAX_SPLITS)})));
 }
 
-template <int DQ, int DV>
-int launch_tiled(const AttnArgs& a, int max_q, int max_kv, void* ws, int64_t ws_bytes, cudaStream_t s) {
+template <int DQ, int DV, int CAP>
+int launch_tiled_cap(const AttnArgs& a, int max_q, int max_kv, void* ws, int64_t ws_bytes, cudaStream_t s) {
   using C = CfgTile<DQ, DV>;
-  const int rep = a.nq / a.nkv, shift = log2_exact(a.block_size);
+  const int rep = a.nq / a.nkv;
+  const bool whole = a.block_size % BN == 0;
   if (a.cu_q != nullptr) {
-    static bool set = false;
-    if (!set) {
-      B2_CUDA(cudaFuncSetAttribute(attn_prefill_kernel<DQ, DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, C::SMEM_PREFILL));
-      set = true;
-    }
+    static const cudaError_t set = cudaFuncSetAttribute(attn_prefill_kernel<DQ, DV, CAP>, cudaFuncAttributeMaxDynamicSharedMemorySize, C::SMEM_PREFILL);
+    B2_CUDA(set);
     const int64_t tiles = (static_cast<int64_t>(max_q) * rep + 63) / 64;
-    B2_CUDA(b2_launch(attn_prefill_kernel<DQ, DV>, dim3(static_cast<unsigned>(tiles), a.nkv, a.B), dim3(128), C::SMEM_PREFILL, s, a, rep, shift));
+    B2_CUDA(b2_launch(attn_prefill_kernel<DQ, DV, CAP>, dim3(static_cast<unsigned>(tiles), a.nkv, a.B), dim3(128), C::SMEM_PREFILL, s, a, rep, whole));
     return B2_OK;
   }
-  static bool set = false;
-  if (!set) {
-    B2_CUDA(cudaFuncSetAttribute(attn_decode_kernel<DQ, DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, C::SMEM_DECODE));
-    set = true;
-  }
+  static const cudaError_t set = cudaFuncSetAttribute(attn_decode_kernel<DQ, DV, CAP>, cudaFuncAttributeMaxDynamicSharedMemorySize, C::SMEM_DECODE);
+  B2_CUDA(set);
   const int row_tiles = (rep + 15) / 16;
   const int64_t groups = static_cast<int64_t>(a.B) * a.nkv * row_tiles;
   int splits = decode_splits(a.B, max_kv, a.nq, a.nkv, a.window, a.keep_first);
@@ -638,9 +663,16 @@ int launch_tiled(const AttnArgs& a, int max_q, int max_kv, void* ws, int64_t ws_
   if (groups > DEC_MAX_GROUPS) splits = 1;
   if (splits > 1 && (ws == nullptr || ws_bytes < need)) return b2::set_error(B2_ERR_SHAPE, "b2_attention: workspace of %lld bytes, %lld needed",
                                                                              static_cast<long long>(ws_bytes), static_cast<long long>(need));
-  B2_CUDA(b2_launch(attn_decode_kernel<DQ, DV>, dim3(splits, a.nkv * row_tiles, a.B), dim3(128), C::SMEM_DECODE, s, a, rep, row_tiles, shift, splits,
-                    static_cast<int*>(ws), reinterpret_cast<float*>(static_cast<unsigned char*>(ws) + DEC_MAX_GROUPS * 4ll)));
+  B2_CUDA(b2_launch(attn_decode_kernel<DQ, DV, CAP>, dim3(splits, a.nkv * row_tiles, a.B), dim3(128), C::SMEM_DECODE, s, a, rep, row_tiles, whole,
+                    splits, static_cast<int*>(ws), reinterpret_cast<float*>(static_cast<unsigned char*>(ws) + DEC_MAX_GROUPS * 4ll)));
   return B2_OK;
+}
+
+template <int DQ, int DV>
+int launch_tiled(const AttnArgs& a, int max_q, int max_kv, void* ws, int64_t ws_bytes, cudaStream_t s) {
+  if (!(a.softcap > 0.f)) return launch_tiled_cap<DQ, DV, CAP_NONE>(a, max_q, max_kv, ws, ws_bytes, s);
+  if (a.softcap <= 256.f) return launch_tiled_cap<DQ, DV, CAP_SHORT>(a, max_q, max_kv, ws, ws_bytes, s);
+  return launch_tiled_cap<DQ, DV, CAP_FULL>(a, max_q, max_kv, ws, ws_bytes, s);
 }
 
 bool aligned16(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; }

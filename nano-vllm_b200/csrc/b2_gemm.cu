@@ -293,7 +293,8 @@ __device__ __forceinline__ uint2 act_mul_pairs(int act, const uint4& w) {
   return make_uint2(b2::pack_bf16(act_mul(act, b2::bf16_lo(w.x), b2::bf16_hi(w.x)), act_mul(act, b2::bf16_lo(w.y), b2::bf16_hi(w.y))),
                     b2::pack_bf16(act_mul(act, b2::bf16_lo(w.z), b2::bf16_hi(w.z)), act_mul(act, b2::bf16_lo(w.w), b2::bf16_hi(w.w))));
 }
-__device__ __forceinline__ float silu_f32(float x) { return x / (1.0f + expf(-x)); }
+// (rounded to bf16 by the store that follows; the quotient is zero where the exponential overflows)
+__device__ __forceinline__ float silu_f32(float x) { return __fdividef(x, 1.0f + __expf(-x)); }
 
 // NC columns (tokens token0 ..) of one feature per lane, features = consecutive lanes.
 // Lanes 2i and 2i+1 hold features f and f+1 of the same tokens.  They swap

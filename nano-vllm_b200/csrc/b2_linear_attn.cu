@@ -447,7 +447,7 @@ int launch_segments(const SegArgs& sa, int max_q, cudaStream_t s) {
 // dim_pad (the padding of o is zero).  One CTA per row.
 // ---------------------------------------------------------------------------
 template <typename T>
-__global__ void gated_norm_kernel(const float* __restrict__ o, int64_t ldo, const T* __restrict__ gate, int64_t ldg,
+__global__ void __launch_bounds__(1024) gated_norm_kernel(const float* __restrict__ o, int64_t ldo, const T* __restrict__ gate, int64_t ldg,
                                   const float* __restrict__ w, float eps, int dim, int dim_pad, T* __restrict__ out, int64_t ld_out) {
   __shared__ float red[32];
   b2::pdl_launch_dependents();
@@ -455,9 +455,14 @@ __global__ void gated_norm_kernel(const float* __restrict__ o, int64_t ldo, cons
   const int row = blockIdx.x;
   const int nvec = dim_pad >> 2;
   const float* orow = o + row * ldo;
-  constexpr int KEEP = 4;  // vectors of the row a thread keeps in registers
-  float4 kept[KEEP];
+  constexpr int KEEP = 4;  // vectors of the row, and of the gate, a thread keeps in registers
+  float4 kept[KEEP], gates[KEEP];
   float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < KEEP; ++i) {
+    const int v = threadIdx.x + i * blockDim.x;
+    gates[i] = v < nvec ? b2::load4<T>(gate + row * ldg + v * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
+  }
 #pragma unroll
   for (int i = 0; i < KEEP; ++i) {
     const int v = threadIdx.x + i * blockDim.x;
@@ -470,19 +475,19 @@ __global__ void gated_norm_kernel(const float* __restrict__ o, int64_t ldo, cons
   }
   ss = b2::block_sum(ss, red);
   const float rstd = 1.0f / sqrtf(ss / static_cast<float>(dim) + eps);
-  auto finish = [&](int v, float4 x) {
-    const float4 g = b2::load4<T>(gate + row * ldg + v * 4);
+  auto sig = [](float x) { return sizeof(T) == 2 ? b2::sigmoid_fast(x) : b2::sigmoid(x); };
+  auto finish = [&](int v, float4 x, const float4& g) {
     const float4 wv = __ldg(reinterpret_cast<const float4*>(w + v * 4));
-    x.x *= rstd * wv.x * b2::sigmoid(g.x); x.y *= rstd * wv.y * b2::sigmoid(g.y);
-    x.z *= rstd * wv.z * b2::sigmoid(g.z); x.w *= rstd * wv.w * b2::sigmoid(g.w);
+    x.x *= rstd * wv.x * sig(g.x); x.y *= rstd * wv.y * sig(g.y);
+    x.z *= rstd * wv.z * sig(g.z); x.w *= rstd * wv.w * sig(g.w);
     b2::store4<T>(out + row * ld_out + v * 4, x);
   };
 #pragma unroll
   for (int i = 0; i < KEEP; ++i) {
     const int v = threadIdx.x + i * blockDim.x;
-    if (v < nvec) finish(v, kept[i]);
+    if (v < nvec) finish(v, kept[i], gates[i]);
   }
-  for (int v = threadIdx.x + KEEP * blockDim.x; v < nvec; v += blockDim.x) finish(v, *reinterpret_cast<const float4*>(orow + v * 4));
+  for (int v = threadIdx.x + KEEP * blockDim.x; v < nvec; v += blockDim.x) finish(v, *reinterpret_cast<const float4*>(orow + v * 4), b2::load4<T>(gate + row * ldg + v * 4));
 }
 
 bool aligned16(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; }

@@ -35,8 +35,10 @@ struct StreamArgs {
 constexpr int MAX_STREAMS = 32;
 
 // ST > 0: number of streams at compile time; ST = 0: a.S streams (at most MAX_STREAMS)
+constexpr int MAX_THREADS = 512;
+
 template <typename T, int ST>
-__global__ void stream_step_kernel(const StreamArgs a) {
+__global__ void __launch_bounds__(MAX_THREADS) stream_step_kernel(const StreamArgs a) {
   extern __shared__ float u_row[];  // [dim_pad]
   __shared__ float coef[MAX_STREAMS * MAX_STREAMS + 2 * MAX_STREAMS];
   __shared__ float red[32];
@@ -124,9 +126,8 @@ bool aligned16(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 
 template <typename T, int ST>
 int launch_step(const StreamArgs& a, cudaStream_t s) {
   const int nvec = a.dim_pad / 4;
-  // few rows: all of a row's vectors at once; many rows: 256 threads, so that several rows share an SM
-  int threads = std::min(a.M <= 296 ? 1024 : 256, (nvec + 31) / 32 * 32);
-  if (ST == 0 || ST > 4) threads = std::min(threads, 256);
+  // few rows: more threads per row; many rows: 256 threads, so that several rows share an SM
+  const int threads = std::min(a.M <= 296 ? MAX_THREADS : 256, (nvec + 31) / 32 * 32);
   const size_t smem = static_cast<size_t>(a.dim_pad) * sizeof(float);
   if (smem > 48 * 1024) B2_CUDA(cudaFuncSetAttribute(stream_step_kernel<T, ST>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)));
   B2_CUDA(b2_launch(stream_step_kernel<T, ST>, dim3(a.M), dim3(threads), smem, s, a));

@@ -15,6 +15,11 @@ cases:
   rowpar_prefill  fused row-parallel launch, M=1024, N=5120, Kr=1024
   store_kvcache   paged-KV scatter, 16384 tokens x D=1024
   add_rmsnorm     residual add + RMSNorm, 16384 x 4096
+  window_prefill  window attention (soft cap, sink, 1024 + 4 tokens), 4 prompts of 2048, 32 query / 8 key-value heads of 128
+  window_decode   the same for 64 sequences of 1024 tokens, one row each, 6 layers' caches
+  linear_prefill  decayed linear attention, 4 prompts of 2048, 32 heads of 128 x 128
+  linear_decode   the same for 64 sequences, one row each, 4 layers' states
+  stream_step     residual streams (4) between two sublayers, 8192 x 4096
   embed           embedding lookup, 16384 ids into a [151936, 4096] table (one rank)
 """
 from __future__ import annotations
@@ -86,6 +91,29 @@ def main():
     elif a.case == "add_rmsnorm":
         xs, rs, nw = [rnd(16384, 4096) for _ in range(2)], [rnd(16384, 4096) for _ in range(2)], rnd(4096)
         call = lambda i: ops.add_rmsnorm(xs[i % 2], rs[i % 2], nw, 1e-6)
+    elif a.case in ("window_prefill", "window_decode", "linear_prefill", "linear_decode"):
+        heads, nkv, d = 32, 8, 128
+        prefill = a.case.endswith("prefill")
+        seqs, length, layers = (4, 2048, 1) if prefill else (64, 1024, 6)
+        rows = seqs * length if prefill else seqs
+        cu = torch.arange(0, rows + 1, length, device=dev, dtype=torch.int32) if prefill else None
+        kl = torch.full((seqs,), length, dtype=torch.int32, device=dev)
+        if a.case.startswith("window"):
+            blocks = seqs * length // 256
+            kc, vc = ([rnd(blocks, 256, nkv, d) for _ in range(layers)] for _ in range(2))
+            bt = torch.randperm(blocks, device=dev, generator=g).int().view(seqs, -1).contiguous()
+            q, sink = rnd(rows, heads * d), torch.zeros(heads, device=dev)
+            call = lambda i: ops.window_attention(q, heads, kc[i % layers], vc[i % layers], bt, cu, kl, length if prefill else 1, length, d ** -0.5, 30.0, 1024, 4, sink)
+        else:
+            decay = 1.0 - 2.0 ** (-2 - 6 * torch.arange(heads, dtype=torch.float64) / heads)
+            dec, pw = decay.float().to(dev), (decay.unsqueeze(1) ** torch.arange(65)).float().to(dev)
+            states = [torch.zeros(seqs, heads, d, d, device=dev) for _ in range(min(4, layers))]
+            p, sl = rnd(rows, 4 * heads * d), torch.arange(seqs, device=dev, dtype=torch.int32)
+            call = lambda i: ops.linear_attn(p, heads, d, d, states[i % len(states)], sl, cu, kl, length if prefill else 1, dec, pw)
+    elif a.case == "stream_step":
+        x, y = torch.randn(8192, 4, 4096, device=dev), rnd(8192, 4096)
+        mix, one, nw = torch.eye(4, device=dev), torch.ones(4, device=dev), torch.ones(4096, device=dev)
+        call = lambda i: ops.stream_step(x, y, mix, one, 0.1, one / 4, nw, 1e-6, 4096)
     elif a.case == "embed":
         w = rnd(151936, 4096)
         ids = [torch.randint(0, 151936, (16384,), device=dev, generator=g) for _ in range(2)]
