@@ -375,9 +375,11 @@ def _kernel_table(torch, z: dict, peaks: dict, batch: int, ctx_len: int) -> list
     us2 = time_in_graph(lambda i: ops.linear_attn(p, H, d, d, state, sl, cu, kl, L, dec, pw), 4, 24)
     full = 4.0 * H * d * B * L * (L + 1) / 2
     lus2 = time_in_graph(lambda i: flash_attn_varlen_func(q.view(M, H, d), k, v, cu, cu, L, L, softmax_scale=d ** -0.5, causal=True), 4, 24)
-    add(f"linear_attn prefill {B}x{L}", "flash-attn, full causal", lin_flops, us2, full, lus2, "tensor")
-    lin_bytes = M * H * d * (3 * 2 + 4.0)
-    rows[-1]["frac_of_hbm"] = round(lin_bytes / (us2 * 1e-6) / (peaks["hbm_gbs"] * 1e9), 3)
+    # bound by memory: its bytes (q, k, v in bf16, o in fp32) take longer than its flops; the like kernel by the tensor pipe
+    roof = max(M * H * d * (3 * 2 + 4.0) / (peaks["hbm_gbs"] * 1e9), lin_flops / (peaks["bf16_tflops"] * 1e12)) * 1e6
+    lroof = full / (peaks["bf16_tflops"] * 1e12) * 1e6
+    rows.append({"kernel": f"linear_attn prefill {B}x{L}", "us": round(us2, 2), "bound": "hbm", "frac": round(roof / us2, 3), "like": "flash-attn, full causal",
+                 "like_us": round(lus2, 2), "like_frac": round(lroof / lus2, 3), "like_over_this": round((lroof / lus2) / (roof / us2), 2)})
     # decode
     nblk = -(-ctx_len // 256)
     n_layers = 6

@@ -153,8 +153,8 @@ __global__ void __launch_bounds__(256) linear_attn_decode_kernel(const LinArgs a
 }
 
 // ---------------------------------------------------------------------------
-// Prefill, bf16, heads up to 128 wide, on the tensor cores.  A sequence is cut into segments of SEG tokens, a segment
-// into chunks of 64.  With P_n = decay^n, inside a chunk that starts from state S:
+// Prefill, bf16, heads up to 128 wide, on the tensor cores.  A sequence is walked in chunks of 64 tokens; where there
+// are too few heads and sequences to fill the SMs it is cut into segments that run side by side.  With P_n = decay^n, inside a chunk that starts from state S:
 //     o_i = P_(i+1) S^T q_i + sum_(j <= i) P_(i-j) (q_i . k_j) v_j
 //     S'  = P_n S + sum_j k_j (P_(n-1-j) v_j)^T
 // q, k, v are exact bf16; S, the decayed scores and the decayed values are fp32 and enter the products as a sum of two
@@ -166,8 +166,9 @@ constexpr int CH = 64, SEG = 512, VT = 64;
 struct SegArgs {
   LinArgs a;
   const float* powers;  // [heads][65]
-  float* seg_state;     // [segments][heads][qk_pad][v_pad]; sequence b's segments start at cu_q[b] / SEG + b
-  int multi;            // the segments' start states are in seg_state
+  float* seg_state;     // [segments][heads][qk_pad][v_pad]; sequence b's segments start at cu_q[b] / seg + b
+  int seg;              // tokens per segment, a multiple of 64
+  int multi;            // some sequence has several segments: their start states are in seg_state
 };
 
 template <int DQ>
@@ -192,7 +193,7 @@ __global__ void __launch_bounds__(128, 2) linear_attn_segment_kernel(const SegAr
   b2::pdl_wait();
   const int row0 = a.cu_q[b];
   const int n_q = a.cu_q[b + 1] - row0;
-  const int t_begin = seg * SEG, t_end = min(n_q, t_begin + SEG);
+  const int t_begin = seg * sa.seg, t_end = min(n_q, t_begin + sa.seg);
   if (t_begin >= n_q) return;
   const bool final_seg = t_end == n_q;
   if (SUMS && final_seg) return;  // no segment starts from its sum
@@ -200,7 +201,7 @@ __global__ void __launch_bounds__(128, 2) linear_attn_segment_kernel(const SegAr
   const int D = a.qk_pad;
   const int64_t head_state = static_cast<int64_t>(D) * a.v_pad;
   float* slot_state = slot >= 0 ? a.state + (static_cast<int64_t>(slot) * a.heads + h) * head_state : nullptr;
-  float* seg_state = sa.seg_state + (static_cast<int64_t>(row0 / SEG + b + seg) * a.heads + h) * head_state;
+  float* seg_state = sa.seg_state + (static_cast<int64_t>(row0 / sa.seg + b + seg) * a.heads + h) * head_state;
 
   const uint16_t* qkv = static_cast<const uint16_t*>(a.qkv);
   const int64_t off_q = static_cast<int64_t>(h) * D, off_k = static_cast<int64_t>(a.heads + h) * D;
@@ -233,7 +234,7 @@ __global__ void __launch_bounds__(128, 2) linear_attn_segment_kernel(const SegAr
     return (src != nullptr && r < D && c < a.v_pad) ? *reinterpret_cast<const float2*>(src + static_cast<int64_t>(r) * a.v_pad + c) : make_float2(0.f, 0.f);
   };
   const float* start = nullptr;
-  if (!SUMS) start = sa.multi && n_q > SEG ? seg_state : (a.kv_len[b] == n_q ? nullptr : slot_state);
+  if (!SUMS) start = sa.multi && n_q > sa.seg ? seg_state : (a.kv_len[b] == n_q ? nullptr : slot_state);
 #pragma unroll
   for (int mt = 0; mt < MT; ++mt)
 #pragma unroll
@@ -399,29 +400,42 @@ __global__ void __launch_bounds__(256) linear_attn_scan_kernel(const SegArgs sa)
   b2::pdl_wait();
   const int b = blockIdx.z, h = blockIdx.y;
   const int row0 = a.cu_q[b], n_q = a.cu_q[b + 1] - row0;
-  if (n_q <= SEG) return;
-  const int segs = (n_q + SEG - 1) / SEG;
+  if (n_q <= sa.seg) return;
+  const int segs = (n_q + sa.seg - 1) / sa.seg;
   const int64_t head_state = static_cast<int64_t>(a.qk_pad) * a.v_pad;
   const int64_t e = (static_cast<int64_t>(blockIdx.x) * 256 + threadIdx.x) * 4;
   if (e >= head_state) return;
   float p = sa.powers[h * (CH + 1) + CH], ps = 1.0f;
-  for (int i = 0; i < SEG / CH; ++i) ps *= p;
+  for (int i = 0; i < sa.seg / CH; ++i) ps *= p;
   const int slot = a.slots[b];
   float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
   if (slot >= 0 && a.kv_len[b] != n_q) s = *reinterpret_cast<const float4*>(a.state + (static_cast<int64_t>(slot) * a.heads + h) * head_state + e);
-  float* at = sa.seg_state + (static_cast<int64_t>(row0 / SEG + b) * a.heads + h) * head_state + e;
+  float* at = sa.seg_state + (static_cast<int64_t>(row0 / sa.seg + b) * a.heads + h) * head_state + e;
   const int64_t step = a.heads * head_state;
-  for (int i = 0; i < segs; ++i, at += step) {
-    float4 own = make_float4(0.f, 0.f, 0.f, 0.f);
-    if (i + 1 < segs) own = *reinterpret_cast<const float4*>(at);
-    *reinterpret_cast<float4*>(at) = s;
-    s.x = fmaf(ps, s.x, own.x); s.y = fmaf(ps, s.y, own.y); s.z = fmaf(ps, s.z, own.z); s.w = fmaf(ps, s.w, own.w);
+  constexpr int AHEAD = 4;  // contributions in flight per thread
+  for (int i0 = 0; i0 < segs; i0 += AHEAD) {
+    float4 own[AHEAD];
+#pragma unroll
+    for (int i = 0; i < AHEAD; ++i)
+      own[i] = i0 + i + 1 < segs ? *reinterpret_cast<const float4*>(at + i * step) : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+    for (int i = 0; i < AHEAD; ++i, at += step) {
+      if (i0 + i >= segs) return;
+      *reinterpret_cast<float4*>(at) = s;
+      s.x = fmaf(ps, s.x, own[i].x); s.y = fmaf(ps, s.y, own[i].y); s.z = fmaf(ps, s.z, own[i].z); s.w = fmaf(ps, s.w, own[i].w);
+    }
   }
 }
 
 bool segment_form(int dtype, int qk_pad, int v_pad) { return dtype == B2_DT_BF16 && qk_pad <= 128; }
 
-int64_t segment_slots(int B, int total_q) { return static_cast<int64_t>(total_q) / SEG + B + 1; }
+// Tokens per segment.  A sequence in one piece does no work twice, so it is cut only where the CTAs of whole sequences
+// (total / longest of them run side by side, two on an SM) would leave SMs idle.
+int segment_length(int max_q, int total_q, int heads, int v_pad) {
+  const int64_t ctas = static_cast<int64_t>(heads) * ((v_pad + VT - 1) / VT) * std::max(total_q, 1) / std::max(max_q, 1);
+  return max_q <= SEG || ctas >= 230 ? (max_q + CH - 1) / CH * CH : SEG;
+}
+int64_t segment_slots(int B, int total_q, int seg) { return static_cast<int64_t>(total_q) / seg + B + 1; }
 
 template <int DQ>
 int launch_segments(const SegArgs& sa, int max_q, cudaStream_t s) {
@@ -432,7 +446,7 @@ int launch_segments(const SegArgs& sa, int max_q, cudaStream_t s) {
     B2_CUDA(cudaFuncSetAttribute(linear_attn_segment_kernel<DQ, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, CfgSeg<DQ>::SMEM));
     set = true;
   }
-  const dim3 grid((max_q + SEG - 1) / SEG, a.heads * ((a.v_pad + VT - 1) / VT), a.B);
+  const dim3 grid((max_q + sa.seg - 1) / sa.seg, a.heads * ((a.v_pad + VT - 1) / VT), a.B);
   if (sa.multi) {
     B2_CUDA(b2_launch(linear_attn_segment_kernel<DQ, true>, grid, dim3(128), CfgSeg<DQ>::SMEM, s, sa));
     const int64_t quads = static_cast<int64_t>(a.qk_pad) * a.v_pad / 4;
@@ -505,8 +519,9 @@ int launch_any(const LinArgs& a, cudaStream_t s) {
 extern "C" {
 
 int64_t b2_linear_attn_workspace(int dtype, int B, int max_q, int total_q, int heads, int qk_pad, int v_pad) {
-  if (max_q <= SEG || B <= 0 || !segment_form(dtype, qk_pad, v_pad)) return 0;
-  return segment_slots(B, total_q) * heads * qk_pad * v_pad * 4;
+  if (max_q <= 0 || B <= 0 || heads <= 0 || !segment_form(dtype, qk_pad, v_pad)) return 0;
+  const int seg = segment_length(max_q, total_q, heads, v_pad);
+  return max_q <= seg ? 0 : segment_slots(B, total_q, seg) * heads * qk_pad * v_pad * 4;
 }
 
 int b2_linear_attn(int dtype, const void* qkv, int64_t ld_qkv, float* o, int64_t ldo, float* state, const int32_t* slots, const int32_t* cu_q,
@@ -534,9 +549,10 @@ int b2_linear_attn(int dtype, const void* qkv, int64_t ld_qkv, float* o, int64_t
   SegArgs sa{};
   sa.a = a;
   sa.powers = decay_powers;
-  sa.multi = max_q > SEG;
+  sa.seg = segment_length(max_q, total_q, heads, v_pad);
+  sa.multi = max_q > sa.seg;
   sa.seg_state = static_cast<float*>(workspace);
-  if (sa.multi && (workspace == nullptr || workspace_bytes < segment_slots(B, total_q) * heads * qk_pad * v_pad * 4))
+  if (sa.multi && (workspace == nullptr || workspace_bytes < segment_slots(B, total_q, sa.seg) * heads * qk_pad * v_pad * 4))
     return b2::set_error(B2_ERR_SHAPE, "b2_linear_attn: workspace of %lld bytes is too small", static_cast<long long>(workspace_bytes));
   return qk_pad <= 64 ? launch_segments<64>(sa, max_q, s) : launch_segments<128>(sa, max_q, s);
 }

@@ -317,6 +317,10 @@ def test_linear_attention_across_segments(case):
     run_linear(torch.bfloat16, heads, d, dv, decay, [700, 1090, 5], [600, 1025, 2], seed=case + 5, slots=[2, 0, 5])
 
 
+def test_linear_attention_many_heads_walk_long_prompts_in_one_piece():
+    run_linear(torch.bfloat16, 130, 16, 24, [0.5 + i / 270 for i in range(130)], [600, 585], [600, 520])
+
+
 @pytest.mark.parametrize("case", range(len(LIN)))
 @pytest.mark.parametrize("dtype,form", [(torch.float32, 0), (torch.bfloat16, 0), (torch.bfloat16, 1)])
 def test_linear_attention_decode(case, dtype, form):
