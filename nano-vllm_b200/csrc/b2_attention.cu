@@ -20,10 +20,9 @@ namespace {
 // per lane and pass.  Head strides are padded to 8 elements; the padding is zero and stays zero.
 // ---------------------------------------------------------------------------
 template <typename T, int LANES>
-__global__ void __launch_bounds__(256) qk_norm_store_kernel(T* __restrict__ qkv, int64_t ld, int M, int nq, int nkv, int qk_dim, int qk_pad,
+__global__ void __launch_bounds__(256) qk_norm_store_kernel(T* qkv, int64_t ld, int M, int nq, int nkv, int qk_dim, int qk_pad,
                                                             int v_pad, const T* __restrict__ qw, const T* __restrict__ kw, float eps,
-                                                            T* __restrict__ k_cache, T* __restrict__ v_cache,
-                                                            const int32_t* __restrict__ slots) {
+                                                            T* k_cache, T* v_cache, const int32_t* slots) {
   b2::pdl_launch_dependents();
   b2::pdl_wait();
   const int heads = nq + 2 * nkv;

@@ -93,6 +93,9 @@ __device__ __forceinline__ void report_timeout(B2Status* st, int detail) {
 // does before pdl_wait() must be independent of earlier kernels (set-up,
 // loads of weights); pdl_wait() returns once every earlier kernel has
 // completed and its writes are visible.  Both are no-ops for a plain launch.
+// Kernel parameters that an earlier kernel writes must not be __restrict__: the
+// compiler may then take the memory clobber below as not concerning them and
+// move their loads in front of the wait.
 __device__ __forceinline__ void pdl_wait() { asm volatile("griddepcontrol.wait;" ::: "memory"); }
 __device__ __forceinline__ void pdl_launch_dependents() { asm volatile("griddepcontrol.launch_dependents;" ::: "memory"); }
 

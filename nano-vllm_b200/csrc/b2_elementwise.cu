@@ -353,7 +353,7 @@ __device__ __forceinline__ unsigned long long argmax_key(float v, int idx) {
   return (static_cast<unsigned long long>(b) << 32) | (0xFFFFFFFFu - static_cast<uint32_t>(idx));
 }
 
-__global__ void __launch_bounds__(256) argmax_partial_kernel(const uint16_t* __restrict__ logits, int64_t ld, int V, int cols_per_block,
+__global__ void __launch_bounds__(256) argmax_partial_kernel(const uint16_t* logits, int64_t ld, int V, int cols_per_block,
                                                              unsigned long long* __restrict__ keys) {
   b2::pdl_launch_dependents();
   b2::pdl_wait();
@@ -364,7 +364,7 @@ __global__ void __launch_bounds__(256) argmax_partial_kernel(const uint16_t* __r
   const int v0 = c0 >> 3, v1 = c1 >> 3;  // cols_per_block is a multiple of 8
   for (int v = v0 + threadIdx.x; v < v1; v += blockDim.x) {
     float f[8];
-    unpack8(ldg_v4(row + v * 8), f);
+    unpack8(*reinterpret_cast<const uint4*>(row + v * 8), f);
 #pragma unroll
     for (int e = 0; e < 8; ++e)
       if (f[e] > best) { best = f[e]; best_i = v * 8 + e; }
@@ -388,7 +388,7 @@ __global__ void __launch_bounds__(256) argmax_partial_kernel(const uint16_t* __r
   }
 }
 
-__global__ void argmax_finish_kernel(int64_t* __restrict__ out, int B) {
+__global__ void argmax_finish_kernel(int64_t* out, int B) {
   b2::pdl_launch_dependents();
   b2::pdl_wait();
   const int i = blockIdx.x * blockDim.x + threadIdx.x;

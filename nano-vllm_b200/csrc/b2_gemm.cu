@@ -1936,9 +1936,7 @@ int check_operands(const void* A, int64_t lda, const void* W, int64_t ldw, int M
 
 // rows of h picked by index into a contiguous staging buffer (the prefill
 // "last token of every sequence" selection)
-__global__ void __launch_bounds__(256) gather_rows_kernel(const uint16_t* __restrict__ h, int64_t ldh,
-                                                          const int32_t* __restrict__ idx, int B, int H,
-                                                          uint16_t* __restrict__ out) {
+__global__ void __launch_bounds__(256) gather_rows_kernel(const uint16_t* h, int64_t ldh, const int32_t* idx, int B, int H, uint16_t* out) {
   b2::pdl_launch_dependents();
   b2::pdl_wait();
   const int vpr = H >> 3;
@@ -1947,7 +1945,7 @@ __global__ void __launch_bounds__(256) gather_rows_kernel(const uint16_t* __rest
        i += static_cast<int64_t>(gridDim.x) * blockDim.x) {
     const int b = static_cast<int>(i / vpr), v = static_cast<int>(i - static_cast<int64_t>(b) * vpr);
     *reinterpret_cast<uint4*>(out + static_cast<int64_t>(b) * H + v * 8) =
-        __ldg(reinterpret_cast<const uint4*>(h + idx[b] * ldh + v * 8));
+        *reinterpret_cast<const uint4*>(h + idx[b] * ldh + v * 8);
   }
 }
 

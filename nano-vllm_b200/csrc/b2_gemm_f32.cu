@@ -11,8 +11,8 @@ __device__ __forceinline__ float act_pair(float g, float u, int act) {
   return (act == B2_ACT_RELU ? fmaxf(g, 0.f) : g * b2::sigmoid(g)) * u;
 }
 
-__global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__ A, int64_t lda, const float* __restrict__ W, int64_t ldw,
-                                                       float* __restrict__ C, int64_t ldc, int M, int N, int K, int pair_act, int silu_cols) {
+__global__ void __launch_bounds__(256) gemm_f32_kernel(const float* A, int64_t lda, const float* __restrict__ W, int64_t ldw,
+                                                       float* C, int64_t ldc, int M, int N, int K, int pair_act, int silu_cols) {
   __shared__ float sa[TK][TM + 4];
   __shared__ float sw[TK][TN + 4];
   b2::pdl_launch_dependents();

@@ -461,8 +461,8 @@ int launch_segments(const SegArgs& sa, int max_q, cudaStream_t s) {
 // dim_pad (the padding of o is zero).  One CTA per row.
 // ---------------------------------------------------------------------------
 template <typename T>
-__global__ void __launch_bounds__(1024) gated_norm_kernel(const float* __restrict__ o, int64_t ldo, const T* __restrict__ gate, int64_t ldg,
-                                  const float* __restrict__ w, float eps, int dim, int dim_pad, T* __restrict__ out, int64_t ld_out) {
+__global__ void __launch_bounds__(1024) gated_norm_kernel(const float* o, int64_t ldo, const T* gate, int64_t ldg, const float* w, float eps, int dim,
+                                                           int dim_pad, T* out, int64_t ld_out) {
   __shared__ float red[32];
   b2::pdl_launch_dependents();
   b2::pdl_wait();
