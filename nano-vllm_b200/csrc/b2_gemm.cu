@@ -280,10 +280,12 @@ __host__ __device__ __forceinline__ int owned_rows3(int M, int world, int rank) 
 // (row of the P tile) q*32 + lane and columns c*32 .. c*32+31 (rows of the Q
 // tile).
 // ---------------------------------------------------------------------------
+// fp32 to a few units in the last place: every user rounds it to bf16 (zero where the exponential overflows)
+__device__ __forceinline__ float silu_f32(float x) { return __fdividef(x, 1.0f + __expf(-x)); }
 // silu(gate) * up on bf16-rounded inputs, with the reference's roundings (nanovllm/layers/activation.py:8-11, eager):
 // the activation is rounded to bf16 before the product, the product once more by the caller's pack
 __device__ __forceinline__ float silu_mul(float gate, float up) {
-  return b2::bf16_round(gate / (1.0f + expf(-gate))) * up;
+  return b2::bf16_round(silu_f32(gate)) * up;
 }
 __device__ __forceinline__ float act_mul(int act, float gate, float up) {
   return act == B2_ACT_RELU ? fmaxf(gate, 0.f) * up : silu_mul(gate, up);
@@ -293,8 +295,6 @@ __device__ __forceinline__ uint2 act_mul_pairs(int act, const uint4& w) {
   return make_uint2(b2::pack_bf16(act_mul(act, b2::bf16_lo(w.x), b2::bf16_hi(w.x)), act_mul(act, b2::bf16_lo(w.y), b2::bf16_hi(w.y))),
                     b2::pack_bf16(act_mul(act, b2::bf16_lo(w.z), b2::bf16_hi(w.z)), act_mul(act, b2::bf16_lo(w.w), b2::bf16_hi(w.w))));
 }
-// (rounded to bf16 by the store that follows; the quotient is zero where the exponential overflows)
-__device__ __forceinline__ float silu_f32(float x) { return __fdividef(x, 1.0f + __expf(-x)); }
 
 // NC columns (tokens token0 ..) of one feature per lane, features = consecutive lanes.
 // Lanes 2i and 2i+1 hold features f and f+1 of the same tokens.  They swap
