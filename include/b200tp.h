@@ -352,6 +352,14 @@ int b2_lm_head(b2_ctx* ctx, const void* h, int64_t ldh, const int32_t* row_index
 int b2_lm_head_sample(b2_ctx* ctx, const void* h, int64_t ldh, const int32_t* row_index, const void* W, int64_t ldw,
                       int B, int Vr, int H, const float* temperatures, uint64_t seed, int64_t* tokens_out, void* stream);
 
+/* The same for a model that transforms its logits: the sampled logit is
+ * logit_cap tanh(logit_scale logit / logit_cap), or logit_scale logit when
+ * logit_cap <= 0.  logit_scale must be positive (a greedy pick then does not
+ * depend on either). */
+int b2_lm_head_sample_capped(b2_ctx* ctx, const void* h, int64_t ldh, const int32_t* row_index, const void* W, int64_t ldw,
+                             int B, int Vr, int H, float logit_scale, float logit_cap, const float* temperatures,
+                             uint64_t seed, int64_t* tokens_out, void* stream);
+
 /* Host copies of the fused sampler's generator, for tests (no CUDA call): the
  * 32 random bits behind E for (vocab_id, row `token`) in call number `call`
  * (u = ((bits >> 9) + 0.5) * 2^-23), and Philox4x32-10 itself. */
@@ -472,6 +480,83 @@ int b2_linear_attn(int dtype, const void* qkv, int64_t ld_qkv, float* o, int64_t
  * the mean over `dim` of dim_pad elements (the rest of o is zero). */
 int b2_gated_norm(int dtype, const float* o, int64_t ldo, const void* gate, int64_t ldg, const float* w, float eps, int M,
                   int dim, int dim_pad, void* out, int64_t ld_out, void* stream);
+
+/* Residual (one copy, fp32) with a norm before and after every sublayer and a
+ * short causal convolution on what a sublayer reads; everything between two
+ * sublayers in one launch.  Per token t of a sequence:
+ *   ids != NULL:  x = table[ids]                               (start of the model)
+ *   y != NULL:    x <- x + post_w * y / sqrt(mean(y^2) + eps)
+ *   h   = norm_w * x / sqrt(mean(x^2) + eps), rounded to the activations' type
+ *   out = h + sum_j conv_w[j] * h_(t - taps + 1 + j)            (taps 0: out = h)
+ * means over `dim` elements; post_w / norm_w are fp32 with 1 element (a gain) or
+ * dim_pad (one per channel).  conv_w is [taps][dim_pad], state
+ * [slots][taps - 1][dim_pad], both in the activations' type: h before the step's
+ * first token is read from the sequence's slot (zeros when the step starts at
+ * position 0, whatever the slot holds), and the slot is left with the step's last
+ * taps - 1 values; slots[b] -1 marks a padded row.  cu_q / kv_len as in
+ * b2_attention (cu_q NULL: row b is sequence b's only token).  x_out (NULL = not
+ * stored) must be another buffer than x_in unless cu_q is NULL or taps is 0.
+ * run: tokens per CTA, 0 = the library chooses. */
+int b2_sandwich_step(int dtype, const float* x_in, float* x_out, const int64_t* ids, const void* table, int64_t ld_table,
+                     int64_t vocab, const void* y, int64_t ldy, const float* post_w, int post_len, const float* norm_w,
+                     int norm_len, float eps, const void* conv_w, int taps, void* state, const int32_t* slots,
+                     const int32_t* cu_q, const int32_t* kv_len, int B, int max_q, void* out, int64_t ldo, int dim,
+                     int dim_pad, int run, void* stream);
+
+/* out = coef[0] N(z) + coef[1] N(z^2) + coef[2] N(z^3) + coef[3] per element, N
+ * dividing by sqrt(mean + eps) of the squares over the row's `dim` elements;
+ * elements dim .. dim_pad of out are zero.  coef: 4 fp32 on the device. */
+int b2_poly_norm(int dtype, const void* z, int64_t ldz, const float* coef, float eps, int M, int dim, int dim_pad, void* out,
+                 int64_t ldo, void* stream);
+
+/* fp32 out = cap tanh(scale x / cap) (cap <= 0: scale x); cols a multiple of 8. */
+int b2_logit_cap(int dtype, const void* x, int64_t ldx, float scale, float cap, int M, int cols, float* out, int64_t ldo,
+                 void* stream);
+
+/* ---- latent attention: the cache holds one row [latent | rotated key part] of
+ * kv_pad + rot_pad elements per token, shared by all heads.  Pairs of adjacent
+ * elements (u, v) of a rotated part become (u cos - v sin, v cos + u sin);
+ * cos_sin: fp32 [max_pos][rot_pad / 2][2], positions past it use its last row.
+ *
+ * Rows [q_pad query latent | kv_pad latent | rot_pad rotated part | ...] in place:
+ * both latents RMS-normed (weights fp32, q_pad / kv_pad elements), the last part
+ * rotated; latent and rotated part are also written to the cache row of
+ * slot_mapping[token] (-1 stores nothing; cache may be NULL). */
+int b2_latent_store(int dtype, void* rows, int64_t ld, int M, int q_dim, int q_pad, int kv_dim, int kv_pad, int rot_pad,
+                    const float* q_norm_w, const float* kv_norm_w, float eps, const int64_t* positions,
+                    const float* cos_sin, int max_pos, void* cache, const int32_t* slot_mapping, void* stream);
+/* Cached rows (row elements each) of every sequence as contiguous rows: position j of sequence b to row cu_k[b] + j. */
+int b2_latent_gather(int dtype, const void* cache, const int32_t* block_tables, int64_t bt_stride, int block_size,
+                     const int32_t* cu_k, int B, int max_kv, int row, void* out, void* stream);
+
+/* One matrix product per head: out[m, h, n] = sum_k x[m, h, k] W_h[n, k], W_h at
+ * w + h w_head with rows of ldw elements, [N][K] or (w_is_kn) [K][N]; a head's
+ * inputs / outputs start every x_head / out_head elements.  gate (may be NULL):
+ * out is multiplied by sigmoid(gate[m, h gate_head + n]).  rot_pad > 0: the
+ * rot_pad elements behind a head's K inputs are rotated by positions[m] and
+ * written behind its N outputs. */
+int b2_heads_gemm(int dtype, const void* x, int64_t ldx, int x_head, const void* w, int64_t ldw, int64_t w_head, int w_is_kn,
+                  void* out, int64_t ldo, int out_head, int M, int heads, int N, int K, const void* gate, int64_t ldg,
+                  int gate_head, int rot_pad, const int64_t* positions, const float* cos_sin, int max_pos, void* stream);
+
+/* Absorbed attention: every head's query [lat_pad | rot_pad] attends to the cached
+ * rows themselves (score = q . row * scale) and mixes their first lat_pad
+ * elements: out [M][heads][lat_pad].  Causal; the rest as in b2_attention. */
+int64_t b2_latent_attention_workspace(int dtype, int B, int max_q, int max_kv, int heads, int lat_pad, int rot_pad);
+int b2_latent_attention(int dtype, const void* q, int64_t ldq, void* out, int64_t ldo, const void* cache,
+                        const int32_t* block_tables, int64_t bt_stride, int block_size, const int32_t* cu_q,
+                        const int32_t* kv_len, int B, int max_q, int max_kv, int heads, int lat_pad, int rot_pad, float scale,
+                        const float* sink, void* workspace, int64_t workspace_bytes, int form, void* stream);
+
+/* Expanded attention (bf16; dim_pad + rot_pad <= 192, v_pad <= 128): rows of kv hold
+ * [dim_pad key | v_pad value] per head, rows of rot the shared rotated key part;
+ * position j of sequence b is row cu_k[b] + j of both.  q heads are
+ * [dim_pad | rot_pad], not yet rotated.  out [M][heads][v_pad] is multiplied by
+ * sigmoid(gate) when gate ([M][heads][v_pad], row stride ldg) is given. */
+int b2_expanded_attention(const void* q, int64_t ldq, void* out, int64_t ldo, const void* kv, int64_t ld_kv, const void* rot,
+                          int64_t ld_rot, const int32_t* cu_q, const int32_t* cu_k, int B, int max_q, int heads, int dim_pad,
+                          int rot_pad, int v_pad, float scale, const float* sink, const float* cos_sin, int max_pos,
+                          const void* gate, int64_t ldg, void* stream);
 
 /* Greedy pick: out[i] = argmax_j logits[i, j] (first index on ties), int64.
  * The reference's Sampler (nanovllm/layers/sampler.py:7-12) at temperature -> 0. */

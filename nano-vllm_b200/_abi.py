@@ -68,6 +68,14 @@ SIGNATURES = {
     "b2_attention": [_i, _p, _i64, _p, _i64, _p, _p, _p, _i64, _i, _p, _p, _i, _i, _i, _i, _i, _i, _i, _f, _f, _i, _i, _p, _p, _i64, _i, _p],
     "b2_linear_attn": [_i, _p, _i64, _p, _i64, _p, _p, _p, _p, _p, _p, _i, _i, _i, _i, _i, _i, _p, _i64, _i, _p],
     "b2_gated_norm": [_i, _p, _i64, _p, _i64, _p, _f, _i, _i, _i, _p, _i64, _p],
+    "b2_sandwich_step": [_i, _p, _p, _p, _p, _i64, _i64, _p, _i64, _p, _i, _p, _i, _f, _p, _i, _p, _p, _p, _p, _i, _i, _p, _i64, _i, _i, _i, _p],
+    "b2_poly_norm": [_i, _p, _i64, _p, _f, _i, _i, _i, _p, _i64, _p],
+    "b2_logit_cap": [_i, _p, _i64, _f, _f, _i, _i, _p, _i64, _p],
+    "b2_latent_store": [_i, _p, _i64, _i, _i, _i, _i, _i, _i, _p, _p, _f, _p, _p, _i, _p, _p, _p],
+    "b2_latent_gather": [_i, _p, _p, _i64, _i, _p, _i, _i, _i, _p, _p],
+    "b2_heads_gemm": [_i, _p, _i64, _i, _p, _i64, _i64, _i, _p, _i64, _i, _i, _i, _i, _i, _p, _i64, _i, _i, _p, _p, _i, _p],
+    "b2_latent_attention": [_i, _p, _i64, _p, _i64, _p, _p, _i64, _i, _p, _p, _i, _i, _i, _i, _i, _i, _f, _p, _p, _i64, _i, _p],
+    "b2_expanded_attention": [_p, _i64, _p, _i64, _p, _i64, _p, _i64, _p, _p, _i, _i, _i, _i, _i, _i, _f, _p, _p, _i, _p, _i64, _p],
     "b2_gemm_static_scratch": [_p, _i64, _p, _i64, _p, _p, _i64, _i, _i, _i, _p],
     "b2_rowpar_fused": [_p, _p, _i64, _p, _i64, _p, _i, _i, _i, _p, _p, _f, _p, _p, _p],
     "b2_ctx_set_option": [_p, _i, _i64],
@@ -79,6 +87,7 @@ SIGNATURES = {
     "b2_embed": [_p, _p, _p, _i64, _i64, _i, _i, _p, _p],
     "b2_lm_head": [_p, _p, _i64, _p, _p, _i64, _i, _i, _i, C.POINTER(_p), _p],
     "b2_lm_head_sample": [_p, _p, _i64, _p, _p, _i64, _i, _i, _i, _p, C.c_uint64, _p, _p],
+    "b2_lm_head_sample_capped": [_p, _p, _i64, _p, _p, _i64, _i, _i, _i, _f, _f, _p, C.c_uint64, _p, _p],
     "b2_sampler_noise_bits": [C.c_uint64, C.c_uint32, C.c_uint32, C.c_uint32, C.POINTER(C.c_uint32)],
     "b2_philox4x32_10": [C.POINTER(C.c_uint32), C.POINTER(C.c_uint32), C.POINTER(C.c_uint32)],
     "b2_silu_and_mul": [_p, _i64, _i, _i, _p, _p],
@@ -101,7 +110,8 @@ for _name, _args in SIGNATURES.items():
     _fn = getattr(lib, _name)
     _fn.argtypes = _args
     _fn.restype = _i
-for _name, _args in {"b2_attention_workspace": [_i] * 10, "b2_linear_attn_workspace": [_i] * 7}.items():
+WORKSPACES = {"b2_attention_workspace": [_i] * 10, "b2_linear_attn_workspace": [_i] * 7, "b2_latent_attention_workspace": [_i] * 7}
+for _name, _args in WORKSPACES.items():
     _fn = getattr(lib, _name)
     _fn.argtypes = _args
     _fn.restype = _i64
@@ -110,7 +120,7 @@ lib.b2_last_error.argtypes = []
 lib.b2_launch_count.restype = _i64
 lib.b2_launch_count.argtypes = []
 
-EXPORTED = list(SIGNATURES) + ["b2_attention_workspace", "b2_linear_attn_workspace", "b2_last_error", "b2_launch_count"]
+EXPORTED = list(SIGNATURES) + list(WORKSPACES) + ["b2_last_error", "b2_launch_count"]
 
 
 def check(rc: int, what: str) -> None:

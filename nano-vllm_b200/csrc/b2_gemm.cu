@@ -125,6 +125,7 @@ struct GemmArgs {
   unsigned long long* sample_keys;  // [M] best (score, vocab id) per token row, zero between calls
   const float* temperatures;        // [M], or null = greedy
   unsigned long long seed;
+  float logit_scale, logit_cap;     // applied to the logit before the temperature; cap <= 0 = none
   int vocab_offset;                 // vocabulary id of feature 0 (rank * vocab / world)
 };
 
@@ -470,7 +471,11 @@ __device__ __forceinline__ void sample_feature_lanes(const GemmArgs& a, float (&
     for (int i = 0; i < 4; ++i) {
       const int token = token0 + j0 + i;
       float z = b2::bf16_round(v[j0 + i] + bias);  // the logit as the unfused path stores it
-      if (a.temperatures != nullptr && token < a.M) z = z / __ldg(a.temperatures + token) + gumbel_from_bits(r[i]);
+      if (a.temperatures != nullptr && token < a.M) {
+        if (a.logit_scale != 1.0f) z *= a.logit_scale;  // scale and cap keep the order, so a greedy pick needs neither
+        if (a.logit_cap > 0.f) z = a.logit_cap * tanhf(z / a.logit_cap);
+        z = z / __ldg(a.temperatures + token) + gumbel_from_bits(r[i]);
+      }
       k[j0 + i] = (live && token < a.M) ? sample_key(__float_as_uint(z), vocab_id) : 0ull;
     }
   }
@@ -2076,7 +2081,12 @@ int b2_lm_head(b2_ctx* ctx, const void* h, int64_t ldh, const int32_t* row_index
 
 int b2_lm_head_sample(b2_ctx* ctx, const void* h, int64_t ldh, const int32_t* row_index, const void* W, int64_t ldw, int B, int Vr,
                       int H, const float* temperatures, uint64_t seed, int64_t* tokens_out, void* stream) {
-  if (ctx == nullptr) return B2_ERR_ARG;
+  return b2_lm_head_sample_capped(ctx, h, ldh, row_index, W, ldw, B, Vr, H, 1.0f, 0.0f, temperatures, seed, tokens_out, stream);
+}
+
+int b2_lm_head_sample_capped(b2_ctx* ctx, const void* h, int64_t ldh, const int32_t* row_index, const void* W, int64_t ldw, int B, int Vr,
+                             int H, float logit_scale, float logit_cap, const float* temperatures, uint64_t seed, int64_t* tokens_out, void* stream) {
+  if (ctx == nullptr || !(logit_scale > 0.f)) return B2_ERR_ARG;
   int rc = check_operands(h, ldh, W, ldw, B, Vr, H);
   if (rc != B2_OK) return rc;
   const int world = ctx->cfg.world, rank = ctx->cfg.rank;
@@ -2101,6 +2111,8 @@ int b2_lm_head_sample(b2_ctx* ctx, const void* h, int64_t ldh, const int32_t* ro
   args.sample_keys = ctx->sample_keys;
   args.temperatures = temperatures;
   args.seed = seed;
+  args.logit_scale = logit_scale;
+  args.logit_cap = logit_cap;
   args.vocab_offset = rank * Vr;
   args.dstate = ctx->dstate;
   rc = launch_gemm<EPI_SAMPLE>(ctx, A, lda, W, ldw, B, Vr, H, args, 0, s);

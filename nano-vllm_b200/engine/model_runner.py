@@ -93,6 +93,8 @@ class ModelRunner:
             else:
                 random_init_(self.model, seed, self.rank)
             self.sampler = Sampler()
+            if hasattr(self.model, "bind_positions"):
+                self.model.bind_positions(max_model_len)  # rotation tables for every position a sequence can reach
             self._allocate_kv_cache(num_kvcache_blocks, gpu_memory_utilization)
             self.graphs: dict[int, torch.cuda.CUDAGraph] = {}
             if not enforce_eager:
@@ -115,7 +117,7 @@ class ModelRunner:
         kv, states = self.model.kv_layers(), self.model.state_layers()
         self.num_state_slots = self.max_num_seqs if states else 0
         for s in states:
-            s.state = torch.zeros(self.num_state_slots, *s.shape, dtype=torch.float32, device=self.device)
+            s.state = torch.zeros(self.num_state_slots, *s.shape, dtype=s.dtype or self.dtype, device=self.device)
         itemsize = torch.tensor([], dtype=self.dtype).element_size()
         block_bytes = sum(self.block_size * l.num_kv_heads * (l.k_dim + l.v_dim) for l in kv) * itemsize
         if num_blocks is None:
@@ -172,7 +174,7 @@ class ModelRunner:
         kv_len = self._h2d([b - a for a, b in zip(cu_k[:-1], cu_k[1:])], torch.int32) if paged else None
         ids_t, pos_t = self._h2d(ids, torch.int64), self._h2d(pos, torch.int64)
         set_context(True, self._h2d(cu_q, torch.int32), self._h2d(cu_k, torch.int32), max_q, max_k,
-                    self._h2d(slots, torch.int32) if slots else None, kv_len, block_tables, self._state_slots(seqs))
+                    self._h2d(slots, torch.int32) if slots else None, kv_len, block_tables, self._state_slots(seqs), cu_k[-1])
         return ids_t, pos_t
 
     def prepare_decode(self, seqs: list[Seq]):

@@ -55,9 +55,8 @@ class ParallelLMHead(VocabParallelEmbedding):
         return ops.lm_head_sample(x, self.weight, ctx.last_token_index if ctx.is_prefill else None, temperatures, seed, out)
 
 
-class TiedEmbedding(nn.Module):
-    """One table [vocab, width] that serves as embedding (read by the first stream launch) and as LM head.  Stored padded
-    to multiples of 8 in both directions; the padded vocabulary entries never leave this class."""
+class PaddedTable(nn.Module):
+    """A table [vocab, width] stored padded with zeros to multiples of 8 in both directions."""
 
     def __init__(self, num_embeddings: int, embedding_dim: int):
         super().__init__()
@@ -65,20 +64,32 @@ class TiedEmbedding(nn.Module):
         self.weight = nn.Parameter(torch.zeros(pad8(num_embeddings), pad8(embedding_dim)), requires_grad=False)
         self.weight.weight_loader = self.weight_loader
 
-    @property
-    def fused_sampling(self) -> bool:
-        """The LM head fused with the sampler scans every stored entry, so it needs a vocabulary without padding."""
-        return self.weight.dtype == torch.bfloat16 and self.weight.shape[0] == self.num_embeddings
-
     def weight_loader(self, param: nn.Parameter, loaded_weight: torch.Tensor):
         param.data[:self.num_embeddings, :self.embedding_dim].copy_(loaded_weight)
 
+
+class PaddedLMHead(PaddedTable):
+    """LM head over a padded table; the padded vocabulary entries never leave this class.  The logits are
+    cap tanh(scale W x / cap), or scale W x without a cap."""
+
+    def __init__(self, num_embeddings: int, embedding_dim: int, scale: float = 1.0, cap: float = 0.0):
+        super().__init__(num_embeddings, embedding_dim)
+        self.scale, self.cap = scale, cap
+
+    @property
+    def fused_sampling(self) -> bool:
+        """The LM head fused with the sampler scans every stored entry, so it needs a vocabulary without padding."""
+        return self.weight.dtype == torch.bfloat16 and self.weight.shape[0] == self.num_embeddings and self.scale > 0
+
     def logits(self, x: torch.Tensor, rows: torch.Tensor | None) -> torch.Tensor:
-        """Logits of the rows of x picked by int32 `rows` (None: all).  bf16 results are a view of the runtime's buffer."""
+        """Logits of the rows of x picked by int32 `rows` (None: all).  Untransformed bf16 logits are a view of the runtime's
+        buffer; scaled or capped ones are fp32."""
         if x.dtype == torch.float32:
             y = ops.gemm(x if rows is None else x[rows.long()], self.weight)
         else:
             y = ops.lm_head(x, self.weight, rows)
+        if self.scale != 1.0 or self.cap > 0:
+            y = ops.logit_cap(y, self.scale, self.cap)
         return y[:, :self.num_embeddings]
 
     def head(self, x: torch.Tensor) -> torch.Tensor:
@@ -87,4 +98,8 @@ class TiedEmbedding(nn.Module):
 
     def head_sample(self, x: torch.Tensor, temperatures: torch.Tensor | None, seed: int, out: torch.Tensor | None = None):
         ctx = get_context()
-        return ops.lm_head_sample(x, self.weight, ctx.last_token_index if ctx.is_prefill else None, temperatures, seed, out)
+        return ops.lm_head_sample(x, self.weight, ctx.last_token_index if ctx.is_prefill else None, temperatures, seed, out, self.scale, self.cap)
+
+
+class TiedEmbedding(PaddedLMHead):
+    """One table that serves as embedding (read by the first stream launch) and as LM head."""

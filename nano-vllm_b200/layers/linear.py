@@ -195,21 +195,27 @@ def pad8(n: int) -> int:
 
 class HeadsLinear(nn.Module):
     """Several head-structured projections of one input, stacked along the output dimension: section (heads, dim)
-    takes heads * pad8(dim) rows, the rows that pad a head are zero.  The first `silu_sections` sections leave the
-    product activated.  A checkpoint tensor [heads * dim, in] is loaded by section number."""
+    takes heads * pad8(dim) rows, the rows that pad a head are zero.  dim may be a tuple of parts, each padded on its own.
+    The first `silu_sections` sections leave the product activated.  A checkpoint tensor [heads * dim, in] is loaded by
+    section number."""
 
-    def __init__(self, input_size: int, sections: list[tuple[int, int]], silu_sections: int = 0):
+    def __init__(self, input_size: int, sections: list[tuple], silu_sections: int = 0):
         super().__init__()
-        self.input_size, self.sections = input_size, list(sections)
-        self.widths = [h * pad8(d) for h, d in sections]
+        self.input_size = input_size
+        self.sections = [(h, d if isinstance(d, tuple) else (d,)) for h, d in sections]
+        self.widths = [h * sum(map(pad8, parts)) for h, parts in self.sections]
         self.silu_cols = sum(self.widths[:silu_sections])
         self.weight = nn.Parameter(torch.zeros(sum(self.widths), pad8(input_size)), requires_grad=False)
         self.weight.weight_loader = self.weight_loader
 
     def weight_loader(self, param: nn.Parameter, loaded_weight: torch.Tensor, shard_id: int):
-        heads, dim = self.sections[shard_id]
-        rows = param.data.narrow(0, sum(self.widths[:shard_id]), self.widths[shard_id])
-        rows.view(heads, pad8(dim), -1)[:, :dim, :self.input_size].copy_(loaded_weight.view(heads, dim, self.input_size))
+        heads, parts = self.sections[shard_id]
+        rows = param.data.narrow(0, sum(self.widths[:shard_id]), self.widths[shard_id]).view(heads, sum(map(pad8, parts)), -1)
+        loaded_weight = loaded_weight.view(heads, sum(parts), self.input_size)
+        src = dst = 0
+        for dim in parts:
+            rows[:, dst:dst + dim, :self.input_size].copy_(loaded_weight[:, src:src + dim])
+            src, dst = src + dim, dst + pad8(dim)
 
     def forward(self, x: torch.Tensor) -> torch.Tensor:
         return ops.gemm(x, self.weight, silu_cols=self.silu_cols)

@@ -7,16 +7,16 @@ from torch import nn
 from .. import ops
 from ..utils.context import get_context
 from .linear import HeadsLinear, MergeHeadsLinear, pad8
+from .state import SlotState
 
 DECAY_POWERS = 65  # decay^0 .. decay^64: one chunk of the prefill kernel
 
 
-class RecurrentState:
-    """One layer run's state [slots, heads, qk_pad, v_pad] in fp32, bound by the runner."""
+class RecurrentState(SlotState):
+    """One layer run's state [slots, heads, qk_pad, v_pad] in fp32."""
 
     def __init__(self, heads: int, qk_pad: int, v_pad: int):
-        self.shape = (heads, qk_pad, v_pad)
-        self.state: torch.Tensor | None = None
+        super().__init__((heads, qk_pad, v_pad), torch.float32)
 
 
 class DecayedLinearAttention(nn.Module):

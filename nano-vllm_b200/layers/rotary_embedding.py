@@ -46,3 +46,28 @@ class RotaryEmbedding(nn.Module):
 @lru_cache(1)
 def get_rope(head_size: int, rotary_dim: int, max_position: int, base: float) -> RotaryEmbedding:
     return RotaryEmbedding(head_size, rotary_dim, max_position, base)
+
+
+class PairRotation:
+    """Rotation of adjacent pairs: (u, v) = elements 2i and 2i + 1 of a part of `dim` elements turn by position * base^(-2i / dims),
+    i < dims / 2; the other pairs stay as they are.  `table` fp32 [positions, pad8(dim) / 2, 2] holds (cos, sin), the angles
+    taken in fp64; bind() builds it, shared by all rotations of the same kind on a device."""
+    _tables: dict = {}
+
+    def __init__(self, dim: int, dims: int, base: float) -> None:
+        if dims % 2 or not 0 <= dims <= dim:
+            raise ValueError(f"{dims} rotated of {dim} elements")
+        self.dim, self.dims, self.base = dim, dims, float(base)
+        self.pairs = (dim + 7) // 8 * 4
+        self.table: torch.Tensor | None = None
+
+    def bind(self, positions: int, device) -> None:
+        key = (self.pairs, self.dims, self.base, positions, torch.device(device))
+        if key not in self._tables:
+            i = torch.arange(self.dims // 2, dtype=torch.float64, device="cpu")
+            angles = torch.outer(torch.arange(positions, dtype=torch.float64, device="cpu"), self.base ** (-2.0 * i / max(self.dims, 1)))
+            table = torch.zeros(positions, self.pairs, 2, dtype=torch.float32, device="cpu")
+            table[..., 0] = 1.0
+            table[:, :self.dims // 2, 0], table[:, :self.dims // 2, 1] = angles.cos().float(), angles.sin().float()
+            self._tables[key] = table.to(device)
+        self.table = self._tables[key]

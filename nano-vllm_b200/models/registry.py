@@ -5,6 +5,7 @@ import json
 import os
 from dataclasses import dataclass, fields
 
+from .mupulorn import MupulornConfig, MupulornForCausalLM
 from .qwen3 import Qwen3ForCausalLM
 from .vekerax import VekeraxConfig, VekeraxForCausalLM
 
@@ -48,6 +49,7 @@ class ModelConfig:
 REGISTRY = {
     "Qwen3ForCausalLM": (ModelConfig, Qwen3ForCausalLM),
     "Vekerax": (VekeraxConfig, VekeraxForCausalLM),
+    "Mupulorn": (MupulornConfig, MupulornForCausalLM),
 }
 
 

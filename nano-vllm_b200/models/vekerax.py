@@ -23,6 +23,7 @@ from ..layers.embed_head import TiedEmbedding
 from ..layers.linear import MergedColumnParallelLinear, MergeHeadsLinear, _tp_rank_world, pad8
 from ..layers.linear_attention import DecayedLinearAttention, RecurrentState
 from ..layers.streams import StreamConnection, StreamNorm
+from ..utils.loader import load_exactly
 
 
 @dataclass
@@ -237,16 +238,7 @@ class VekeraxForCausalLM(nn.Module):
         return put(mixer.norm_weight) if leaf == "norm" else put(mixer.in_proj.weight, "qkvg".index(leaf))
 
     def load_full_weights(self, weights) -> None:
-        """Every tensor of a checkpoint, by name; names and shapes must be exactly this configuration's."""
-        want = self.weight_shapes()
-        missing, extra = sorted(set(want) - set(weights)), sorted(set(weights) - set(want))
-        if missing or extra:
-            raise ValueError(f"checkpoint does not fit the configuration: missing {missing[:4]}, unexpected {extra[:4]}")
-        for name in want:
-            w = weights[name]
-            if tuple(w.shape) != want[name]:
-                raise ValueError(f"{name}: shape {tuple(w.shape)}, expected {want[name]}")
-            self.load_weight(name, w)
+        load_exactly(self, weights)
 
     def random_init_(self, seed: int) -> None:
         """Seeded weights generated on the device: N(0, 0.02) matrices, unit norms, streams that stay alike in size."""

@@ -302,9 +302,10 @@ def lm_head(h: torch.Tensor, w: torch.Tensor, row_index: torch.Tensor | None):
 
 
 def lm_head_sample(h: torch.Tensor, w: torch.Tensor, row_index: torch.Tensor | None, temperatures: torch.Tensor | None,
-                   seed: int, out: torch.Tensor | None = None) -> torch.Tensor:
+                   seed: int, out: torch.Tensor | None = None, scale: float = 1.0, cap: float = 0.0) -> torch.Tensor:
     """LM head and sampler in one pass over the vocabulary shard (no logits in memory).  Returns int64 token ids
-    [B], valid on rank 0 only.  temperatures: fp32 [B] on the device, or None for greedy decoding."""
+    [B], valid on rank 0 only.  temperatures: fp32 [B] on the device, or None for greedy decoding.  The sampled logits are
+    cap tanh(scale logit / cap) (cap 0: scale logit)."""
     rt = get_runtime()
     h2 = _as2d(_bf16_rows(h, "lm_head input"))
     if h2.stride(0) % 8 != 0 or h2.data_ptr() % 16 != 0:
@@ -318,9 +319,10 @@ def lm_head_sample(h: torch.Tensor, w: torch.Tensor, row_index: torch.Tensor | N
         out = torch.empty(B, dtype=torch.int64, device=h.device)
     assert out.dtype == torch.int64 and out.is_cuda and out.numel() >= B
     Vr, H = w.shape
-    _abi.check(_lib.b2_lm_head_sample(rt.ctx, h2.data_ptr(), h2.stride(0), row_index.data_ptr() if row_index is not None else None,
-                                      w.data_ptr(), w.stride(0), B, Vr, H, temperatures.data_ptr() if temperatures is not None else None,
-                                      int(seed) & 0xFFFFFFFFFFFFFFFF, out.data_ptr(), _stream()), "b2_lm_head_sample")
+    _abi.check(_lib.b2_lm_head_sample_capped(rt.ctx, h2.data_ptr(), h2.stride(0), row_index.data_ptr() if row_index is not None else None,
+                                             w.data_ptr(), w.stride(0), B, Vr, H, float(scale), float(cap),
+                                             temperatures.data_ptr() if temperatures is not None else None,
+                                             int(seed) & 0xFFFFFFFFFFFFFFFF, out.data_ptr(), _stream()), "b2_lm_head_sample")
     return out[:B]
 
 
@@ -416,6 +418,132 @@ def gated_norm(o: torch.Tensor, gate: torch.Tensor, w: torch.Tensor, eps: float,
     out = torch.empty(M, pad, dtype=gate.dtype, device=o.device)
     _abi.check(_lib.b2_gated_norm(_dt(gate), o.data_ptr(), o.stride(0), gate.data_ptr(), gate.stride(0), w.data_ptr(), float(eps), M, dim, pad,
                                   out.data_ptr(), out.stride(0), _stream()), "b2_gated_norm")
+    return out
+
+
+def sandwich_step(x: torch.Tensor | None, y: torch.Tensor | None, post_w, norm_w: torch.Tensor, eps: float, dim: int, batch, conv_w=None, state=None,
+                  store: bool = True, embed: tuple | None = None, run: int = 0) -> tuple[torch.Tensor | None, torch.Tensor]:
+    """Everything between two sublayers: x <- x + post_w y / rms(y) (fp32 x [M, D]; embed = (ids, table): x = table[ids]),
+    h = norm_w x / rms(x), out = h + causal convolution of h.  batch = (cu_q or None, kv_len, state slots, max_q).  Returns
+    (new x or None when store is False, out)."""
+    if embed is not None:
+        ids, table = embed
+        M, D, dtype, dev = ids.numel(), table.shape[1], table.dtype, table.device
+    else:
+        ids = table = None
+        (M, D), dtype, dev = x.shape, y.dtype, x.device
+        assert x.dtype == torch.float32 and x.is_contiguous() and y.shape == (M, D) and y.stride(1) == 1
+        assert post_w.dtype == torch.float32 and post_w.numel() in (1, D)
+    assert norm_w.dtype == torch.float32 and norm_w.numel() in (1, D)
+    cu_q, kv_len, slots, max_q = batch
+    taps = 0
+    if conv_w is not None:
+        taps = conv_w.shape[0]
+        assert conv_w.shape == (taps, D) and conv_w.is_contiguous() and conv_w.dtype == dtype and state.dtype == dtype and state.is_contiguous()
+        assert state.shape[1:] == (taps - 1, D) and slots.dtype == torch.int32 and kv_len.dtype == torch.int32
+        B = kv_len.numel() if cu_q is None else cu_q.numel() - 1
+    else:  # no neighbours: every row is on its own
+        cu_q, B, max_q = None, M, 1
+    x_out = torch.empty(M, D, dtype=torch.float32, device=dev) if store else None
+    out = torch.empty(M, D, dtype=dtype, device=dev)
+    _abi.check(_lib.b2_sandwich_step(_dt(out), _ptr(x) if embed is None else None, _ptr(x_out), _ptr(ids), _ptr(table),
+                                     table.stride(0) if table is not None else 0, table.shape[0] if table is not None else 0, _ptr(y),
+                                     y.stride(0) if y is not None else 0, _ptr(post_w), post_w.numel() if post_w is not None else 0, norm_w.data_ptr(),
+                                     norm_w.numel(), float(eps), _ptr(conv_w), taps, _ptr(state), _ptr(slots), _ptr(cu_q), _ptr(kv_len), B, max_q,
+                                     out.data_ptr(), D, dim, D, run, _stream()), "b2_sandwich_step")
+    return x_out, out
+
+
+def poly_norm(z: torch.Tensor, coef: torch.Tensor, eps: float, dim: int) -> torch.Tensor:
+    """a N(z) + b N(z^2) + c N(z^3) + e with coef = (a, b, c, e) in fp32; N divides a row by its root mean square."""
+    M, D = z.shape
+    assert z.stride(1) == 1 and coef.dtype == torch.float32 and coef.numel() == 4
+    out = torch.empty(M, D, dtype=z.dtype, device=z.device)
+    _abi.check(_lib.b2_poly_norm(_dt(z), z.data_ptr(), z.stride(0), coef.data_ptr(), float(eps), M, dim, D, out.data_ptr(), D, _stream()), "b2_poly_norm")
+    return out
+
+
+def logit_cap(x: torch.Tensor, scale: float, cap: float) -> torch.Tensor:
+    """fp32 cap tanh(scale x / cap); cap 0: scale x."""
+    M, V = x.shape
+    assert x.stride(1) == 1
+    out = torch.empty(M, V, dtype=torch.float32, device=x.device)
+    _abi.check(_lib.b2_logit_cap(_dt(x), x.data_ptr(), x.stride(0), float(scale), float(cap), M, V, out.data_ptr(), V, _stream()), "b2_logit_cap")
+    return out
+
+
+def latent_store(rows: torch.Tensor, q_dim: int, q_pad: int, kv_dim: int, kv_pad: int, rot_pad: int, q_norm, kv_norm, eps: float, positions: torch.Tensor,
+                 cos_sin: torch.Tensor, cache, slot_mapping) -> None:
+    """In place on rows [query latent | latent | rotated part | ...]: norms and rotation; the last two also to the cache."""
+    assert rows.dim() == 2 and rows.stride(1) == 1 and positions.dtype == torch.int64
+    assert cos_sin.dtype == torch.float32 and cos_sin.is_contiguous() and cos_sin.shape[1:] == (rot_pad // 2, 2)
+    have = cache is not None and cache.numel() > 0
+    if have:
+        assert cache.dtype == rows.dtype and cache.is_contiguous() and cache.shape[-1] == kv_pad + rot_pad and slot_mapping.dtype == torch.int32
+    _abi.check(_lib.b2_latent_store(_dt(rows), rows.data_ptr(), rows.stride(0), rows.shape[0], q_dim, q_pad, kv_dim, kv_pad, rot_pad, _ptr(q_norm),
+                                    kv_norm.data_ptr(), float(eps), positions.data_ptr(), cos_sin.data_ptr(), cos_sin.shape[0],
+                                    _ptr(cache) if have else None, _ptr(slot_mapping) if have else None, _stream()), "b2_latent_store")
+
+
+def latent_gather(cache: torch.Tensor, block_tables: torch.Tensor, cu_k: torch.Tensor, max_kv: int, total: int) -> torch.Tensor:
+    """The cached rows of every sequence, contiguous [total, row]; cache [blocks, block_size, 1, row]."""
+    row = cache.shape[-1]
+    assert cache.is_contiguous() and block_tables.dtype == torch.int32 and cu_k.dtype == torch.int32
+    out = torch.empty(total, row, dtype=cache.dtype, device=cache.device)
+    _abi.check(_lib.b2_latent_gather(_dt(cache), cache.data_ptr(), block_tables.data_ptr(), block_tables.stride(0), cache.shape[1], cu_k.data_ptr(),
+                                     cu_k.numel() - 1, max_kv, row, out.data_ptr(), _stream()), "b2_latent_gather")
+    return out
+
+
+def heads_gemm(x: torch.Tensor, x_head: int, w: torch.Tensor, kn: bool, out_head: int, gate: torch.Tensor | None = None, gate_head: int = 0,
+               rotate: tuple | None = None) -> torch.Tensor:
+    """One product per head: w [heads, N, K] (kn: [heads, K, N]; may be a view); x [M, heads * x_head], returns
+    [M, heads * out_head].  rotate = (rot_pad, positions, cos_sin): the elements behind a head's K inputs, rotated, go behind
+    its N outputs."""
+    heads, N, K = w.shape[0], w.shape[2 if kn else 1], w.shape[1 if kn else 2]
+    M = x.shape[0]
+    rot_pad, positions, cos_sin = rotate if rotate is not None else (0, None, None)
+    assert x.stride(1) == 1 and x.dtype == w.dtype and w.stride(2) == 1 and x.shape[1] >= heads * x_head
+    assert gate is None or (gate.dtype == x.dtype and gate.stride(1) == 1 and gate.shape[0] == M)
+    out = torch.empty(M, heads * out_head, dtype=x.dtype, device=x.device)
+    _abi.check(_lib.b2_heads_gemm(_dt(x), x.data_ptr(), x.stride(0), x_head, w.data_ptr(), w.stride(1), w.stride(0), int(kn), out.data_ptr(), out.stride(0),
+                                  out_head, M, heads, N, K, _ptr(gate), gate.stride(0) if gate is not None else 0, gate_head, rot_pad, _ptr(positions),
+                                  _ptr(cos_sin), cos_sin.shape[0] if cos_sin is not None else 0, _stream()), "b2_heads_gemm")
+    return out
+
+
+def latent_attention(q: torch.Tensor, heads: int, cache: torch.Tensor, lat_pad: int, block_tables: torch.Tensor, cu_q, kv_len: torch.Tensor, max_q: int,
+                     max_kv: int, scale: float, sink, form: int = 0) -> torch.Tensor:
+    """Absorbed attention of q [M, heads * row] over cached rows [blocks, block_size, 1, row]; cu_q None = decode.  Returns the
+    mixed latents [M, heads * lat_pad]."""
+    row = cache.shape[-1]
+    M, B = q.shape[0], kv_len.numel() if cu_q is None else cu_q.numel() - 1
+    assert q.stride(1) == 1 and q.dtype == cache.dtype and cache.is_contiguous() and q.shape[1] >= heads * row
+    assert block_tables.dtype == torch.int32 and kv_len.dtype == torch.int32 and (sink is None or sink.dtype == torch.float32)
+    out = torch.empty(M, heads * lat_pad, dtype=q.dtype, device=q.device)
+    max_kv = min(max_kv, block_tables.shape[1] * cache.shape[1])
+    nbytes = _lib.b2_latent_attention_workspace(_dt(q), B, max_q, max_kv, heads, lat_pad, row - lat_pad)
+    ws = _workspace("latent_attention", nbytes, q.device)
+    _abi.check(_lib.b2_latent_attention(_dt(q), q.data_ptr(), q.stride(0), out.data_ptr(), out.stride(0), cache.data_ptr(), block_tables.data_ptr(),
+                                        block_tables.stride(0), cache.shape[1], _ptr(cu_q), kv_len.data_ptr(), B, max_q, max_kv, heads, lat_pad,
+                                        row - lat_pad, float(scale), _ptr(sink), _ptr(ws), ws.numel() if ws is not None else 0, form, _stream()),
+               "b2_latent_attention")
+    return out
+
+
+def expanded_attention(q: torch.Tensor, heads: int, kv: torch.Tensor, rot: torch.Tensor, cu_q: torch.Tensor, cu_k: torch.Tensor, max_q: int, dim_pad: int,
+                       rot_pad: int, v_pad: int, scale: float, sink, cos_sin: torch.Tensor, gate: torch.Tensor | None) -> torch.Tensor:
+    """Attention of the unrotated q [M, heads * (dim_pad + rot_pad)] over contiguous rows kv [keys, heads * (dim_pad + v_pad)]
+    and rot [keys, rot_pad]; the output is multiplied by sigmoid(gate)."""
+    M = q.shape[0]
+    assert q.dtype == kv.dtype == rot.dtype == torch.bfloat16 and q.stride(1) == kv.stride(1) == rot.stride(1) == 1
+    assert cu_q.dtype == cu_k.dtype == torch.int32 and cos_sin.is_contiguous() and (sink is None or sink.dtype == torch.float32)
+    assert gate is None or (gate.dtype == q.dtype and gate.stride(1) == 1)
+    out = torch.empty(M, heads * v_pad, dtype=q.dtype, device=q.device)
+    _abi.check(_lib.b2_expanded_attention(q.data_ptr(), q.stride(0), out.data_ptr(), out.stride(0), kv.data_ptr(), kv.stride(0), rot.data_ptr(),
+                                          rot.stride(0), cu_q.data_ptr(), cu_k.data_ptr(), cu_q.numel() - 1, max_q, heads, dim_pad, rot_pad, v_pad,
+                                          float(scale), _ptr(sink), cos_sin.data_ptr(), cos_sin.shape[0], _ptr(gate),
+                                          gate.stride(0) if gate is not None else 0, _stream()), "b2_expanded_attention")
     return out
 
 

@@ -58,3 +58,17 @@ class Checkpoint(Mapping):
 
     def __len__(self):
         return len(self._where)
+
+
+def load_exactly(model, weights: Mapping) -> None:
+    """Every tensor of a checkpoint into model.load_weight(name, tensor); names and shapes must be exactly those of
+    model.weight_shapes()."""
+    want = model.weight_shapes()
+    missing, extra = sorted(set(want) - set(weights)), sorted(set(weights) - set(want))
+    if missing or extra:
+        raise ValueError(f"checkpoint does not fit the configuration: missing {missing[:4]}, unexpected {extra[:4]}")
+    for name in want:
+        w = weights[name]
+        if tuple(w.shape) != want[name]:
+            raise ValueError(f"{name}: shape {tuple(w.shape)}, expected {want[name]}")
+        model.load_weight(name, w)
