@@ -1,4 +1,4 @@
-"""The other workloads, behind `bench.py --workload cfg2|cfg5|vekerax` (the JSON line of the default workload).
+"""The other workloads, behind `bench.py --workload cfg2|cfg5|vekerax|mupulorn` (the JSON line of the default workload).
 
 cfg2  the reference's own bench.py workload (bench.py:9-27): Qwen3-0.6B random-init bf16 on one GPU, 256 sequences,
       prompt ids uniform in [0, 10000], prompt and output lengths uniform in [100, 1024], temperature 0.6, ignore_eos;
@@ -263,6 +263,27 @@ def _model_throughput(torch, cfg: dict, vocab: int, batch: int, prompt: int, ste
     return out
 
 
+class KernelTable:
+    """Rows (kernel, microseconds, fraction of the roofline) beside the like kernel of another model.  Rooflines: the measured
+    copy bandwidth or burst bf16 throughput, or (bound "sum") seconds the caller has added up from both."""
+
+    def __init__(self, peaks: dict):
+        self.peaks, self.rows = peaks, []
+
+    def roof_us(self, work, bound) -> float:
+        return work * 1e6 if bound == "sum" else work / (self.peaks["hbm_gbs"] * 1e9 if bound == "hbm" else self.peaks["bf16_tflops"] * 1e12) * 1e6
+
+    def add(self, name, like, work, us, like_work, like_us, bound, like_bound=None):
+        f, g = self.roof_us(work, bound) / us, self.roof_us(like_work, like_bound or bound) / like_us
+        self.rows.append({"kernel": name, "us": round(us, 2), "bound": bound, "frac": round(f, 3), "like": like, "like_us": round(like_us, 2),
+                          "like_frac": round(g, 3), "like_over_this": round(g / f, 2)})
+
+    @staticmethod
+    def variants(make, nbytes):
+        """Enough copies of an input that a round through them exceeds L2."""
+        return [make() for _ in range(max(2, min(48, int(4e8 / nbytes) + 1)))]
+
+
 def _kernel_table(torch, z: dict, peaks: dict, batch: int, ctx_len: int) -> list[dict]:
     """Microseconds and fraction of the roofline (measured copy bandwidth or burst bf16 throughput) of every kernel of the
     design at this layer size, each next to the like kernel of Qwen3 on the same sizes.  Inputs rotate through more than L2."""
@@ -271,16 +292,8 @@ def _kernel_table(torch, z: dict, peaks: dict, batch: int, ctx_len: int) -> list
     from nanovllm_b200.rowpar_microbench import time_in_graph
     dev, bf, W, S = "cuda", torch.bfloat16, z["width"], VEKERAX_STREAMS
     H, G, d, ff, win, keep = z["heads"], z["kv_heads"], z["dim"], z["ff"], VEKERAX_WINDOW, VEKERAX_KEEP
-    rows = []
-
-    def add(name, like, work, us, like_work, like_us, bound):
-        peak = peaks["hbm_gbs"] * 1e9 if bound == "hbm" else peaks["bf16_tflops"] * 1e12
-        f, g = work / (us * 1e-6) / peak, like_work / (like_us * 1e-6) / peak
-        rows.append({"kernel": name, "us": round(us, 2), "bound": bound, "frac": round(f, 3), "like": like, "like_us": round(like_us, 2),
-                     "like_frac": round(g, 3), "like_over_this": round(g / f, 2)})
-
-    def variants(make, nbytes):
-        return [make() for _ in range(max(2, min(48, int(4e8 / nbytes) + 1)))]
+    table = KernelTable(peaks)
+    rows, add, variants = table.rows, table.add, table.variants
 
     for M in (batch, 8192):
         # residual: streams against add + RMSNorm
@@ -427,5 +440,187 @@ def run_vekerax(args, peaks, clock_sampler_cls) -> None:
                       "config": {"workload": f"Vekerax and Qwen3 with the same layer sizes, random weights; {VEKERAX_STREAMS} streams, window {VEKERAX_WINDOW} + {VEKERAX_KEEP}, "
                                              "attention and lightning layers in turn; value: width 4096, batch 64, 1024-token prompts, device-resident decode",
                                  "l2": "weights, caches and rotated kernel inputs exceed the 126 MB L2"},
+                      "clocks": clocks.summary(), "gpu_launches": _abi.launch_count(), "sizes": sizes}), flush=True)
+    dist.destroy_process_group()
+
+
+# ---------------------------------------------------------------------------------------------------------------------
+# mupulorn
+# ---------------------------------------------------------------------------------------------------------------------
+# the layer sizes above with latents; its feed-forward has two matrices instead of three, so ff is 1.5 times as wide
+MUPULORN_SIZES = {
+    "width1024": dict(VEKERAX_SIZES["width1024"], q_rank=512, kv_rank=256, rot_dim=64),
+    "width4096": dict(VEKERAX_SIZES["width4096"], q_rank=1536, kv_rank=512, rot_dim=64),
+}
+MUPULORN_TAPS = 4
+
+
+def _mupulorn_config(z: dict) -> dict:
+    mixer = {"heads": z["heads"], "dim": z["dim"], "rot_dim": z["rot_dim"], "vdim": z["dim"], "q_rank": z["q_rank"], "kv_rank": z["kv_rank"],
+             "scale": (z["dim"] + z["rot_dim"]) ** -0.5, "rot": {"base": 10000.0, "dims": z["rot_dim"]}}
+    layer = {"type": "latent_attention", "mixer": mixer, "mlp": {"kind": "dense", "ff": z["ff"] * 3 // 2}}
+    return {"architecture": "Mupulorn", "canon": {"taps": MUPULORN_TAPS}, "layers": [layer] * z["layers"], "logit_scale": 0.5, "logit_softcap": 30.0,
+            "norm": {"eps": 1e-6}, "vocab": z["vocab"], "width": z["width"]}
+
+
+def _mupulorn_kernels(torch, z: dict, peaks: dict, batch: int, ctx_len: int) -> list[dict]:
+    """Every kernel of the design at this layer size next to the like kernel of Qwen3."""
+    from flash_attn import flash_attn_varlen_func, flash_attn_with_kvcache
+    from nanovllm_b200 import ops
+    from nanovllm_b200.layers.rotary_embedding import PairRotation
+    from nanovllm_b200.rowpar_microbench import time_in_graph
+    dev, bf, W, taps = "cuda", torch.bfloat16, z["width"], MUPULORN_TAPS
+    H, G, d, rot, L, Q, ff = z["heads"], z["kv_heads"], z["dim"], z["rot_dim"], z["kv_rank"], z["q_rank"], z["ff"] * 3 // 2
+    row, qh = L + rot, d + rot
+    table = KernelTable(peaks)
+    add, variants = table.add, table.variants
+    hbm, tensor = peaks["hbm_gbs"] * 1e9, peaks["bf16_tflops"] * 1e12
+    rnd = lambda *s, k=1.0: (torch.randn(*s, device=dev) * k).to(bf)
+    rope = PairRotation(rot, rot, 10000.0)
+    rope.bind(8192, dev)
+    one = torch.ones(1, device=dev)
+    conv = rnd(taps, W, k=0.1)
+    nwb = torch.ones(W, device=dev, dtype=bf)
+
+    for M in (batch, 8192):
+        seqs = batch if M == batch else 4
+        slots = torch.arange(seqs, device=dev, dtype=torch.int32)
+        lens = torch.full((seqs,), 1024 if M == batch else M // seqs, device=dev, dtype=torch.int32)
+        cu = None if M == batch else torch.arange(0, M + 1, M // seqs, device=dev, dtype=torch.int32)
+        per = 1 if M == batch else M // seqs
+        cuts = (cu, lens, slots, per)
+        states = [torch.zeros(seqs, taps - 1, W, device=dev, dtype=bf) for _ in range(8)]
+        step = lambda x, y, i: ops.sandwich_step(x, y, one, one, 1e-6, W, cuts, conv, states[i % 8])
+        # residual: x read and written in fp32, y in, h out (and the states of decoded rows)
+        nb = M * W * (8 + 4) + (2 * (taps - 1) * seqs * W * 2)
+        vs = variants(lambda: (torch.randn(M, W, device=dev), rnd(M, W)), nb)
+        us = time_in_graph(lambda i: step(*vs[i], i), len(vs), 4 * len(vs))
+        nl = M * W * 8
+        ls = variants(lambda: (rnd(M, W), rnd(M, W)), nl)
+        lus = time_in_graph(lambda i: ops.add_rmsnorm(ls[i][0], ls[i][1], nwb, 1e-6), len(ls), 4 * len(ls))
+        add(f"sandwich_step M={M}", "add_rmsnorm", nb, us, nl, lus, "hbm")
+        del vs, ls
+        # PolyNorm (rows of ff) against RMSNorm (rows of the width)
+        nb = M * ff * 4
+        vs = variants(lambda: rnd(M, ff), nb)
+        coef = torch.full((4,), 0.3, device=dev)
+        us = time_in_graph(lambda i: ops.poly_norm(vs[i], coef, 1e-6, ff), len(vs), 4 * len(vs))
+        ls = variants(lambda: rnd(M, W), M * W * 4)
+        lus = time_in_graph(lambda i: ops.rmsnorm(ls[i], nwb, 1e-6), len(ls), 4 * len(ls))
+        add(f"poly_norm M={M}", "rmsnorm", nb, us, M * W * 4, lus, "hbm")
+        del vs, ls
+        # latent norms, rotation and scatter against head norm, rotation and scatter
+        N = Q + row + H * d
+        cache = torch.zeros(64, 256, 1, row, dtype=bf, device=dev)
+        sm = torch.randperm(64 * 256, device=dev)[:M].int()
+        pos = torch.arange(M, device=dev) % 2048
+        qw, kw = torch.ones(Q, device=dev), torch.ones(L, device=dev)
+        nb = M * (2 * Q * 2 + 3 * row * 2)
+        vs = variants(lambda: rnd(M, N), M * N * 2)
+        us = time_in_graph(lambda i: ops.latent_store(vs[i], Q, Q, L, L, rot, qw, kw, 1e-6, pos, rope.table, cache, sm), len(vs), 4 * len(vs))
+        del vs
+        kc = torch.zeros(64, 256, G, d, dtype=bf, device=dev)
+        vc, cs, hw = torch.zeros_like(kc), torch.randn(2048, d, device=dev), torch.ones(d, device=dev, dtype=bf)
+        nl = M * d * (4 * H + 10 * G)
+        ls = variants(lambda: rnd(M, (H + 2 * G) * d), nl)
+        lus = time_in_graph(lambda i: ops.qk_norm_rope_store(ls[i], H, G, d, hw, hw, 1e-6, pos, cs, kc, vc, sm), len(ls), 4 * len(ls))
+        add(f"latent_store M={M}", "qk_norm_rope_store", nb, us, nl, lus, "hbm")
+        del ls, kc, vc, cache
+        # o / down projection and what follows against the fused row-parallel block
+        for nm, K in (("o_proj", H * d), ("down_proj", ff)):
+            ws = [rnd(W, K, k=0.02) for _ in range(max(2, min(24, int(3e8 / (W * K * 2)) + 1)))]
+            x, r, xs = rnd(M, K), rnd(M, W), torch.randn(M, W, device=dev)
+            us = time_in_graph(lambda i: step(xs, ops.gemm(x, ws[i]), i), len(ws), 4 * len(ws))
+            lus = time_in_graph(lambda i: ops.rowpar_fused(x, ws[i], None, r, nwb, 1e-6), len(ws), 4 * len(ws))
+            if M > 1000:
+                roof, lroof = 2.0 * M * W * K / tensor + M * W * 12.0 / hbm, 2.0 * M * W * K / tensor + M * W * 8.0 / hbm
+            else:
+                roof, lroof = (2.0 * (W * K + M * K) + M * W * 24.0) / hbm, (2.0 * (W * K + M * K) + M * W * 8.0) / hbm
+            add(f"{nm} + sandwich_step M={M}", "rowpar_fused", roof, us, lroof, lus, "sum")
+            del ws, x, r, xs
+        # the design's other projections run on the same GEMM; a plain one of Qwen3's sizes beside them
+        def gemm_us(N, K):
+            ws = [rnd(N, K, k=0.02) for _ in range(max(2, min(24, int(3e8 / (N * K * 2)) + 1)))]
+            x = rnd(M, K)
+            return time_in_graph(lambda i: ops.gemm(x, ws[i]), len(ws), 4 * len(ws))
+        work = lambda N, K: 2.0 * M * N * K if M > 1000 else 2.0 * (N * K + M * K + M * N)
+        bound = "tensor" if M > 1000 else "hbm"
+        Nq = (H + 2 * G) * d
+        qkv_us = gemm_us(Nq, W)
+        for nm, N, K in (("in_proj", Q + row + H * d, W), ("q_proj", H * qh, Q), ("up_proj", ff, W)) + ((("kv_proj", H * 2 * d, L),) if M > 1000 else ()):
+            add(f"{nm} M={M}", "qkv projection GEMM", work(N, K), gemm_us(N, K), work(Nq, W), qkv_us, bound)
+        if M == batch:  # per-head products of the absorbed form
+            ws = [rnd(H, 2 * d, L, k=0.05) for _ in range(max(2, min(48, int(3e8 / (H * 2 * d * L * 2)) + 1)))]
+            q, o, gate = rnd(M, H * qh), rnd(M, H * L), rnd(M, H * d)
+            nb = 2.0 * (H * d * L + M * H * (qh + row))
+            us = time_in_graph(lambda i: ops.heads_gemm(q, qh, ws[i][:, :d], True, row, rotate=(rot, pos, rope.table)), len(ws), 4 * len(ws))
+            add(f"heads_gemm q Wk + rotation M={M}", "qkv projection GEMM", nb, us, work(Nq, W), qkv_us, "hbm")
+            nb = 2.0 * (H * d * L + M * H * (L + 2 * d))
+            us = time_in_graph(lambda i: ops.heads_gemm(o, L, ws[i][:, d:], False, d, gate=gate, gate_head=d), len(ws), 4 * len(ws))
+            add(f"heads_gemm Wv + gate M={M}", "qkv projection GEMM", nb, us, work(Nq, W), qkv_us, "hbm")
+            del ws
+    sink = torch.zeros(H, device=dev)
+    # prompts: 4 sequences of 2048, full causal
+    B, T = 4, 2048
+    M = B * T
+    cu = torch.arange(0, M + 1, T, device=dev, dtype=torch.int32)
+    q, kv, kr, gate = rnd(M, H * qh), rnd(M, H * 2 * d), rnd(M, rot), rnd(M, H * d)
+    pairs = B * T * (T + 1) / 2
+    us = time_in_graph(lambda i: ops.expanded_attention(q, H, kv, kr, cu, cu, T, d, rot, d, qh ** -0.5, sink, rope.table, gate), 4, 16)
+    fq, fk, fv = rnd(M, H, d), rnd(M, G, d), rnd(M, G, d)
+    lus = time_in_graph(lambda i: flash_attn_varlen_func(fq, fk, fv, cu, cu, T, T, softmax_scale=d ** -0.5, causal=True), 4, 16)
+    add(f"expanded_attention {B}x{T}", "flash-attn, full causal", 2.0 * H * (qh + d) * pairs, us, 4.0 * H * d * pairs, lus, "tensor")
+    # decoding, and a portion of 64 tokens (absorbed) against decoding / flash-attn on the cache
+    nblk = -(-ctx_len // 256)
+    layers = max(4, int(4e8 / (batch * nblk * 256 * row * 2)) + 1)
+    caches = [rnd(batch * nblk, 256, 1, row) for _ in range(layers)]
+    bt = torch.randperm(batch * nblk, device=dev).int().view(batch, nblk).contiguous()
+    kl = torch.full((batch,), ctx_len, dtype=torch.int32, device=dev)
+    q = rnd(batch, H * row)
+    us = time_in_graph(lambda i: ops.latent_attention(q, H, caches[i], L, bt, None, kl, 1, nblk * 256, qh ** -0.5, sink), layers, 10 * layers)
+    kcs = [rnd(batch * nblk, 256, G, d) for _ in range(4)]
+    vcs = [rnd(batch * nblk, 256, G, d) for _ in range(4)]
+    fq = rnd(batch, 1, H, d)
+    lus = time_in_graph(lambda i: flash_attn_with_kvcache(fq, kcs[i], vcs[i], cache_seqlens=kl, block_table=bt, softmax_scale=d ** -0.5, causal=True), 4, 40)
+    like = 2.0 * batch * ctx_len * G * d * 2
+    add(f"latent_attention decode {batch} x {ctx_len}", "flash-attn kvcache", 2.0 * batch * (ctx_len * row + H * (row + L)), us, like, lus, "hbm")
+    P = 64
+    cu = torch.tensor([0, P], device=dev, dtype=torch.int32)
+    big = bt.view(1, -1)
+    n = min(16384, batch * nblk * 256)
+    q, kl1 = rnd(P, H * row), torch.tensor([n], device=dev, dtype=torch.int32)
+    us = time_in_graph(lambda i: ops.latent_attention(q, H, caches[i], L, big, cu, kl1, P, n, qh ** -0.5, sink), layers, 4 * layers)
+    fq = rnd(P, H, d)
+    cuk = torch.tensor([0, n], device=dev, dtype=torch.int32)
+    lus = time_in_graph(lambda i: flash_attn_varlen_func(fq, kcs[i], vcs[i], cu, cuk, P, n, softmax_scale=d ** -0.5, causal=True, block_table=big), 4, 16)
+    seen = P * (n - P / 2)
+    add(f"latent_attention portion of {P} at {n}", "flash-attn, paged, the same portion", 2.0 * H * (row + L) * seen, us, 4.0 * H * d * seen, lus, "tensor")
+    return table.rows
+
+
+def run_mupulorn(args, peaks, clock_sampler_cls) -> None:
+    torch, dist, rank, world, local = _setup(args)
+    assert world == 1, "Mupulorn runs on one GPU"
+    from nanovllm_b200 import runtime as rt
+    K, W = min(args.steps, 128), max(3, args.warmup)
+    sizes = {}
+    with clock_sampler_cls(local) as clocks:
+        for name, z in MUPULORN_SIZES.items():
+            res = {}
+            for batch, prompt in ((64, 1024), (4, 4096)):
+                res[f"batch {batch}, prompts of {prompt}"] = {"mupulorn": _model_throughput(torch, _mupulorn_config(z), z["vocab"], batch, prompt, K, W),
+                                                              "qwen3": _model_throughput(torch, _qwen_config(z), z["vocab"], batch, prompt, K, W)}
+            rt.init_runtime(max_tokens=8192, hidden=z["width"], oneshot_tokens=1024)
+            with torch.inference_mode():
+                kernels = _mupulorn_kernels(torch, z, peaks, 64, 1024)
+            rt.shutdown_runtime()
+            torch.cuda.empty_cache()
+            sizes[name] = {"layer_sizes": z, "throughput": res, "kernels": kernels}
+    from nanovllm_b200 import _abi
+    head = sizes["width4096"]["throughput"]["batch 64, prompts of 1024"]["mupulorn"]
+    print(json.dumps({"metric": "mupulorn_decode_tokens_per_s", "value": head["decode_tok_s"], "unit": "tok/s", "n_gpus": 1, "steps": K, "warmup": W,
+                      "ms_per_step": head["decode_ms_per_step"], "higher_is_better": True, "scaling": "strong", "vs_baseline": None, "dtype": "bf16", "data": "synthetic",
+                      "config": {"workload": "Mupulorn and Qwen3 with the same layer sizes, random weights; value: width 4096, batch 64, 1024-token prompts, "
+                                             "device-resident decode", "l2": "weights, caches and rotated kernel inputs exceed the 126 MB L2"},
                       "clocks": clocks.summary(), "gpu_launches": _abi.launch_count(), "sizes": sizes}), flush=True)
     dist.destroy_process_group()
