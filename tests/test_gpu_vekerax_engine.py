@@ -10,6 +10,7 @@ import torch
 from oracle import vekerax as V
 from tests import vekerax_util as U
 from tests.gpu_util import ensure_group
+from tests.model_util import greedy, save, tokens
 
 pytestmark = pytest.mark.gpu
 ROOT = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
@@ -21,9 +22,9 @@ def test_greedy_generation_through_the_engine(pkg, blocks):
     from nanovllm_b200.engine.llm_engine import SamplingParams
     m = U.Model("mixed", torch.float32, max_num_batched_tokens=24, num_kvcache_blocks=blocks)
     try:
-        prompts = [U.tokens(n, m.cfg["vocab"], 40 + n) for n in (30, 3, 55, 1, 20)]
+        prompts = [tokens(n, m.cfg["vocab"], 40 + n) for n in (30, 3, 55, 1, 20)]
         got = m.llm.generate(prompts, SamplingParams(max_tokens=9))
-        assert got == [U.greedy(m, p, 9) for p in prompts]
+        assert got == [greedy(m, p, 9) for p in prompts]
         assert len(m.cache.free_blocks) == blocks and len(m.cache.free_slots) == 4
     finally:
         m.llm.exit()
@@ -35,7 +36,7 @@ def test_generation_in_bf16_repeats_and_samples(pkg):
     for case in ("wide", "odd"):
         m = U.Model(case, torch.bfloat16)
         try:
-            prompts = [U.tokens(n, m.cfg["vocab"], n) for n in (33, 2, 64)]
+            prompts = [tokens(n, m.cfg["vocab"], n) for n in (33, 2, 64)]
             got = m.llm.generate(prompts, SamplingParams(max_tokens=12))
             assert got == m.llm.generate(prompts, SamplingParams(max_tokens=12))
             for p, g in zip(prompts, got):
@@ -52,7 +53,7 @@ def test_resident_decoder_matches_steps(pkg):
     from nanovllm_b200.engine.model_runner import ResidentDecoder, Seq
     m = U.Model("wide", torch.bfloat16)
     try:
-        prompts = [U.tokens(n, m.cfg["vocab"], n) for n in (20, 45)]
+        prompts = [tokens(n, m.cfg["vocab"], n) for n in (20, 45)]
         rd = ResidentDecoder(m.runner, 2)
 
         def start():
@@ -84,9 +85,9 @@ def test_trace_runner_and_command_line(pkg, tmp_path):
     """bin/trace_run and the generate command on a saved model folder."""
     cfg = U.CASES["odd"]
     w = U.weights(cfg, 5)
-    U.save(tmp_path / "m", cfg, w)
+    save(tmp_path / "m", cfg, w)
     w64 = {k: t.double() for k, t in w.items()}
-    toks = U.tokens(30, cfg["vocab"], 7)
+    toks = tokens(30, cfg["vocab"], 7)
     steps = [{"step": 0, "entries": [{"id": "x", "tokens": toks[:20], "want": [0, 19]}], "end": []},
              {"step": 1, "entries": [{"id": "x", "tokens": toks[20:28], "want": []}], "end": []},
              {"step": 2, "entries": [{"id": "x", "tokens": toks[28:29], "want": [0]}], "end": ["x"]},
@@ -104,8 +105,8 @@ def test_trace_runner_and_command_line(pkg, tmp_path):
     r = subprocess.run([sys.executable, os.path.join(ROOT, "bin", "generate"), "--model", str(tmp_path / "m"), "--dtype", "float32", "--max-tokens", "3",
                         "--prompt-ids", ",".join(map(str, toks[:5]))], text=True, capture_output=True, timeout=300)
     assert r.returncode == 0, r.stderr[-800:]
-    m = type("M", (), {"cfg": cfg, "w64": w64})
-    assert json.loads(r.stdout.splitlines()[-1])["token_ids"] == U.greedy(m, toks[:5], 3)
+    m = type("M", (), {"forward": staticmethod(lambda t: V.forward(cfg, w64, t))})
+    assert json.loads(r.stdout.splitlines()[-1])["token_ids"] == greedy(m, toks[:5], 3)
 
 
 def test_qwen3_through_the_same_engine(pkg):
@@ -114,7 +115,7 @@ def test_qwen3_through_the_same_engine(pkg):
     from nanovllm_b200.engine.llm_engine import LLM, SamplingParams
     cfg = {"architectures": ["Qwen3ForCausalLM"], "hidden_size": 256, "num_attention_heads": 4, "num_key_value_heads": 2, "head_dim": 128,
            "intermediate_size": 512, "num_hidden_layers": 2, "vocab_size": 512, "attention_bias": False}
-    prompts = [U.tokens(n, 512, n) for n in (300, 20, 5)]
+    prompts = [tokens(n, 512, n) for n in (300, 20, 5)]
     got = []
     for budget in (512, 100):
         llm = LLM(cfg, max_num_seqs=4, max_model_len=512, max_num_batched_tokens=budget, num_kvcache_blocks=16, seed=3)

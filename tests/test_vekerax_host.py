@@ -5,6 +5,7 @@ import torch
 
 from oracle import vekerax as V
 from tests import vekerax_util as U
+from tests.model_util import save, tokens
 
 
 def test_recurrence_equals_its_closed_form():
@@ -42,7 +43,7 @@ def test_streams_equal_one_residual_when_they_are_not_mixed():
         w[f"l0.hc{q}.in"][:] = 0.25
         w[f"l0.hc{q}.out"][:] = 1.0
         w[f"l0.hc{q}.mix"] = torch.eye(4, dtype=torch.float64)
-    toks = U.tokens(7, cfg["vocab"])
+    toks = tokens(7, cfg["vocab"])
     _, trail = V.forward(cfg, w, toks)
     x = V.embedding(toks, w["embed"], cfg["embedding"]["scale"])
     eps, m = cfg["norm"]["eps"], cfg["residual_mult"]
@@ -99,7 +100,7 @@ def test_checkpoint_reader(pkg, tmp_path):
     from nanovllm_b200.utils.loader import Checkpoint
     cfg = U.CASES["odd"]
     w = U.weights(cfg, 1)
-    U.save(tmp_path, cfg, w)
+    save(tmp_path, cfg, w)
     ck = Checkpoint(str(tmp_path))
     assert set(ck) == set(w) and all(torch.equal(ck[n], w[n]) for n in w)
     assert load_config(str(tmp_path)).width == 60

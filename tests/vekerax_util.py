@@ -2,6 +2,7 @@
 import torch
 
 from oracle import vekerax as V
+from tests.model_util import ServedModel
 
 
 def attn(heads=6, kv_heads=2, dim=24, vdim=40, size=37, keep=3, cap=20.0, scale=0.3, ff=88):
@@ -70,82 +71,7 @@ def weights(cfg, seed=0):
     return w
 
 
-def save(folder, cfg, w):
-    """config.json and model.safetensors (8-byte header length, JSON header, data)."""
-    import json
-    import os
-    import struct
-    os.makedirs(folder, exist_ok=True)
-    with open(os.path.join(folder, "config.json"), "w") as f:
-        json.dump(cfg, f)
-    header, blobs, at = {}, [], 0
-    for name, t in w.items():
-        raw = t.contiguous().view(torch.int16).numpy().tobytes()
-        header[name] = {"dtype": "BF16", "shape": list(t.shape), "data_offsets": [at, at + len(raw)]}
-        blobs.append(raw)
-        at += len(raw)
-    head = json.dumps(header).encode()
-    with open(os.path.join(folder, "model.safetensors"), "wb") as f:
-        f.write(struct.pack("<Q", len(head)) + head + b"".join(blobs))
-
-
-def tokens(n, vocab, seed=0):
-    return torch.randint(0, vocab, (n,), generator=torch.Generator().manual_seed(1000 + seed)).tolist()
-
-
-# root mean square of the logits' error over their own; bf16: what rounding does to these deliberately lively weights
-TOL = {torch.float32: 2e-4, torch.bfloat16: 0.12}
-
-
-class Model:
-    """A test model behind the framework's engine, beside the plain implementation's logits for the same weights (GPU)."""
-
+class Model(ServedModel):
     def __init__(self, case, dtype, **kw):
-        from tests.gpu_util import ensure_group
-        ensure_group()
-        from nanovllm_b200.engine.llm_engine import LLM
-        self.cfg = CASES[case] if isinstance(case, str) else case
-        w = weights(self.cfg, 5)
-        self.w64 = {k: t.double() for k, t in w.items()}
-        self.dtype = dtype
-        self.llm = LLM(self.cfg, w, dtype=dtype, **({"max_num_seqs": 4, "max_model_len": 512, "max_num_batched_tokens": 512, "kvcache_block_size": 16,
-                                                     "num_kvcache_blocks": 80} | kw))
-        self.runner, self.cache = self.llm.runner, self.llm.cache
-        self.memo = {}
-
-    def want(self, toks):
-        key = tuple(toks)
-        if key not in self.memo:
-            self.memo[key] = V.forward(self.cfg, self.w64, list(toks))[0]
-        return self.memo[key]
-
-    def seq(self):
-        from nanovllm_b200.engine.model_runner import Seq
-        return Seq([])
-
-    def feed(self, seqs, parts):
-        """One step that brings `parts` (token lists) to the sequences; logits of every new token, per sequence."""
-        for s, p in zip(seqs, parts):
-            s.token_ids += p
-            self.cache.hold(s, len(s))
-        counts = [len(p) for p in parts]
-        decode = all(c == 1 for c in counts) and all(s.num_cached_tokens for s in seqs)
-        out = self.runner.step_logits(seqs, not decode, None if decode else counts, list(range(sum(counts))))
-        for s, c in zip(seqs, counts):
-            s.num_cached_tokens += c
-        return list(out.split(counts))
-
-    def check(self, got, want, what):
-        err = (got.double() - want).pow(2).mean(-1).sqrt() / want.pow(2).mean(-1).sqrt()
-        assert torch.isfinite(got).all() and err.max() < TOL[self.dtype], f"{what}: error {err.max().item():.2e} at row {int(err.argmax())}"
-
-    def free(self, *seqs):
-        for s in seqs:
-            self.cache.release(s)
-
-
-def greedy(m, prompt, n):
-    toks = list(prompt)
-    for _ in range(n):
-        toks.append(int(V.forward(m.cfg, m.w64, toks)[0][-1].argmax()))
-    return toks[len(prompt):]
+        cfg = CASES[case] if isinstance(case, str) else case
+        super().__init__(V.forward, cfg, weights(cfg, 5), dtype, **kw)
