@@ -74,11 +74,11 @@ struct Vec8<float> {
 };
 
 // TAPS > 0: that many taps, history and weights in registers; 0: no convolution; -1: a.taps, history in shared memory.
-// NV vectors of 8 channels per thread.
-template <typename T, int NV, int TAPS>
+// NV vectors of 8 channels per thread; RB tokens at a time, so that their loads are in flight together and share barriers.
+template <typename T, int NV, int TAPS, int RB>
 __global__ void __launch_bounds__(512) sandwich_step_kernel(const SandwichArgs a) {
   extern __shared__ __align__(16) unsigned char hist_smem[];  // TAPS < 0: [taps - 1][dim_pad], a ring by row
-  __shared__ float red[2][32];
+  __shared__ __align__(16) float red[2][16][RB];
   constexpr bool CONV = TAPS != 0, REG = TAPS > 0;
   constexpr int HIST = REG && TAPS > 1 ? TAPS - 1 : 1;
   const int taps = REG ? TAPS : a.taps;
@@ -122,122 +122,163 @@ __global__ void __launch_bounds__(512) sandwich_step_kernel(const SandwichArgs a
         else v.store(ring + static_cast<int64_t>(j) * a.dim_pad + nv[i]);
       }
   }
+  const int warps = (blockDim.x + 31) >> 5;
   int flip = 0;
-  auto total = [&](float v) {  // sum over the CTA; two buffers in turn, so one barrier per sum is enough
-    v = b2::block_sum(v, red[flip]);
+  auto total = [&](float (&v)[RB]) {  // sums over the CTA; two buffers in turn, so one barrier per call is enough
+#pragma unroll
+    for (int r = 0; r < RB; ++r) v[r] = b2::group_sum(v[r]);
+    if ((threadIdx.x & 31) == 0) {
+#pragma unroll
+      for (int r = 0; r < RB; ++r) red[flip][threadIdx.x >> 5][r] = v[r];
+    }
+    __syncthreads();
+#pragma unroll
+    for (int r = 0; r < RB; ++r) v[r] = 0.f;
+    for (int i = 0; i < warps; ++i) {
+      if constexpr (RB == 4) {
+        const float4 q = *reinterpret_cast<const float4*>(red[flip][i]);
+        v[0] += q.x; v[1] += q.y; v[2] += q.z; v[3] += q.w;
+      } else {
+#pragma unroll
+        for (int r = 0; r < RB; ++r) v[r] += red[flip][i][r];
+      }
+    }
     flip ^= 1;
-    return v;
   };
   const float inv_dim = 1.0f / static_cast<float>(a.dim);
 
-  auto process = [&](int t, bool emit) {
-    const int64_t row = row0 + t;
-    float x[NV][8];
-    const T* emb = nullptr;
-    if (a.ids != nullptr) {
-      int64_t id = a.ids[row];
-      if (id < 0 || id >= a.vocab) id = 0;
-      emb = static_cast<const T*>(a.table) + id * a.ld_table;
-    }
-    float y[NV][8], ss = 0.f;
+  // tokens t0 .. min(t0 + RB, end) - 1, of which those from `emit` on are written
+  auto process = [&](int t0, int end, int emit) {
+    float x[RB][NV][8], ss[RB];
+    Vec8<T> y[RB][NV];
 #pragma unroll
-    for (int i = 0; i < NV; ++i) {
+    for (int r = 0; r < RB; ++r) {
+      const bool live = t0 + r < end;
+      const int64_t row = row0 + t0 + (live ? r : 0);
+      const T* emb = nullptr;
+      if (a.ids != nullptr) {
+        int64_t id = a.ids[row];
+        if (id < 0 || id >= a.vocab) id = 0;
+        emb = static_cast<const T*>(a.table) + id * a.ld_table;
+      }
 #pragma unroll
-      for (int e = 0; e < 8; ++e) x[i][e] = y[i][e] = 0.f;
-      if (nv[i] < 0) continue;
-      if (emb != nullptr) b2::load8<T>(emb + nv[i], x[i]);
-      else b2::load8<float>(a.x_in + row * a.dim_pad + nv[i], x[i]);
-      if (a.y != nullptr) b2::load8<T>(static_cast<const T*>(a.y) + row * a.ldy + nv[i], y[i]);
+      for (int i = 0; i < NV; ++i) {
+#pragma unroll
+        for (int e = 0; e < 8; ++e) x[r][i][e] = 0.f;
+        y[r][i].zero();
+        if (nv[i] < 0) continue;
+        if (emb != nullptr) b2::load8<T>(emb + nv[i], x[r][i]);
+        else b2::load8<float>(a.x_in + row * a.dim_pad + nv[i], x[r][i]);
+        if (a.y != nullptr) y[r][i].load(static_cast<const T*>(a.y) + row * a.ldy + nv[i]);
+      }
     }
     if (a.y != nullptr) {
 #pragma unroll
-      for (int i = 0; i < NV; ++i)
+      for (int r = 0; r < RB; ++r) {
+        ss[r] = 0.f;
 #pragma unroll
-        for (int e = 0; e < 8; ++e) ss += y[i][e] * y[i][e];
-      const float r = 1.0f / sqrtf(total(ss) * inv_dim + a.eps);
+        for (int i = 0; i < NV; ++i) {
+          float f[8];
+          y[r][i].get(f);
+#pragma unroll
+          for (int e = 0; e < 8; ++e) ss[r] += f[e] * f[e];
+        }
+      }
+      total(ss);
+      float g[8];
+#pragma unroll
+      for (int e = 0; e < 8; ++e) g[e] = a.post_w[0];
 #pragma unroll
       for (int i = 0; i < NV; ++i) {
         if (nv[i] < 0) continue;
-        if (a.post_vec) {
+        if (a.post_vec) b2::load8<float>(a.post_w + nv[i], g);
+#pragma unroll
+        for (int r = 0; r < RB; ++r) {
+          const float rstd = 1.0f / sqrtf(ss[r] * inv_dim + a.eps);
+          float f[8];
+          y[r][i].get(f);
+#pragma unroll
+          for (int e = 0; e < 8; ++e) x[r][i][e] += f[e] * (rstd * g[e]);
+        }
+      }
+    }
+#pragma unroll
+    for (int r = 0; r < RB; ++r) {
+      const bool out = t0 + r >= emit && t0 + r < end;
+      ss[r] = 0.f;
+#pragma unroll
+      for (int i = 0; i < NV; ++i) {
+#pragma unroll
+        for (int e = 0; e < 8; ++e) ss[r] += x[r][i][e] * x[r][i][e];
+        if (out && a.x_out != nullptr && nv[i] >= 0) b2::store8<float>(a.x_out + (row0 + t0 + r) * static_cast<int64_t>(a.dim_pad) + nv[i], x[r][i]);
+      }
+    }
+    total(ss);
+#pragma unroll
+    for (int r = 0; r < RB; ++r) {
+      if (t0 + r >= end) break;
+      const int64_t row = row0 + t0 + r;
+      const float rstd = 1.0f / sqrtf(ss[r] * inv_dim + a.eps);
+#pragma unroll
+      for (int i = 0; i < NV; ++i) {
+        if (nv[i] < 0) continue;
+        if (a.norm_vec) {
           float g[8];
-          b2::load8<float>(a.post_w + nv[i], g);
+          b2::load8<float>(a.norm_w + nv[i], g);
 #pragma unroll
-          for (int e = 0; e < 8; ++e) x[i][e] += y[i][e] * r * g[e];
+          for (int e = 0; e < 8; ++e) x[r][i][e] = x[r][i][e] * rstd * g[e];
         } else {
-          const float g = r * a.post_w[0];
+          const float g = rstd * a.norm_w[0];
 #pragma unroll
-          for (int e = 0; e < 8; ++e) x[i][e] += y[i][e] * g;
+          for (int e = 0; e < 8; ++e) x[r][i][e] *= g;
         }
-      }
-    }
-    ss = 0.f;
+        Vec8<T> h;
+        h.set(x[r][i]);
+        T* dst = static_cast<T*>(a.out) + row * a.ldo + nv[i];
+        if constexpr (!CONV) {
+          h.store(dst);
+        } else {
+          if (t0 + r >= emit) {
+            float acc[8], hf[8], wf[8];
+            h.get(hf);
+            if constexpr (REG) w[TAPS - 1][i].get(wf);
+            else b2::load8<T>(static_cast<const T*>(a.conv_w) + static_cast<int64_t>(taps - 1) * a.dim_pad + nv[i], wf);
 #pragma unroll
-    for (int i = 0; i < NV; ++i) {
+            for (int e = 0; e < 8; ++e) acc[e] = fmaf(wf[e], hf[e], hf[e]);
 #pragma unroll
-      for (int e = 0; e < 8; ++e) ss += x[i][e] * x[i][e];
-      if (emit && a.x_out != nullptr && nv[i] >= 0) b2::store8<float>(a.x_out + row * a.dim_pad + nv[i], x[i]);
-    }
-    const float r = 1.0f / sqrtf(total(ss) * inv_dim + a.eps);
+            for (int j = 0; j < (REG ? TAPS - 1 : taps - 1); ++j) {
+              float f[8];
+              if constexpr (REG) {
+                w[j][i].get(wf);
+                hist[j][i].get(f);
+              } else {
+                b2::load8<T>(static_cast<const T*>(a.conv_w) + static_cast<int64_t>(j) * a.dim_pad + nv[i], wf);
+                b2::load8<T>(ring + static_cast<int64_t>((head + j) % (taps - 1)) * a.dim_pad + nv[i], f);
+              }
 #pragma unroll
-    for (int i = 0; i < NV; ++i) {
-      if (nv[i] < 0) continue;
-      if (a.norm_vec) {
-        float g[8];
-        b2::load8<float>(a.norm_w + nv[i], g);
-#pragma unroll
-        for (int e = 0; e < 8; ++e) x[i][e] = x[i][e] * r * g[e];
-      } else {
-        const float g = r * a.norm_w[0];
-#pragma unroll
-        for (int e = 0; e < 8; ++e) x[i][e] *= g;
-      }
-      Vec8<T> h;
-      h.set(x[i]);
-      T* dst = static_cast<T*>(a.out) + row * a.ldo + nv[i];
-      if constexpr (!CONV) {
-        h.store(dst);
-      } else {
-        float acc[8], hf[8], wf[8];
-        h.get(hf);
-        if (emit) {
-          if constexpr (REG) w[TAPS - 1][i].get(wf);
-          else b2::load8<T>(static_cast<const T*>(a.conv_w) + static_cast<int64_t>(taps - 1) * a.dim_pad + nv[i], wf);
-#pragma unroll
-          for (int e = 0; e < 8; ++e) acc[e] = fmaf(wf[e], hf[e], hf[e]);
-#pragma unroll
-          for (int j = 0; j < (REG ? TAPS - 1 : taps - 1); ++j) {
-            float f[8];
-            if constexpr (REG) {
-              w[j][i].get(wf);
-              hist[j][i].get(f);
-            } else {
-              b2::load8<T>(static_cast<const T*>(a.conv_w) + static_cast<int64_t>(j) * a.dim_pad + nv[i], wf);
-              b2::load8<T>(ring + static_cast<int64_t>((head + j) % (taps - 1)) * a.dim_pad + nv[i], f);
+              for (int e = 0; e < 8; ++e) acc[e] = fmaf(wf[e], f[e], acc[e]);
             }
-#pragma unroll
-            for (int e = 0; e < 8; ++e) acc[e] = fmaf(wf[e], f[e], acc[e]);
+            b2::store8<T>(dst, acc);
           }
-          b2::store8<T>(dst, acc);
-        }
-        if constexpr (REG) {
+          if constexpr (REG) {
 #pragma unroll
-          for (int j = 0; j + 1 < TAPS - 1; ++j) hist[j][i] = hist[j + 1][i];
-          if (TAPS > 1) hist[HIST - 1][i] = h;
-        } else if (taps > 1) {
-          h.store(ring + static_cast<int64_t>(head) * a.dim_pad + nv[i]);
+            for (int j = 0; j + 1 < TAPS - 1; ++j) hist[j][i] = hist[j + 1][i];
+            if (TAPS > 1) hist[HIST - 1][i] = h;
+          } else if (taps > 1) {
+            h.store(ring + static_cast<int64_t>(head) * a.dim_pad + nv[i]);
+          }
         }
       }
+      if (!REG && CONV && taps > 1) head = (head + 1) % (taps - 1);
     }
-    if (!REG && CONV && taps > 1) head = (head + 1) % (taps - 1);
   };
 
-  if (CONV && start > 0)
-    for (int t = start - (taps - 1); t < start; ++t) process(t, false);  // run >= taps - 1: these tokens are part of the step
-  for (int t = start; t < stop; ++t) process(t, true);
+  // the tokens before a later run are part of the step (run >= taps - 1): computed again, not written
+  for (int t = CONV && start > 0 ? start - (taps - 1) : start; t < stop; t += RB) process(t, stop, start);
   if constexpr (CONV) {
     if (start > 0 || state == nullptr) return;
     if (stop < n_q)
-      for (int t = n_q - (taps - 1); t < n_q; ++t) process(t, false);
+      for (int t = n_q - (taps - 1); t < n_q; t += RB) process(t, n_q, n_q);
 #pragma unroll
     for (int j = 0; j < (REG ? TAPS - 1 : taps - 1); ++j)
 #pragma unroll
@@ -257,31 +298,57 @@ __global__ void __launch_bounds__(512) sandwich_step_kernel(const SandwichArgs a
 
 bool aligned16(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; }
 
-template <typename T, int NV, int TAPS>
-int launch(const SandwichArgs& a, dim3 grid, int threads, size_t smem, cudaStream_t s) {
-  if (smem > 48 * 1024) B2_CUDA(cudaFuncSetAttribute(sandwich_step_kernel<T, NV, TAPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)));
-  B2_CUDA(b2_launch(sandwich_step_kernel<T, NV, TAPS>, grid, dim3(threads), smem, s, a));
+template <typename T, int NV, int TAPS, int RB>
+int launch(SandwichArgs a, int B, int max_q, int run, int threads, size_t smem, cudaStream_t s) {
+  const auto kernel = sandwich_step_kernel<T, NV, TAPS, RB>;
+  if (smem > 48 * 1024) B2_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)));
+  const int back = a.taps > 0 ? a.taps - 1 : 0;
+  if (max_q == 1) run = 1;
+  if (run == 0) {
+    // tokens per CTA: the fewest rounds of groups over all SMs, where a run also walks the tokens in front of it
+    int resident = 1;
+    B2_CUDA(cudaOccupancyMaxActiveBlocksPerMultiprocessor(&resident, kernel, threads, smem));
+    const int64_t at_once = 148ll * std::max(1, resident);
+    int64_t best = INT64_MAX;
+    for (int groups = 1; groups <= 16; ++groups) {
+      const int r = groups * RB - back;
+      if (r < 1) continue;
+      const int64_t ctas = static_cast<int64_t>(B) * ((max_q + r - 1) / r);
+      const int64_t cost = (ctas + at_once - 1) / at_once * groups;
+      if (cost < best) {
+        best = cost;
+        run = r;
+      }
+      if (r >= max_q) break;
+    }
+  }
+  a.run = std::max({run, back, (max_q + 65534) / 65535, 1});
+  B2_CUDA(b2_launch(kernel, dim3(B, (max_q + a.run - 1) / a.run), dim3(threads), smem, s, a));
   return B2_OK;
 }
 template <typename T, int NV>
-int dispatch_taps(const SandwichArgs& a, dim3 grid, int threads, cudaStream_t s) {
-  switch (a.taps) {
-    case 0: return launch<T, NV, 0>(a, grid, threads, 0, s);
-    case 2: if constexpr (NV == 1) return launch<T, NV, 2>(a, grid, threads, 0, s); break;
-    case 3: if constexpr (NV == 1) return launch<T, NV, 3>(a, grid, threads, 0, s); break;
-    case 4: if constexpr (NV == 1) return launch<T, NV, 4>(a, grid, threads, 0, s); break;
-    default: break;
+int dispatch_taps(const SandwichArgs& a, int B, int max_q, int run, int threads, cudaStream_t s) {
+#define B2_STEP(TAPS) return max_q > 1 ? launch<T, NV, TAPS, 4>(a, B, max_q, run, threads, 0, s) : launch<T, NV, TAPS, 1>(a, B, max_q, run, threads, 0, s)
+  if (a.taps == 0) return launch<T, NV, 0, 1>(a, B, max_q, run, threads, 0, s);
+  if constexpr (NV == 1) {
+    switch (a.taps) {
+      case 2: B2_STEP(2);
+      case 3: B2_STEP(3);
+      case 4: B2_STEP(4);
+      default: break;
+    }
   }
+#undef B2_STEP
   const size_t smem = static_cast<size_t>(a.taps - 1) * a.dim_pad * sizeof(T);
   if (smem > 200 * 1024) return b2::set_error(B2_ERR_SHAPE, "b2_sandwich_step: %d taps on %d channels do not fit in shared memory", a.taps, a.dim_pad);
-  return launch<T, NV, -1>(a, grid, threads, smem, s);
+  return launch<T, NV, -1, 1>(a, B, max_q, run, threads, smem, s);
 }
 template <typename T>
-int dispatch(const SandwichArgs& a, dim3 grid, cudaStream_t s) {
+int dispatch(const SandwichArgs& a, int B, int max_q, int run, cudaStream_t s) {
   const int nvec = a.dim_pad / 8;
-  if (nvec <= 512) return dispatch_taps<T, 1>(a, grid, (nvec + 31) / 32 * 32, s);
-  if (nvec <= 1024) return dispatch_taps<T, 2>(a, grid, (nvec + 63) / 64 * 32, s);
-  return dispatch_taps<T, 8>(a, grid, 512, s);
+  if (nvec <= 512) return dispatch_taps<T, 1>(a, B, max_q, run, (nvec + 31) / 32 * 32, s);
+  if (nvec <= 1024) return dispatch_taps<T, 2>(a, B, max_q, run, (nvec + 63) / 64 * 32, s);
+  return dispatch_taps<T, 8>(a, B, max_q, run, 512, s);
 }
 
 // out = a N(z) + b N(z^2) + c N(z^3) + e, N dividing by the root mean square over the row's `dim` elements
@@ -390,16 +457,12 @@ int b2_sandwich_step(int dtype, const float* x_in, float* x_out, const int64_t* 
                        (post_len != 1 && !aligned16(post_w)))) return B2_ERR_ARG;
   if (taps > 0 && (!conv_w || !aligned16(conv_w) || !slots || !kv_len || (taps > 1 && (!state || !aligned16(state))))) return B2_ERR_ARG;
   if (dim_pad > 32768) return B2_ERR_SHAPE;
-  // tokens per CTA: few enough that every SM has some CTAs, many enough that a run's first tokens are cheap to compute again
-  if (run == 0) run = static_cast<int>(std::min<int64_t>(16, std::max<int64_t>(4, static_cast<int64_t>(B) * max_q / (148 * 4))));
-  run = std::max({run, taps - 1, (max_q + 65534) / 65535});
   SandwichArgs a{};
   a.x_in = x_in; a.x_out = x_out; a.ids = ids; a.table = table; a.ld_table = ld_table; a.vocab = vocab; a.y = y; a.ldy = ldy;
   a.post_w = post_w; a.post_vec = post_len != 1; a.norm_w = norm_w; a.norm_vec = norm_len != 1; a.eps = eps; a.conv_w = conv_w; a.taps = taps;
-  a.state = state; a.slots = slots; a.cu_q = cu_q; a.kv_len = kv_len; a.out = out; a.ldo = ldo; a.dim = dim; a.dim_pad = dim_pad; a.run = run;
-  const dim3 grid(B, (max_q + run - 1) / run);
+  a.state = state; a.slots = slots; a.cu_q = cu_q; a.kv_len = kv_len; a.out = out; a.ldo = ldo; a.dim = dim; a.dim_pad = dim_pad;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  return dtype == B2_DT_BF16 ? dispatch<uint16_t>(a, grid, s) : dispatch<float>(a, grid, s);
+  return dtype == B2_DT_BF16 ? dispatch<uint16_t>(a, B, max_q, run, s) : dispatch<float>(a, B, max_q, run, s);
 }
 
 int b2_poly_norm(int dtype, const void* z, int64_t ldz, const float* coef, float eps, int M, int dim, int dim_pad, void* out, int64_t ldo, void* stream) {
