@@ -534,19 +534,26 @@ int b2_latent_gather(int dtype, const void* cache, const int32_t* block_tables, 
  * inputs / outputs start every x_head / out_head elements.  gate (may be NULL):
  * out is multiplied by sigmoid(gate[m, h gate_head + n]).  rot_pad > 0: the
  * rot_pad elements behind a head's K inputs are rotated by positions[m] and
- * written behind its N outputs. */
+ * written behind its N outputs.  w is a constant: it may be fetched while the
+ * previous b2_* kernel is still running. */
 int b2_heads_gemm(int dtype, const void* x, int64_t ldx, int x_head, const void* w, int64_t ldw, int64_t w_head, int w_is_kn,
                   void* out, int64_t ldo, int out_head, int M, int heads, int N, int K, const void* gate, int64_t ldg,
                   int gate_head, int rot_pad, const int64_t* positions, const float* cos_sin, int max_pos, void* stream);
 
 /* Absorbed attention: every head's query [lat_pad | rot_pad] attends to the cached
  * rows themselves (score = q . row * scale) and mixes their first lat_pad
- * elements: out [M][heads][lat_pad].  Causal; the rest as in b2_attention. */
-int64_t b2_latent_attention_workspace(int dtype, int B, int max_q, int max_kv, int heads, int lat_pad, int rot_pad);
-int b2_latent_attention(int dtype, const void* q, int64_t ldq, void* out, int64_t ldo, const void* cache,
-                        const int32_t* block_tables, int64_t bt_stride, int block_size, const int32_t* cu_q,
-                        const int32_t* kv_len, int B, int max_q, int max_kv, int heads, int lat_pad, int rot_pad, float scale,
-                        const float* sink, void* workspace, int64_t workspace_bytes, int form, void* stream);
+ * elements: out [q_rows][heads][lat_pad], row stride ldo.  q is contiguous
+ * [q_rows][heads][lat_pad + rot_pad], the cache [cache_slots][lat_pad + rot_pad]
+ * without values that are not finite.  Causal; the rest as in b2_attention.  bf16,
+ * latents up to 512, rotated parts up to 64 and blocks of a multiple of 128 slots
+ * run on tcgen05 (a bounded wait that expires there shows in b2_status), all
+ * other sizes, fp32 and form 1 on the kernel for any size (ctx may be NULL). */
+int64_t b2_latent_attention_workspace(int dtype, int B, int max_q, int max_kv, int block_size, int heads, int lat_pad, int rot_pad);
+int b2_latent_attention(b2_ctx* ctx, int dtype, const void* q, int64_t q_rows, void* out, int64_t ldo, const void* cache,
+                        int64_t cache_slots, const int32_t* block_tables, int64_t bt_stride, int block_size,
+                        const int32_t* cu_q, const int32_t* kv_len, int B, int max_q, int max_kv, int heads, int lat_pad,
+                        int rot_pad, float scale, const float* sink, void* workspace, int64_t workspace_bytes, int form,
+                        void* stream);
 
 /* Expanded attention (bf16; dim_pad + rot_pad <= 192, v_pad <= 128): rows of kv hold
  * [dim_pad key | v_pad value] per head, rows of rot the shared rotated key part;

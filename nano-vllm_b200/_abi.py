@@ -74,7 +74,7 @@ SIGNATURES = {
     "b2_latent_store": [_i, _p, _i64, _i, _i, _i, _i, _i, _i, _p, _p, _f, _p, _p, _i, _p, _p, _p],
     "b2_latent_gather": [_i, _p, _p, _i64, _i, _p, _i, _i, _i, _p, _p],
     "b2_heads_gemm": [_i, _p, _i64, _i, _p, _i64, _i64, _i, _p, _i64, _i, _i, _i, _i, _i, _p, _i64, _i, _i, _p, _p, _i, _p],
-    "b2_latent_attention": [_i, _p, _i64, _p, _i64, _p, _p, _i64, _i, _p, _p, _i, _i, _i, _i, _i, _i, _f, _p, _p, _i64, _i, _p],
+    "b2_latent_attention": [_p, _i, _p, _i64, _p, _i64, _p, _i64, _p, _i64, _i, _p, _p, _i, _i, _i, _i, _i, _i, _f, _p, _p, _i64, _i, _p],
     "b2_expanded_attention": [_p, _i64, _p, _i64, _p, _i64, _p, _i64, _p, _p, _i, _i, _i, _i, _i, _i, _f, _p, _p, _i, _p, _i64, _p],
     "b2_gemm_static_scratch": [_p, _i64, _p, _i64, _p, _p, _i64, _i, _i, _i, _p],
     "b2_rowpar_fused": [_p, _p, _i64, _p, _i64, _p, _i, _i, _i, _p, _p, _f, _p, _p, _p],
@@ -110,7 +110,7 @@ for _name, _args in SIGNATURES.items():
     _fn = getattr(lib, _name)
     _fn.argtypes = _args
     _fn.restype = _i
-WORKSPACES = {"b2_attention_workspace": [_i] * 10, "b2_linear_attn_workspace": [_i] * 7, "b2_latent_attention_workspace": [_i] * 7}
+WORKSPACES = {"b2_attention_workspace": [_i] * 10, "b2_linear_attn_workspace": [_i] * 7, "b2_latent_attention_workspace": [_i] * 8}
 for _name, _args in WORKSPACES.items():
     _fn = getattr(lib, _name)
     _fn.argtypes = _args

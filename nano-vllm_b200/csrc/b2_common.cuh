@@ -277,6 +277,28 @@ __device__ __forceinline__ void tmem_ld_32x32(uint32_t taddr, uint32_t (&r)[32])
       : "memory");
 }
 
+// The same for 16 columns, and stores of registers back into tensor memory.
+__device__ __forceinline__ void tmem_ld_32x16(uint32_t taddr, uint32_t (&r)[16]) {
+  asm volatile(
+      "tcgen05.ld.sync.aligned.32x32b.x16.b32 "
+      "{%0, %1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15}, [%16];"
+      : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7]),
+        "=r"(r[8]), "=r"(r[9]), "=r"(r[10]), "=r"(r[11]), "=r"(r[12]), "=r"(r[13]), "=r"(r[14]), "=r"(r[15])
+      : "r"(taddr)
+      : "memory");
+}
+__device__ __forceinline__ void tmem_st_32x16(uint32_t taddr, const uint32_t (&r)[16]) {
+  asm volatile(
+      "tcgen05.st.sync.aligned.32x32b.x16.b32 [%16], "
+      "{%0, %1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15};"
+      ::"r"(r[0]), "r"(r[1]), "r"(r[2]), "r"(r[3]), "r"(r[4]), "r"(r[5]), "r"(r[6]), "r"(r[7]),
+        "r"(r[8]), "r"(r[9]), "r"(r[10]), "r"(r[11]), "r"(r[12]), "r"(r[13]), "r"(r[14]), "r"(r[15]), "r"(taddr)
+      : "memory");
+}
+__device__ __forceinline__ void tc_wait_st() { asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory"); }
+// shared-memory writes of this thread become visible to the tensor cores and bulk copies (async proxy)
+__device__ __forceinline__ void fence_proxy_async() { asm volatile("fence.proxy.async.shared::cta;" ::: "memory"); }
+
 // Shared-memory operand descriptor for a K-major bf16 tile whose rows are 128
 // bytes (64 elements) apart, laid out by TMA with the 128-byte swizzle:
 // groups of 8 rows are 1024 bytes apart (stride byte offset), the leading byte
@@ -291,6 +313,21 @@ __device__ __forceinline__ uint64_t umma_smem_desc(uint32_t smem_addr) {
   d |= static_cast<uint64_t>(2) << 61;                     // layout type, bits [61,64)
   return d;
 }
+
+// The same for an operand stored with its M (or N) dimension contiguous: 64 elements (128 bytes, 128-byte swizzle) per k,
+// groups of 8 k 1024 bytes apart (stride byte offset), blocks of 64 M elements `mn_stride` bytes apart (leading byte offset).
+// The instruction descriptor must name the operand as transposed (UMMA_A_MN).
+__device__ __forceinline__ uint64_t umma_smem_desc_mn(uint32_t smem_addr, uint32_t mn_stride) {
+  uint64_t d = 0;
+  d |= static_cast<uint64_t>((smem_addr & 0x3FFFF) >> 4);
+  d |= static_cast<uint64_t>((mn_stride >> 4) & 0x3FFF) << 16;
+  d |= static_cast<uint64_t>(1024 >> 4) << 32;
+  d |= static_cast<uint64_t>(1) << 46;
+  d |= static_cast<uint64_t>(2) << 61;
+  return d;
+}
+constexpr uint32_t UMMA_A_MN = 1u << 15;  // instruction descriptor: A has its M dimension contiguous
+constexpr uint32_t UMMA_B_MN = 1u << 16;  // ... B its N dimension
 
 // Instruction descriptor of tcgen05.mma.kind::f16: fp32 accumulator, bf16 A and
 // B, both K-major, M = 128, N = n.

@@ -8,7 +8,7 @@
 //   latent_store_kernel    RMSNorm of the query latent and of the cached latent, rotation of the key part, scatter
 //   latent_gather_kernel   cached rows of a batch as contiguous rows (a portion whose sequence has earlier tokens)
 //   heads_gemm_kernel      one small matrix product per head, with the rotation of the query part or an output gate
-//   latent_attn_kernel     absorbed attention on the tensor cores: 16 or 32 (token, head) rows x 64 keys
+//   latent_tc_kernel       absorbed attention on tcgen05: 16 or 32 (token, head) rows, 128 keys per tile
 //   expanded_attn_kernel   expanded attention, 64 tokens of one head x 64 keys; rotates the queries it loads, gates its output
 #include <algorithm>
 
@@ -40,23 +40,42 @@ __device__ __forceinline__ void rotate8(float (&f)[8], const float2* cs, int max
 // ---------------------------------------------------------------------------
 template <typename T>
 __device__ __forceinline__ void warp_rms(const T* src, int dim, int pad, const float* w, float eps, int lane, T* dst0, T* dst1) {
-  float ss = 0.f;
-  for (int c = lane * 8; c < pad; c += 256) {
-    float f[8];
-    load8<T>(src + c, f);
+  constexpr int KEEP = sizeof(T) == 2 ? 6 : 3;  // vectors of 8 a lane keeps in registers; longer rows are read again
+  float f[KEEP][8], ss = 0.f;
 #pragma unroll
-    for (int e = 0; e < 8; ++e) ss += f[e] * f[e];
+  for (int i = 0; i < KEEP; ++i) {
+#pragma unroll
+    for (int e = 0; e < 8; ++e) f[i][e] = 0.f;
+    const int c = (lane + 32 * i) * 8;
+    if (c < pad) load8<T>(src + c, f[i]);
+  }
+#pragma unroll
+  for (int i = 0; i < KEEP; ++i)
+#pragma unroll
+    for (int e = 0; e < 8; ++e) ss += f[i][e] * f[i][e];
+  for (int c = (lane + 32 * KEEP) * 8; c < pad; c += 256) {
+    float g[8];
+    load8<T>(src + c, g);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) ss += g[e] * g[e];
   }
   ss = group_sum(ss);
   const float rstd = 1.0f / sqrtf(ss / static_cast<float>(dim) + eps);
-  for (int c = lane * 8; c < pad; c += 256) {
-    float f[8], g[8];
-    load8<T>(src + c, f);
+  auto finish = [&](int c, float (&v)[8]) {
+    float g[8];
     load8<float>(w + c, g);
 #pragma unroll
-    for (int e = 0; e < 8; ++e) f[e] = f[e] * rstd * g[e];
-    store8<T>(dst0 + c, f);
-    if (dst1 != nullptr) store8<T>(dst1 + c, f);
+    for (int e = 0; e < 8; ++e) v[e] = v[e] * rstd * g[e];
+    store8<T>(dst0 + c, v);
+    if (dst1 != nullptr) store8<T>(dst1 + c, v);
+  };
+#pragma unroll
+  for (int i = 0; i < KEEP; ++i)
+    if ((lane + 32 * i) * 8 < pad) finish((lane + 32 * i) * 8, f[i]);
+  for (int c = (lane + 32 * KEEP) * 8; c < pad; c += 256) {
+    float g[8];
+    load8<T>(src + c, g);
+    finish(c, g);
   }
 }
 
@@ -139,50 +158,79 @@ __device__ __forceinline__ void rotate_rows(const HeadsArgs& a, int m0, int h) {
   }
 }
 
+// Output tiles of 64 x NT, K in steps of 64 of which HEADS_STAGES - 1 are in flight
+constexpr int HEADS_STAGES = 4;
+template <bool KN>
+struct CfgHeads {
+  static constexpr int NT = KN ? 64 : 32;
+  static constexpr int A_BYTES = 64 * 64 * 2, STAGE = A_BYTES + 64 * NT * 2;
+  static constexpr int SMEM = HEADS_STAGES * STAGE + 128;
+};
 template <bool KN>
 __global__ void __launch_bounds__(128) heads_gemm_kernel(const HeadsArgs a) {
-  __shared__ __align__(128) unsigned char smem[2][2][64 * 64 * 2];
+  using C = CfgHeads<KN>;
+  constexpr int NT = C::NT;
+  extern __shared__ unsigned char smem_raw[];
+  const uint32_t base = (smem_u32(smem_raw) + 127) & ~127u;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int n0 = blockIdx.x * NT, m0 = blockIdx.y * 64, h = blockIdx.z;
   pdl_launch_dependents();
-  pdl_wait();
-  const int n0 = blockIdx.x * 64, m0 = blockIdx.y * 64, h = blockIdx.z;
-  if (n0 >= a.N) {
-    rotate_rows<uint16_t>(a, m0, h);
-    return;
-  }
   const uint16_t* x = static_cast<const uint16_t*>(a.x) + static_cast<int64_t>(h) * a.x_hs;
   const uint16_t* w = static_cast<const uint16_t*>(a.w) + h * a.w_hs;
-  auto load = [&](int st, int k0) {
-    const uint32_t sa = smem_u32(smem[st][0]), sw = smem_u32(smem[st][1]);
+  auto load_w = [&](int st, int k0) {
+    const uint32_t sw = base + st * C::STAGE + C::A_BYTES;
+#pragma unroll
+    for (int i = 0; i < NT / 16; ++i) {
+      const int idx = threadIdx.x + i * 128, r = idx >> 3, p = idx & 7;
+      const int wr = (KN ? k0 : n0) + r, wc = (KN ? n0 : k0) + p * 8;
+      const bool ok = wr < (KN ? a.K : a.N) && wc < (KN ? a.N : a.K);
+      cp_async16(tile_addr<64>(sw, r, p), ok ? w + wr * a.ldw + wc : w, ok);
+    }
+  };
+  auto load_x = [&](int st, int k0) {
+    const uint32_t sa = base + st * C::STAGE;
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
       const int idx = threadIdx.x + i * 128, r = idx >> 3, p = idx & 7;
       const bool ok = m0 + r < a.M && k0 + p * 8 < a.K;
       cp_async16(tile_addr<64>(sa, r, p), ok ? x + (m0 + r) * a.ldx + k0 + p * 8 : x, ok);
-      const int wr = (KN ? k0 : n0) + r, wc = (KN ? n0 : k0) + p * 8;
-      const bool wok = wr < (KN ? a.K : a.N) && wc < (KN ? a.N : a.K);
-      cp_async16(tile_addr<64>(sw, r, p), wok ? w + wr * a.ldw + wc : w, wok);
     }
   };
-  float acc[8][4];
+  const bool product = n0 < a.N;
+  // weights do not depend on an earlier kernel: the first ones are fetched before the wait
+  if (product)
+    for (int i = 0; i < HEADS_STAGES - 1; ++i)
+      if (i * 64 < a.K) load_w(i, i * 64);
+  pdl_wait();
+  if (!product) {
+    rotate_rows<uint16_t>(a, m0, h);
+    return;
+  }
+  for (int i = 0; i < HEADS_STAGES - 1; ++i) {
+    if (i * 64 < a.K) load_x(i, i * 64);
+    cp_async_commit();
+  }
+  float acc[NT / 8][4];
 #pragma unroll
-  for (int n = 0; n < 8; ++n)
+  for (int n = 0; n < NT / 8; ++n)
 #pragma unroll
     for (int e = 0; e < 4; ++e) acc[n][e] = 0.f;
-  load(0, 0);
-  cp_async_commit();
   for (int k0 = 0, it = 0; k0 < a.K; k0 += 64, ++it) {
-    cp_async_wait<0>();
-    __syncthreads();
-    if (k0 + 64 < a.K) load((it + 1) & 1, k0 + 64);
+    cp_async_wait<HEADS_STAGES - 2>();
+    __syncthreads();  // this step has landed, and everyone has left the stage that is filled next
+    const int ahead = k0 + 64 * (HEADS_STAGES - 1);
+    if (ahead < a.K) {
+      load_w((it + HEADS_STAGES - 1) % HEADS_STAGES, ahead);
+      load_x((it + HEADS_STAGES - 1) % HEADS_STAGES, ahead);
+    }
     cp_async_commit();
-    const uint32_t sa = smem_u32(smem[it & 1][0]), sw = smem_u32(smem[it & 1][1]);
+    const uint32_t sa = base + (it % HEADS_STAGES) * C::STAGE, sw = sa + C::A_BYTES;
 #pragma unroll
     for (int k = 0; k < 4; ++k) {
       uint32_t qa[4];
       frag_a<64>(sa, warp * 16, k * 16, lane, qa);
 #pragma unroll
-      for (int n = 0; n < 4; ++n) {
+      for (int n = 0; n < NT / 16; ++n) {
         uint32_t kb[4];
         if (KN) frag_b_t<64>(sw, n * 16, k * 16, lane, kb);
         else frag_b<64>(sw, n * 16, k * 16, lane, kb);
@@ -198,7 +246,7 @@ __global__ void __launch_bounds__(128) heads_gemm_kernel(const HeadsArgs a) {
     uint16_t* dst = static_cast<uint16_t*>(a.out) + m * a.ldo + static_cast<int64_t>(h) * a.out_hs;
     const uint16_t* g = a.gate != nullptr ? static_cast<const uint16_t*>(a.gate) + m * a.ldg + static_cast<int64_t>(h) * a.gate_hs : nullptr;
 #pragma unroll
-    for (int n = 0; n < 8; ++n) {
+    for (int n = 0; n < NT / 8; ++n) {
       const int c = n0 + n * 8 + (lane & 3) * 2;
       if (c >= a.N) continue;
       float u = acc[n][2 * e], v = acc[n][2 * e + 1];
@@ -210,6 +258,14 @@ __global__ void __launch_bounds__(128) heads_gemm_kernel(const HeadsArgs a) {
       *reinterpret_cast<uint32_t*>(dst + c) = pack_bf16(u, v);
     }
   }
+}
+
+template <bool KN>
+int launch_heads(const HeadsArgs& a, dim3 grid, cudaStream_t s) {
+  static const cudaError_t set = cudaFuncSetAttribute(heads_gemm_kernel<KN>, cudaFuncAttributeMaxDynamicSharedMemorySize, CfgHeads<KN>::SMEM);
+  B2_CUDA(set);
+  B2_CUDA(b2_launch(heads_gemm_kernel<KN>, grid, dim3(128), CfgHeads<KN>::SMEM, s, a));
+  return B2_OK;
 }
 
 // fp32, CUDA cores: 64 x 64 outputs, 4 x 4 per thread
@@ -270,340 +326,445 @@ __global__ void __launch_bounds__(256) heads_gemm_f32_kernel(const HeadsArgs a) 
 }
 
 // ---------------------------------------------------------------------------
-// Absorbed attention.  16 MT rows (token, head) per CTA; 8 warps.  Scores: the warps share the tile's keys (and the MT row
-// groups); values: each warp owns DL / 8 columns of the latent for all rows.  Softmax weights pass through shared memory
-// as a sum of two bf16 numbers.  Key tiles are dealt to `splits` CTAs whose parts the last one to arrive combines.
+// Absorbed attention on tcgen05.  A CTA holds NR (token, head) rows and walks key tiles of 128 cached rows, which TMA brings
+// into shared memory as boxes of 128 keys x 64 columns.  Both products have the big operand on the 128-row side:
+//   scores   S^T [128 keys x NR]   = rows (K-major)           x Q^T
+//   outputs  O^T [128 dims x NR]  += latents^T (M contiguous) x P^T, one accumulator per 128 latent columns
+// from the same boxes.  Warps 0-3: softmax, a thread per key; the weights go back through shared memory as a sum of two bf16
+// numbers.  Warp 4: TMA.  Warp 5: MMA.  Key tiles are dealt to `splits` CTAs whose parts the last one to arrive combines.
 // ---------------------------------------------------------------------------
-constexpr int LAT_ROT = 64;           // columns kept for the rotated part
-constexpr int LAT_MAX_SPLITS = 64;
-constexpr int LAT_MAX_GROUPS = 65536;  // arrival counters at the front of the workspace
+constexpr int LT_KEYS = 128;                 // keys per tile
+constexpr int LT_BOX = LT_KEYS * 64 * 2;     // bytes of one box
+constexpr int LT_THREADS = 192;
+constexpr int LT_MAX_PAIRS = 4;              // latents up to 512 wide
+constexpr int LT_MAX_STAGES = 3;
+constexpr int LT_TMEM = 256;                 // S^T: NR columns, O^T: 4 NR
+constexpr int LT_MAX_SPLITS = 64;
+constexpr int LT_MAX_GROUPS = 65536;         // arrival counters at the front of the workspace
+constexpr uint64_t LT_LIMIT_NS = 1000000000ull;
+constexpr int LT_SMEM_MAX = 227 * 1024;
+constexpr float LT_RESCALE = 8.0f;           // the running maximum may be exceeded by 2^8 before the outputs are rescaled
 
-template <int DL, int MT>
-struct CfgLatent {
-  static constexpr int DK = DL + LAT_ROT;
-  static constexpr int ROWS = 16 * MT;
-  static constexpr int STAGE = BN * DK * 2;
-  static constexpr int Q_BYTES = ROWS * DK * 2;
-  static constexpr int P_BYTES = ROWS * BN * 2;
-  static constexpr int SMEM = Q_BYTES + 2 * STAGE + 2 * P_BYTES + 128;
-  static constexpr int PART = ROWS * (DL + 2);  // floats of one split's part
+struct LatentTcArgs {
+  uint16_t* out;
+  int64_t ldo;
+  const int32_t* block_tables;
+  int64_t bt_stride;
+  int block_size;
+  const int32_t* cu_q;
+  const int32_t* kv_len;
+  int heads, v_pad, boxes, rot;  // boxes: 64-column boxes of the latent; rot: 1 = there is a rotated part
+  int stages, row_tiles, splits;
+  float scale;
+  const float* sink;
+  int* counters;
+  float* part;  // [group][split][2 NR + NR * 128 pairs]: maxima, sums, outputs by row
+  B2Status* status;
 };
 
-// a row [lat_pad | rot_pad] into columns [0, lat_pad) and [DL, DL + rot_pad) of a tile row, zeros elsewhere; one warp per row
-template <int DL>
-__device__ __forceinline__ void load_latent_row(uint32_t tile, int r, const uint16_t* src, bool ok, int lat8, int rot8, int lane) {
-  constexpr int P = (DL + LAT_ROT) / 8;
+// v over the warp's 32 lanes, one result per column: lane l gets column l & (NR - 1).  Destroys v.
+template <int NR, typename Op>
+__device__ __forceinline__ float reduce_columns(float (&v)[NR], int lane, Op op) {
+  if (NR == 16) {
 #pragma unroll
-  for (int i = 0; i < (P + 31) / 32; ++i) {
-    const int p = lane + i * 32;
-    if (p >= P) break;
-    const bool rot = p >= DL / 8;
-    const bool in = ok && (rot ? p - DL / 8 < rot8 : p < lat8);
-    cp_async16(tile_addr<DL + LAT_ROT>(tile, r, p), in ? src + (rot ? lat8 + p - DL / 8 : p) * 8 : src, in);
+    for (int j = 0; j < NR; ++j) v[j] = op(v[j], __shfl_xor_sync(0xffffffffu, v[j], 16));
   }
+#pragma unroll
+  for (int o = NR / 2; o >= 1; o >>= 1) {
+    const bool upper = (lane & o) != 0;
+#pragma unroll
+    for (int j = 0; j < o; ++j) {
+      const float send = upper ? v[j] : v[j + o], keep = upper ? v[j + o] : v[j];
+      v[j] = op(keep, __shfl_xor_sync(0xffffffffu, send, o));
+    }
+  }
+  return v[0];
+}
+// all 128 softmax threads meet; true when every one brought true
+__device__ __forceinline__ bool softmax_meet(bool ok) {
+  uint32_t r;
+  asm volatile("{\n\t.reg .pred p, q;\n\tsetp.ne.u32 p, %1, 0;\n\tbarrier.cta.red.and.pred q, 1, 128, p;\n\tselp.u32 %0, 1, 0, q;\n\t}"
+               : "=r"(r) : "r"(static_cast<uint32_t>(ok)) : "memory");
+  return r != 0;
+}
+template <int NR>
+__device__ __forceinline__ void tmem_load(uint32_t addr, uint32_t (&r)[NR]) {
+  if constexpr (NR == 32) tmem_ld_32x32(addr, r);
+  else tmem_ld_32x16(addr, r);
+  tc_wait_ld();
 }
 
-template <int DL, int MT>
-__global__ void __launch_bounds__(256, 1) latent_attn_kernel(const AttnArgs a, int rot_pad, int row_tiles, int splits, int* counters, float* part) {
-  using C = CfgLatent<DL, MT>;
-  constexpr int DK = C::DK, ROWS = C::ROWS, KG = 8 / MT, WC = DL / 8;  // KG key groups; WC value columns of a warp
+template <int NR>
+__global__ void __launch_bounds__(LT_THREADS, 1)
+latent_tc_kernel(const __grid_constant__ CUtensorMap tm_lat, const __grid_constant__ CUtensorMap tm_rot, const __grid_constant__ CUtensorMap tm_ql,
+                 const __grid_constant__ CUtensorMap tm_qr, const LatentTcArgs a) {
   extern __shared__ unsigned char smem_raw[];
-  __shared__ float s_max[KG][ROWS], s_corr[ROWS], s_ml[ROWS][2];
-  __shared__ int s_last;
-  const uint32_t base = (smem_u32(smem_raw) + 127) & ~127u;
-  const uint32_t sq = base, skv = base + C::Q_BYTES, sp = skv + 2 * C::STAGE, sp_lo = sp + C::P_BYTES;
+  __shared__ __align__(8) uint64_t s_bars[2 * LT_MAX_STAGES * (LT_MAX_PAIRS + 1) + 4];
+  __shared__ float s_red[4][32], s_fac[LT_MAX_SPLITS * 32];
+  __shared__ uint32_t s_tmem;
+  __shared__ int s_abort, s_last;
+  volatile int* abort_flag = &s_abort;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  pdl_launch_dependents();
+  const int pairs = (a.boxes + 1) >> 1, stage_bytes = (2 * pairs + a.rot) * LT_BOX;
+  const uint32_t q_bytes = (a.boxes + a.rot) * NR * 128;
+  const uint32_t sq = (smem_u32(smem_raw) + 1023u) & ~1023u;
+  const uint32_t sp = sq + ((q_bytes + 1023u) & ~1023u);  // P: [hi, lo][two halves of 64 keys][NR rows of 128 bytes]
+  const uint32_t sk = sp + NR * 512;
+  const uint32_t bar_full = smem_u32(s_bars), bar_empty = bar_full + LT_MAX_STAGES * (LT_MAX_PAIRS + 1) * 8;
+  const uint32_t bar_q = bar_empty + LT_MAX_STAGES * (LT_MAX_PAIRS + 1) * 8, bar_s = bar_q + 8, bar_p = bar_q + 16, bar_o = bar_q + 24;
+  const auto full = [&](int st, int i) { return bar_full + (st * (LT_MAX_PAIRS + 1) + i) * 8; };
+  const auto empty = [&](int st, int i) { return bar_empty + (st * (LT_MAX_PAIRS + 1) + i) * 8; };
+  if (threadIdx.x == 0) {
+    for (int i = 0; i < LT_MAX_STAGES * (LT_MAX_PAIRS + 1); ++i) {
+      mbar_init(bar_full + i * 8, 1);
+      mbar_init(bar_empty + i * 8, 1);
+    }
+    mbar_init(bar_q, 1);
+    mbar_init(bar_s, 1);
+    mbar_init(bar_p, 4);
+    mbar_init(bar_o, 1);
+    s_abort = 0;
+    mbar_fence_init();
+    tma_prefetch_desc(&tm_lat);
+    tma_prefetch_desc(&tm_rot);
+    tma_prefetch_desc(&tm_ql);
+    tma_prefetch_desc(&tm_qr);
+  }
+  if (warp == 5) {
+    tmem_alloc(smem_u32(&s_tmem), LT_TMEM);
+    tmem_relinquish();
+  }
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tm_s = s_tmem, tm_o = s_tmem + NR;
+  pdl_launch_dependents();  // only now: a later kernel must not take the tensor memory that a CTA of this one still needs
   pdl_wait();
-  const int b = blockIdx.z, split = blockIdx.x, r_base = blockIdx.y * ROWS;
+
+  const int b = blockIdx.z, split = blockIdx.x, r_base = blockIdx.y * NR;
   const int row0 = a.cu_q ? a.cu_q[b] : b;
   const int n_q = a.cu_q ? a.cu_q[b + 1] - row0 : 1;
-  const int rows = n_q * a.nq;
-  if (r_base >= rows) return;
-  const int nrows = min(ROWS, rows - r_base);
-  const int klen = a.kv_len[b];
-  uint16_t* out = static_cast<uint16_t*>(a.out);
-  const auto out_row = [&](int r) {
-    const int gr = r_base + r, tok = gr / a.nq;
-    return out + (row0 + tok) * a.ldo + static_cast<int64_t>(gr - tok * a.nq) * a.v_pad;
-  };
-  if (klen <= 0) {  // padded row of a decode graph
-    if (split == 0)
-      for (int i = threadIdx.x; i < nrows * a.v_pad; i += 256) out_row(i / a.v_pad)[i % a.v_pad] = 0;
-    return;
-  }
+  const int rows = n_q * a.heads, klen = a.kv_len[b];
+  const int nrows = max(0, min(NR, rows - r_base));
   const int first_pos = klen - n_q;
-  const int pmin = first_pos + r_base / a.nq, pmax = first_pos + (r_base + nrows - 1) / a.nq;
-  const int total = pmax / BN + 1, per = (total + splits - 1) / splits;
+  const int pmin = first_pos + r_base / a.heads, pmax = first_pos + (r_base + max(nrows, 1) - 1) / a.heads;
+  const int total = nrows > 0 && klen > 0 ? pmax / LT_KEYS + 1 : 0, per = (total + a.splits - 1) / a.splits;
   const int t0 = split * per, t1 = min(total, t0 + per);
-  const int lat8 = a.v_pad >> 3, rot8 = rot_pad >> 3;
-  const int32_t* bt = a.block_tables + b * a.bt_stride;
-  const uint16_t* cache = static_cast<const uint16_t*>(a.k_cache);
-  auto load_tile = [&](int tile, uint32_t dst) {
-#pragma unroll 2
-    for (int r = warp; r < BN; r += 8) {
-      const int j = tile * BN + r;
-      const bool ok = j <= pmax;
-      const int blk = ok ? j / a.block_size : 0;
-      const int64_t slot = ok ? static_cast<int64_t>(__ldg(bt + blk)) * a.block_size + (j - blk * a.block_size) : 0;
-      load_latent_row<DL>(dst, r, cache + slot * a.k_row, ok, lat8, rot8, lane);
-    }
+  const auto out_row = [&](int r) {
+    const int gr = r_base + r, tok = gr / a.heads;
+    return a.out + (row0 + tok) * a.ldo + static_cast<int64_t>(gr - tok * a.heads) * a.v_pad;
   };
-  for (int r = warp; r < ROWS; r += 8) {
-    const int gr = r_base + r, tok = r < nrows ? gr / a.nq : 0, h = r < nrows ? gr - tok * a.nq : 0;
-    load_latent_row<DL>(sq, r, static_cast<const uint16_t*>(a.q) + (row0 + tok) * a.ldq + static_cast<int64_t>(h) * a.qk_pad, r < nrows, lat8, rot8, lane);
-  }
-  if (t0 < t1) load_tile(t0, skv);
-  cp_async_commit();
-  const int mt = warp % MT, kg = warp / MT;  // this warp's rows and keys of the score tile
-  int pos[2];
-#pragma unroll
-  for (int e = 0; e < 2; ++e) pos[e] = first_pos + (r_base + min(mt * 16 + (lane >> 2) + e * 8, nrows - 1)) / a.nq;
-  const float scale = a.scale * LOG2E;
-  float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
-  float o[MT][WC / 8][4];
-#pragma unroll
-  for (int i = 0; i < MT; ++i)
-#pragma unroll
-    for (int n = 0; n < WC / 8; ++n)
-#pragma unroll
-      for (int e = 0; e < 4; ++e) o[i][n][e] = 0.f;
-  for (int t = t0; t < t1; ++t) {
-    const uint32_t sk = skv + ((t - t0) & 1) * C::STAGE;
-    cp_async_wait<0>();
-    __syncthreads();  // this tile has landed, and everyone has left the stage that is filled next
-    if (t + 1 < t1) load_tile(t + 1, skv + ((t + 1 - t0) & 1) * C::STAGE);
-    cp_async_commit();
-    // scores of 16 rows x 8 MT keys, even and odd steps of the product in separate accumulators
-    float s[2][MT][4];
-#pragma unroll
-    for (int p = 0; p < 2; ++p)
-#pragma unroll
-      for (int n = 0; n < MT; ++n)
-#pragma unroll
-        for (int e = 0; e < 4; ++e) s[p][n][e] = 0.f;
-#pragma unroll 4
-    for (int k = 0; k < DK / 32; ++k) {
-      uint32_t qa[2][4];
-      frag_a<DK>(sq, mt * 16, k * 32, lane, qa[0]);
-      frag_a<DK>(sq, mt * 16, k * 32 + 16, lane, qa[1]);
-      if (MT == 1) {
-        uint32_t kb[4];  // 8 keys, 32 columns
-        ldsm_x4(tile_addr<DK>(sk, kg * 8 + (lane & 7), k * 4 + (lane >> 3)), kb);
-        mma16816(s[0][0], qa[0], kb[0], kb[1]);
-        mma16816(s[1][0], qa[1], kb[2], kb[3]);
-      } else {
-#pragma unroll
-        for (int p = 0; p < 2; ++p) {
-          uint32_t kb[4];
-          frag_b<DK>(sk, kg * 16, k * 32 + p * 16, lane, kb);
-          mma16816(s[p][0], qa[p], kb[0], kb[1]);
-          mma16816(s[p][MT - 1], qa[p], kb[2], kb[3]);
+
+  if (warp == 4) {
+    // ---------------- TMA ----------------
+    if (lane == 0 && t0 < t1) {
+      mbar_arrive_expect_tx(bar_q, q_bytes);
+      const int qrow = row0 * a.heads + r_base;
+      for (int i = 0; i < a.boxes; ++i) tma_load_2d(sq + i * NR * 128, &tm_ql, bar_q, i * 64, qrow, kEvictFirst);
+      if (a.rot) tma_load_2d(sq + a.boxes * NR * 128, &tm_qr, bar_q, 0, qrow, kEvictFirst);
+      int st = 0;
+      uint32_t phase = 0;
+      const int per_block = a.block_size / LT_KEYS;
+      bool ok = true;
+      for (int t = t0; ok && t < t1; ++t) {
+        const int slot = a.block_tables[b * a.bt_stride + t / per_block] * a.block_size + (t % per_block) * LT_KEYS;
+        const uint32_t base = sk + st * stage_bytes;
+        if (a.rot) {  // free first, read first
+          if (!(ok = mbar_wait(empty(st, pairs), phase ^ 1, abort_flag, LT_LIMIT_NS, B2_WAIT_SMEM_EMPTY))) break;
+          mbar_arrive_expect_tx(full(st, pairs), LT_BOX);
+          tma_load_2d(base + 2 * pairs * LT_BOX, &tm_rot, full(st, pairs), 0, slot, kEvictNormal);
         }
+        for (int p = 0; p < pairs; ++p) {
+          if (!(ok = mbar_wait(empty(st, p), phase ^ 1, abort_flag, LT_LIMIT_NS, B2_WAIT_SMEM_EMPTY))) break;
+          const int n = min(2, a.boxes - 2 * p);
+          mbar_arrive_expect_tx(full(st, p), n * LT_BOX);
+          for (int i = 0; i < n; ++i) tma_load_2d(base + (2 * p + i) * LT_BOX, &tm_lat, full(st, p), (2 * p + i) * 64, slot, kEvictNormal);
+        }
+        if (++st == a.stages) { st = 0; phase ^= 1; }
       }
     }
-    const int j0 = t * BN + kg * 8 * MT;
-    const bool masked = j0 + 8 * MT - 1 > pmin;
-    float mx[2] = {-INFINITY, -INFINITY};
+  } else if (warp == 5) {
+    // ---------------- MMA ----------------
+    if (lane == 0 && t0 < t1) {
+      constexpr uint32_t idesc_s = umma_idesc_bf16(NR), idesc_o = umma_idesc_bf16(NR) | UMMA_A_MN;
+      int st = 0;
+      uint32_t phase = 0;
+      bool ok = mbar_wait(bar_q, 0, abort_flag, LT_LIMIT_NS, B2_WAIT_SMEM_FULL);
+      for (int t = t0; ok && t < t1; ++t) {
+        const uint32_t base = sk + st * stage_bytes;
+        const auto scores = [&](int box, bool first) {
+          const uint64_t dk = umma_smem_desc(base + box * LT_BOX), dq = umma_smem_desc(sq + (box < a.boxes ? box : a.boxes) * NR * 128);
 #pragma unroll
-    for (int n = 0; n < MT; ++n)
+          for (int k = 0; k < 4; ++k) umma_bf16(tm_s, dk + 2 * k, dq + 2 * k, idesc_s, (first && k == 0) ? 0u : 1u);
+        };
+        bool first = true;
+        if (a.rot) {
+          if (!(ok = mbar_wait(full(st, pairs), phase, abort_flag, LT_LIMIT_NS, B2_WAIT_SMEM_FULL))) break;
+          tc_fence_after();
+          scores(2 * pairs, true);
+          first = false;
+          umma_commit(empty(st, pairs));
+        }
+        for (int p = 0; p < pairs; ++p) {
+          if (!(ok = mbar_wait(full(st, p), phase, abort_flag, LT_LIMIT_NS, B2_WAIT_SMEM_FULL))) break;
+          tc_fence_after();
+          for (int i = 2 * p; i < min(a.boxes, 2 * p + 2); ++i) {
+            scores(i, first);
+            first = false;
+          }
+        }
+        if (!ok) break;
+        umma_commit(bar_s);  // also says that the outputs of the previous tile are complete
+        if (!(ok = mbar_wait(bar_p, (t - t0) & 1, abort_flag, LT_LIMIT_NS, B2_WAIT_TMEM_EMPTY))) break;
+        tc_fence_after();
+        for (int p = 0; p < pairs; ++p) {
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        float v = (s[0][n][e] + s[1][n][e]) * scale;
-        if (masked && j0 + n * 8 + (lane & 3) * 2 + (e & 1) > pos[e >> 1]) v = -INFINITY;
-        s[0][n][e] = v;
-        mx[e >> 1] = fmaxf(mx[e >> 1], v);
+          for (int half = 0; half < 2; ++half)  // the weights' leading and trailing parts
+#pragma unroll
+            for (int k = 0; k < LT_KEYS / 16; ++k) {
+              const uint64_t dv = umma_smem_desc_mn(base + 2 * p * LT_BOX + k * 2048, LT_BOX);
+              const uint64_t dp = umma_smem_desc(sp + half * NR * 256 + (k >> 2) * NR * 128) + 2 * (k & 3);
+              umma_bf16(tm_o + p * NR, dv, dp, idesc_o, (t > t0 || half > 0 || k > 0) ? 1u : 0u);
+            }
+          umma_commit(empty(st, p));
+        }
+        if (++st == a.stages) { st = 0; phase ^= 1; }
       }
-#pragma unroll
-    for (int e = 0; e < 2; ++e) {
-      mx[e] = fmaxf(mx[e], __shfl_xor_sync(0xffffffffu, mx[e], 1));
-      mx[e] = fmaxf(mx[e], __shfl_xor_sync(0xffffffffu, mx[e], 2));
-      if ((lane & 3) == 0) s_max[kg][mt * 16 + (lane >> 2) + e * 8] = mx[e];
+      if (ok) umma_commit(bar_o);
     }
-    __syncthreads();
+  } else {
+    // ---------------- softmax: thread = key of the tile ----------------
+    const uint32_t lanes = static_cast<uint32_t>(warp * 32) << 16;
+    const int col = lane & (NR - 1);  // the row whose maximum, sum and factors this lane keeps
+    const float scale = a.scale * LOG2E;
+    float m_col = -INFINITY;
+    float l[NR];
 #pragma unroll
-    for (int e = 0; e < 2; ++e) {
-      const int r = mt * 16 + (lane >> 2) + e * 8;
-      float m_new = m[e];
+    for (int r = 0; r < NR; ++r) l[r] = 0.f;
+    bool ok = true;
+    for (int t = t0; ok && t < t1; ++t) {
+      ok = mbar_wait(bar_s, (t - t0) & 1, abort_flag, LT_LIMIT_NS, B2_WAIT_TMEM_FULL);
+      __syncwarp();
+      tc_fence_after();
+      uint32_t raw[NR];
+      tmem_load<NR>(tm_s + lanes, raw);
+      float v[NR], w[NR];
+      const int j = t * LT_KEYS + threadIdx.x;
+      const bool masked = t * LT_KEYS + LT_KEYS - 1 > pmin;
 #pragma unroll
-      for (int i = 0; i < KG; ++i) m_new = fmaxf(m_new, s_max[i][r]);
-      const float ref = m_new == -INFINITY ? 0.f : m_new;
-      const float corr = fast_exp2(m[e] - ref);
-      m[e] = m_new;
-      if (kg == 0 && (lane & 3) == 0) s_corr[r] = corr;
-      float sum = 0.f;
+      for (int r = 0; r < NR; ++r) {
+        v[r] = __uint_as_float(raw[r]) * scale;
+        if (masked && j > first_pos + (r_base + min(r, nrows - 1)) / a.heads) v[r] = -INFINITY;
+        w[r] = v[r];
+      }
+      const float mx = reduce_columns<NR>(w, lane, [](float x, float y) { return fmaxf(x, y); });
+      s_red[warp][lane] = mx;
+      if (!(ok = softmax_meet(ok))) break;
+      const float m_tile = fmaxf(fmaxf(s_red[0][col], s_red[1][col]), fmaxf(s_red[2][col], s_red[3][col]));
+      const bool grow = m_tile > m_col + LT_RESCALE || m_col == -INFINITY;
+      const float m_new = grow ? fmaxf(m_tile, m_col) : m_col;
+      const float corr = grow && m_col > -INFINITY ? fast_exp2(m_col - m_new) : 1.0f;
+      if (__any_sync(0xffffffffu, corr != 1.0f)) {  // the same in all four warps; never in the first tile
 #pragma unroll
-      for (int n = 0; n < MT; ++n) {
-        const float x = fast_exp2(s[0][n][2 * e] - ref), y = fast_exp2(s[0][n][2 * e + 1] - ref);
-        sum += x + y;
+        for (int r = 0; r < NR; ++r) l[r] *= __shfl_sync(0xffffffffu, corr, r);
+        for (int p = 0; p < pairs; ++p) {
+          tmem_load<NR>(tm_o + p * NR + lanes, raw);
+#pragma unroll
+          for (int r = 0; r < NR; ++r) raw[r] = __float_as_uint(__uint_as_float(raw[r]) * __shfl_sync(0xffffffffu, corr, r));
+#pragma unroll
+          for (int h = 0; h < NR / 16; ++h) {
+            uint32_t part[16];
+#pragma unroll
+            for (int i = 0; i < 16; ++i) part[i] = raw[16 * h + i];
+            tmem_st_32x16(tm_o + p * NR + 16 * h + lanes, part);
+          }
+        }
+        tc_wait_st();
+      }
+      m_col = m_new;
+      const float ref = m_col == -INFINITY ? 0.f : m_col;
+#pragma unroll
+      for (int r = 0; r < NR; ++r) {
+        v[r] = fast_exp2(v[r] - __shfl_sync(0xffffffffu, ref, r));
+        l[r] += v[r];
+      }
+      // neighbours exchange: an even lane stores rows r of keys (lane, lane + 1), an odd one rows r + 1
+      const int odd = lane & 1, key2 = (warp & 1) * 32 + (lane & ~1);  // first of the two keys inside the half tile
+      const uint32_t at = sp + (warp >> 1) * NR * 128 + (key2 & 7) * 2;
+#pragma unroll
+      for (int r = 0; r < NR; r += 2) {
+        const float other = __shfl_xor_sync(0xffffffffu, odd ? v[r] : v[r + 1], 1);
+        const int rr = r + odd;
         uint32_t hi, lo;
-        split_bf16(x, y, hi, lo);
-        const uint32_t at = tile_addr<64>(0, r, kg * MT + n) + (lane & 3) * 4;
-        asm volatile("st.shared.u32 [%0], %1;" ::"r"(sp + at), "r"(hi) : "memory");
-        asm volatile("st.shared.u32 [%0], %1;" ::"r"(sp_lo + at), "r"(lo) : "memory");
+        split_bf16(odd ? other : v[r], odd ? v[r + 1] : other, hi, lo);
+        const uint32_t dst = at + rr * 128 + (((key2 >> 3) ^ (rr & 7)) << 4);
+        asm volatile("st.shared.u32 [%0], %1;" ::"r"(dst), "r"(hi) : "memory");
+        asm volatile("st.shared.u32 [%0], %1;" ::"r"(dst + NR * 256), "r"(lo) : "memory");
       }
-      l[e] = fmaf(l[e], corr, sum);  // this lane's keys
+      fence_proxy_async();
+      tc_fence_before();
+      __syncwarp();
+      if (lane == 0) mbar_arrive(bar_p);
     }
-    __syncthreads();
-#pragma unroll
-    for (int i = 0; i < MT; ++i) {
-      const float c0 = s_corr[i * 16 + (lane >> 2)], c1 = s_corr[i * 16 + (lane >> 2) + 8];
-#pragma unroll
-      for (int n = 0; n < WC / 8; ++n) {
-        o[i][n][0] *= c0; o[i][n][1] *= c0; o[i][n][2] *= c1; o[i][n][3] *= c1;
-      }
-    }
-#pragma unroll
-    for (int k = 0; k < BN / 16; ++k) {
-      uint32_t hi[MT][4], lo[MT][4];
-#pragma unroll
-      for (int i = 0; i < MT; ++i) {
-        frag_a<64>(sp, i * 16, k * 16, lane, hi[i]);
-        frag_a<64>(sp_lo, i * 16, k * 16, lane, lo[i]);
-      }
-#pragma unroll
-      for (int n = 0; n < WC / 16; ++n) {
-        uint32_t vb[4];
-        frag_b_t<DK>(sk, warp * WC + n * 16, k * 16, lane, vb);
-#pragma unroll
-        for (int i = 0; i < MT; ++i) {
-          mma16816(o[i][2 * n], hi[i], vb[0], vb[1]);
-          mma16816(o[i][2 * n + 1], hi[i], vb[2], vb[3]);
-          mma16816(o[i][2 * n], lo[i], vb[0], vb[1]);
-          mma16816(o[i][2 * n + 1], lo[i], vb[2], vb[3]);
-        }
-      }
-    }
-  }
-  cp_async_wait<0>();
-  __syncthreads();
-#pragma unroll
-  for (int e = 0; e < 2; ++e) {
-    const int r = mt * 16 + (lane >> 2) + e * 8;
-    l[e] += __shfl_xor_sync(0xffffffffu, l[e], 1);
-    l[e] += __shfl_xor_sync(0xffffffffu, l[e], 2);
-    if ((lane & 3) == 0) s_max[kg][r] = l[e];
-    if (kg == 0 && (lane & 3) == 0) s_ml[r][0] = m[e];
-  }
-  __syncthreads();
-  if (threadIdx.x < ROWS) {
-    float sum = 0.f;
-#pragma unroll
-    for (int i = 0; i < KG; ++i) sum += s_max[i][threadIdx.x];
-    s_ml[threadIdx.x][1] = sum;
-  }
-  __syncthreads();
-  const int group = b * row_tiles + blockIdx.y;
-  float* my = part + (static_cast<int64_t>(group) * splits + split) * C::PART;
-#pragma unroll
-  for (int i = 0; i < MT; ++i)
-#pragma unroll
-    for (int e = 0; e < 2; ++e) {
-      const int r = i * 16 + (lane >> 2) + e * 8;
-      if (r >= nrows) continue;
-      if (splits == 1) {
-        float f = 1.0f, sum = s_ml[r][1];
-        if (a.sink != nullptr) {
-          const float mr = s_ml[r][0], sk = a.sink[(r_base + r) % a.nq] * LOG2E, m_new = fmaxf(mr, sk);
-          f = fast_exp2(mr - m_new);
-          sum = sum * f + fast_exp2(sk - m_new);
-        }
-        f /= sum;
-        uint16_t* dst = out_row(r);
-#pragma unroll
-        for (int n = 0; n < WC / 8; ++n) {
-          const int c = warp * WC + n * 8 + (lane & 3) * 2;
-          if (c < a.v_pad) *reinterpret_cast<uint32_t*>(dst + c) = pack_bf16(o[i][n][2 * e] * f, o[i][n][2 * e + 1] * f);
-        }
+    if (ok && t0 < t1) ok = mbar_wait(bar_o, 0, abort_flag, LT_LIMIT_NS, B2_WAIT_TMEM_FULL);
+    __syncwarp();
+    tc_fence_after();
+    const float lw = reduce_columns<NR>(l, lane, [](float x, float y) { return x + y; });
+    s_red[warp][lane] = lw;
+    ok = softmax_meet(ok);
+    if (ok && nrows > 0) {
+      const float l_col = s_red[0][col] + s_red[1][col] + s_red[2][col] + s_red[3][col];
+      const int group = b * a.row_tiles + blockIdx.y;
+      const int64_t part_floats = 2 * NR + static_cast<int64_t>(NR) * 128 * pairs;
+      float* my = a.part + (static_cast<int64_t>(group) * a.splits + split) * part_floats;
+      if (klen <= 0) {  // padded row of a decode graph
+        if (split == 0)
+          for (int i = threadIdx.x; i < nrows * a.v_pad; i += 128) out_row(i / a.v_pad)[i % a.v_pad] = 0;
       } else {
+        float f = 1.0f;
+        if (a.splits == 1) {
+          float sum = l_col;
+          if (a.sink != nullptr) {
+            const float sk_ = a.sink[(r_base + col) % a.heads] * LOG2E, m_new = fmaxf(m_col, sk_);
+            f = fast_exp2(m_col - m_new);
+            sum = sum * f + fast_exp2(sk_ - m_new);
+          }
+          f /= sum;
+        } else if (warp == 0 && lane < nrows && lane < NR) {
+          my[lane] = m_col;
+          my[NR + lane] = l_col;
+        }
+        if (t0 < t1) {
+          for (int p = 0; p < pairs; ++p) {
+            uint32_t raw[NR];
+            tmem_load<NR>(tm_o + p * NR + lanes, raw);
+            const int dim = p * 128 + threadIdx.x;
 #pragma unroll
-        for (int n = 0; n < WC / 8; ++n)
-          *reinterpret_cast<float2*>(my + 2 * ROWS + r * DL + warp * WC + n * 8 + (lane & 3) * 2) = make_float2(o[i][n][2 * e], o[i][n][2 * e + 1]);
+            for (int r = 0; r < NR; ++r) {
+              const float fr = __shfl_sync(0xffffffffu, f, r);
+              if (r < nrows) {
+                if (a.splits > 1) my[2 * NR + r * 128 * pairs + dim] = __uint_as_float(raw[r]);
+                else if (dim < a.v_pad) out_row(r)[dim] = from_float<uint16_t>(__uint_as_float(raw[r]) * fr);
+              }
+            }
+          }
+        }
+        if (a.splits > 1) {
+          __threadfence();
+          softmax_meet(true);
+          if (threadIdx.x == 0) s_last = atomicAdd(a.counters + group, 1) == a.splits - 1;
+          softmax_meet(true);
+          if (s_last) {
+            if (threadIdx.x == 0) a.counters[group] = 0;
+            __threadfence();
+            const float* all = a.part + static_cast<int64_t>(group) * a.splits * part_floats;
+            if (static_cast<int>(threadIdx.x) < nrows) {
+              const int r = threadIdx.x;
+              const float sk_ = a.sink != nullptr ? a.sink[(r_base + r) % a.heads] * LOG2E : -INFINITY;
+              float mt = sk_;
+              for (int s = 0; s < a.splits; ++s) mt = fmaxf(mt, ld_cg_f32(all + s * part_floats + r));
+              float lt = fast_exp2(sk_ - mt);
+              for (int s = 0; s < a.splits; ++s) {
+                const float ms = ld_cg_f32(all + s * part_floats + r);
+                const float fs = ms > -INFINITY ? fast_exp2(ms - mt) : 0.f;
+                s_fac[s * NR + r] = fs;
+                if (fs > 0.f) lt += fs * ld_cg_f32(all + s * part_floats + NR + r);
+              }
+              for (int s = 0; s < a.splits; ++s) s_fac[s * NR + r] /= lt;
+            }
+            softmax_meet(true);
+            const int vecs = a.v_pad >> 2;
+            for (int i = threadIdx.x; i < nrows * vecs; i += 128) {
+              const int r = i / vecs, c = (i - r * vecs) * 4;
+              float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 4
+              for (int s = 0; s < a.splits; ++s) {
+                const float fs = s_fac[s * NR + r];
+                if (fs == 0.f) continue;  // a split without keys for this row may hold anything
+                const uint4 q = ld_cg_v4(all + s * part_floats + 2 * NR + r * 128 * pairs + c);
+                acc.x += fs * __uint_as_float(q.x); acc.y += fs * __uint_as_float(q.y);
+                acc.z += fs * __uint_as_float(q.z); acc.w += fs * __uint_as_float(q.w);
+              }
+              *reinterpret_cast<uint2*>(out_row(r) + c) = make_uint2(pack_bf16(acc.x, acc.y), pack_bf16(acc.z, acc.w));
+            }
+          }
+        }
       }
     }
-  if (splits == 1) return;
-  if (threadIdx.x < nrows) {
-    my[threadIdx.x] = s_ml[threadIdx.x][0];
-    my[ROWS + threadIdx.x] = s_ml[threadIdx.x][1];
   }
-  __threadfence();
+  __syncwarp();
+  tc_fence_before();
   __syncthreads();
-  if (threadIdx.x == 0) s_last = atomicAdd(counters + group, 1) == splits - 1;
-  __syncthreads();
-  if (!s_last) return;
-  if (threadIdx.x == 0) counters[group] = 0;
-  __threadfence();
-  const float* all = part + static_cast<int64_t>(group) * splits * C::PART;
-  float* s_f = reinterpret_cast<float*>(smem_raw);  // [splits][ROWS] factors of the parts
-  if (threadIdx.x < nrows) {
-    const int r = threadIdx.x;
-    const float sk = a.sink != nullptr ? a.sink[(r_base + r) % a.nq] * LOG2E : -INFINITY;
-    float mt_ = sk;
-    for (int s = 0; s < splits; ++s) mt_ = fmaxf(mt_, ld_cg_f32(all + static_cast<int64_t>(s) * C::PART + r));
-    float lt = fast_exp2(sk - mt_);
-    for (int s = 0; s < splits; ++s) {
-      const float ms = ld_cg_f32(all + static_cast<int64_t>(s) * C::PART + r);
-      const float f = ms > -INFINITY ? fast_exp2(ms - mt_) : 0.f;
-      s_f[s * ROWS + r] = f;
-      if (f > 0.f) lt += f * ld_cg_f32(all + static_cast<int64_t>(s) * C::PART + ROWS + r);
-    }
-    for (int s = 0; s < splits; ++s) s_f[s * ROWS + r] /= lt;
+  tc_fence_after();
+  if (s_abort) {  // let bulk copies that may still be in flight land before the CTA leaves
+    for (int i = 0; i < 100; ++i) __nanosleep(2000);
+    if (threadIdx.x == 0) report_timeout(a.status, s_abort);
   }
-  __syncthreads();
-  for (int idx = threadIdx.x; idx < nrows * (DL / 4); idx += 256) {
-    const int r = idx / (DL / 4), c = (idx % (DL / 4)) * 4;
-    if (c >= a.v_pad) continue;
-    float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
-    for (int s = 0; s < splits; ++s) {
-      const float f = s_f[s * ROWS + r];
-      if (f == 0.f) continue;  // a split without keys for this row may hold anything
-      const uint4 v = ld_cg_v4(all + static_cast<int64_t>(s) * C::PART + 2 * ROWS + r * DL + c);
-      acc.x += f * __uint_as_float(v.x); acc.y += f * __uint_as_float(v.y);
-      acc.z += f * __uint_as_float(v.z); acc.w += f * __uint_as_float(v.w);
-    }
-    *reinterpret_cast<uint2*>(out_row(r) + c) = make_uint2(pack_bf16(acc.x, acc.y), pack_bf16(acc.z, acc.w));
-  }
+  if (warp == 5) tmem_dealloc(s_tmem, LT_TMEM);
 }
 
-bool latent_tiled(int dtype, int lat_pad, int rot_pad) { return dtype == B2_DT_BF16 && lat_pad <= 512 && rot_pad <= LAT_ROT; }
-int latent_width(int lat_pad) { return lat_pad <= 128 ? 128 : lat_pad <= 256 ? 256 : 512; }
-
 struct LatentPlan {
-  int rows, row_tiles, splits;
+  int rows, row_tiles, splits, boxes, rot, pairs, stages, smem;
   int64_t groups, bytes;
 };
-// Rows per CTA and how many CTAs share a group's key tiles: as few rounds of one CTA per SM as possible, counting a part's
-// combine as about two tiles.
-LatentPlan latent_plan(int B, int max_q, int max_kv, int heads, int lat_pad) {
+bool latent_tiled(int dtype, int block_size, int lat_pad, int rot_pad) {
+  return dtype == B2_DT_BF16 && lat_pad <= 128 * LT_MAX_PAIRS && rot_pad <= 64 && block_size % LT_KEYS == 0;
+}
+// Rows per CTA, tiles in shared memory, and how many CTAs share a group's key tiles: as few rounds of one CTA per SM as
+// possible, where a CTA's start and end cost about three tiles and a combine one more.
+LatentPlan latent_plan(int B, int max_q, int max_kv, int heads, int lat_pad, int rot_pad) {
   LatentPlan p{};
   const int64_t all = static_cast<int64_t>(max_q) * heads;
   p.rows = all > 16 ? 32 : 16;
-  p.row_tiles = static_cast<int>((all + p.rows - 1) / p.rows);
+  p.row_tiles = static_cast<int>(std::min<int64_t>((all + p.rows - 1) / p.rows, INT_MAX));
+  p.boxes = (lat_pad + 63) / 64;
+  p.rot = rot_pad > 0;
+  p.pairs = (p.boxes + 1) / 2;
+  const int fixed = 1024 + (((p.boxes + p.rot) * p.rows * 128 + 1023) & ~1023) + p.rows * 512 + 12 * 1024 /* static */;
+  const int stage = (2 * p.pairs + p.rot) * LT_BOX;
+  p.stages = std::max(1, std::min(LT_MAX_STAGES, (LT_SMEM_MAX - fixed) / stage));
+  p.smem = fixed - 12 * 1024 + p.stages * stage;
   p.groups = static_cast<int64_t>(B) * p.row_tiles;
-  const int64_t tiles = std::max<int64_t>(1, (static_cast<int64_t>(max_kv) + BN - 1) / BN);
+  const int64_t tiles = std::max<int64_t>(1, (static_cast<int64_t>(max_kv) + LT_KEYS - 1) / LT_KEYS);
   p.splits = 1;
-  if (p.groups <= LAT_MAX_GROUPS && p.groups < 4 * 148) {
+  if (p.groups <= LT_MAX_GROUPS && p.groups < 4 * 148) {
     int64_t best = INT64_MAX;
-    for (int s = 1; s <= std::min<int64_t>(LAT_MAX_SPLITS, tiles); ++s) {
-      const int64_t cost = ((p.groups * s + 147) / 148) * ((tiles + s - 1) / s + 1 + (s > 1 ? 2 : 0)) + s / 8;
+    for (int s = 1; s <= std::min<int64_t>(LT_MAX_SPLITS, tiles); ++s) {
+      const int64_t cost = ((p.groups * s + 147) / 148) * (8 * ((tiles + s - 1) / s) + 24 + (s > 1 ? 8 : 0)) + s;
       if (cost < best) {
         best = cost;
         p.splits = s;
       }
     }
   }
-  p.bytes = p.splits > 1 ? LAT_MAX_GROUPS * 4ll + p.groups * p.splits * p.rows * (latent_width(lat_pad) + 2) * 4ll : 0;
+  p.bytes = p.splits > 1 ? LT_MAX_GROUPS * 4ll + p.groups * p.splits * p.rows * (2ll + 128 * p.pairs) * 4 : 0;
   return p;
 }
 
-template <int DL, int MT>
-int launch_latent(const AttnArgs& a, int rot_pad, const LatentPlan& p, void* ws, cudaStream_t s) {
-  using C = CfgLatent<DL, MT>;
-  static const cudaError_t set = cudaFuncSetAttribute(latent_attn_kernel<DL, MT>, cudaFuncAttributeMaxDynamicSharedMemorySize, C::SMEM);
+template <int NR>
+int launch_latent(const b2_ctx* ctx, const AttnArgs& a, int64_t slots, int64_t q_rows, int rot_pad, const LatentPlan& p, void* ws, cudaStream_t s) {
+  static const cudaError_t set = cudaFuncSetAttribute(latent_tc_kernel<NR>, cudaFuncAttributeMaxDynamicSharedMemorySize, LT_SMEM_MAX - 12 * 1024);
   B2_CUDA(set);
-  float* part = ws != nullptr ? reinterpret_cast<float*>(static_cast<unsigned char*>(ws) + LAT_MAX_GROUPS * 4ll) : nullptr;
-  B2_CUDA(b2_launch(latent_attn_kernel<DL, MT>, dim3(p.splits, p.row_tiles, a.B), dim3(256), C::SMEM, s, a, rot_pad, p.row_tiles, p.splits,
-                    static_cast<int*>(ws), part));
+  CUtensorMap maps[4];
+  const uint16_t* cache = static_cast<const uint16_t*>(a.k_cache);
+  const uint16_t* q = static_cast<const uint16_t*>(a.q);
+  int rc = encode_tmap_2d(&maps[0], cache, a.v_pad, slots, a.k_row, 64, LT_KEYS);
+  if (rc == B2_OK) rc = encode_tmap_2d(&maps[2], q, a.v_pad, q_rows, a.qk_pad, 64, NR);
+  if (rc == B2_OK && p.rot) rc = encode_tmap_2d(&maps[1], cache + a.v_pad, rot_pad, slots, a.k_row, 64, LT_KEYS);
+  if (rc == B2_OK && p.rot) rc = encode_tmap_2d(&maps[3], q + a.v_pad, rot_pad, q_rows, a.qk_pad, 64, NR);
+  if (rc != B2_OK) return rc;
+  if (!p.rot) {
+    maps[1] = maps[0];
+    maps[3] = maps[2];
+  }
+  LatentTcArgs t{};
+  t.out = static_cast<uint16_t*>(a.out); t.ldo = a.ldo; t.block_tables = a.block_tables; t.bt_stride = a.bt_stride; t.block_size = a.block_size;
+  t.cu_q = a.cu_q; t.kv_len = a.kv_len; t.heads = a.nq; t.v_pad = a.v_pad; t.boxes = p.boxes; t.rot = p.rot; t.stages = p.stages;
+  t.row_tiles = p.row_tiles; t.splits = p.splits; t.scale = a.scale; t.sink = a.sink;
+  t.counters = static_cast<int*>(ws);
+  t.part = ws != nullptr ? reinterpret_cast<float*>(static_cast<unsigned char*>(ws) + LT_MAX_GROUPS * 4ll) : nullptr;
+  t.status = ctx->status_dev;
+  B2_CUDA(b2_launch(latent_tc_kernel<NR>, dim3(p.splits, p.row_tiles, a.B), dim3(LT_THREADS), p.smem, s, maps[0], maps[1], maps[2], maps[3], t));
   return B2_OK;
 }
 
@@ -774,10 +935,11 @@ int b2_heads_gemm(int dtype, const void* x, int64_t ldx, int x_head, const void*
   a.M = M; a.N = N; a.K = K; a.gate = gate; a.ldg = ldg; a.gate_hs = gate_head; a.rot_pad = rot_pad; a.positions = positions;
   a.cs = reinterpret_cast<const float2*>(cos_sin); a.max_pos = max_pos;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  const dim3 grid((N + 63) / 64 + (rot_pad > 0 ? 1 : 0), (M + 63) / 64, heads);
+  const int nt = dtype == B2_DT_BF16 && !w_is_kn ? CfgHeads<false>::NT : 64;
+  const dim3 grid((N + nt - 1) / nt + (rot_pad > 0 ? 1 : 0), (M + 63) / 64, heads);
   if (dtype == B2_DT_BF16) {
-    if (w_is_kn) B2_CUDA(b2_launch(heads_gemm_kernel<true>, grid, dim3(128), 0, s, a));
-    else B2_CUDA(b2_launch(heads_gemm_kernel<false>, grid, dim3(128), 0, s, a));
+    if (w_is_kn) return launch_heads<true>(a, grid, s);
+    return launch_heads<false>(a, grid, s);
   } else {
     if (w_is_kn) B2_CUDA(b2_launch(heads_gemm_f32_kernel<true>, grid, dim3(256), 0, s, a));
     else B2_CUDA(b2_launch(heads_gemm_f32_kernel<false>, grid, dim3(256), 0, s, a));
@@ -785,38 +947,37 @@ int b2_heads_gemm(int dtype, const void* x, int64_t ldx, int x_head, const void*
   return B2_OK;
 }
 
-int64_t b2_latent_attention_workspace(int dtype, int B, int max_q, int max_kv, int heads, int lat_pad, int rot_pad) {
-  if (B <= 0 || max_q <= 0 || heads <= 0 || !latent_tiled(dtype, lat_pad, rot_pad)) return 0;
-  return latent_plan(B, max_q, max_kv, heads, lat_pad).bytes;
+int64_t b2_latent_attention_workspace(int dtype, int B, int max_q, int max_kv, int block_size, int heads, int lat_pad, int rot_pad) {
+  if (B <= 0 || max_q <= 0 || heads <= 0 || block_size < 1 || !latent_tiled(dtype, block_size, lat_pad, rot_pad)) return 0;
+  return latent_plan(B, max_q, max_kv, heads, lat_pad, rot_pad).bytes;
 }
 
-int b2_latent_attention(int dtype, const void* q, int64_t ldq, void* out, int64_t ldo, const void* cache, const int32_t* block_tables,
-                        int64_t bt_stride, int block_size, const int32_t* cu_q, const int32_t* kv_len, int B, int max_q, int max_kv, int heads,
-                        int lat_pad, int rot_pad, float scale, const float* sink, void* workspace, int64_t workspace_bytes, int form, void* stream) {
+int b2_latent_attention(b2_ctx* ctx, int dtype, const void* q, int64_t q_rows, void* out, int64_t ldo, const void* cache, int64_t cache_slots,
+                        const int32_t* block_tables, int64_t bt_stride, int block_size, const int32_t* cu_q, const int32_t* kv_len, int B, int max_q,
+                        int max_kv, int heads, int lat_pad, int rot_pad, float scale, const float* sink, void* workspace, int64_t workspace_bytes,
+                        int form, void* stream) {
   if (B < 0 || max_q < 0 || bad_dtype(dtype) || heads <= 0 || lat_pad <= 0 || rot_pad < 0 || lat_pad % 8 != 0 || rot_pad % 8 != 0) return B2_ERR_ARG;
-  if (block_size < 1 || (cu_q == nullptr && max_q > 1)) return B2_ERR_ARG;
+  if (block_size < 1 || (cu_q == nullptr && max_q > 1) || q_rows < 0 || cache_slots < 0) return B2_ERR_ARG;
   if (B == 0 || max_q == 0) return B2_OK;
   if (!q || !out || !cache || !block_tables || !kv_len) return B2_ERR_ARG;
-  if (!aligned16(q) || !aligned16(out) || !aligned16(cache) || ldq % 8 != 0 || ldo % 8 != 0) return B2_ERR_ARG;
-  if (lat_pad + rot_pad > 2048 || lat_pad > 1024 || B > 65535 || heads > 65535) return B2_ERR_SHAPE;
+  if (!aligned16(q) || !aligned16(out) || !aligned16(cache) || ldo % 8 != 0) return B2_ERR_ARG;
+  if (lat_pad + rot_pad > 2048 || lat_pad > 1024 || B > 65535 || heads > 65535 || cache_slots > INT_MAX || q_rows * heads > INT_MAX) return B2_ERR_SHAPE;
   AttnArgs a{};
-  a.q = q; a.ldq = ldq; a.out = out; a.ldo = ldo; a.k_cache = a.v_cache = cache;
+  a.q = q; a.ldq = static_cast<int64_t>(heads) * (lat_pad + rot_pad); a.out = out; a.ldo = ldo; a.k_cache = a.v_cache = cache;
   a.block_tables = block_tables; a.bt_stride = bt_stride; a.block_size = block_size; a.cu_q = cu_q; a.kv_len = kv_len;
   a.B = B; a.nq = heads; a.nkv = 1; a.qk_pad = lat_pad + rot_pad; a.v_pad = lat_pad; a.k_row = a.v_row = lat_pad + rot_pad;
   a.window = INT_MAX; a.scale = scale; a.sink = sink;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   if (dtype == B2_DT_F32) return launch_any<float>(a, max_q, s);
-  if (form == 1 || !latent_tiled(dtype, lat_pad, rot_pad)) return launch_any<uint16_t>(a, max_q, s);
-  const LatentPlan p = latent_plan(B, max_q, max_kv, heads, lat_pad);
+  if (form == 1 || !latent_tiled(dtype, block_size, lat_pad, rot_pad)) return launch_any<uint16_t>(a, max_q, s);
+  if (ctx == nullptr) return B2_ERR_ARG;
+  const LatentPlan p = latent_plan(B, max_q, max_kv, heads, lat_pad, rot_pad);
   if (p.row_tiles > 65535) return B2_ERR_SHAPE;
   if (p.splits > 1 && (workspace == nullptr || workspace_bytes < p.bytes))
     return set_error(B2_ERR_SHAPE, "b2_latent_attention: workspace of %lld bytes, %lld needed", static_cast<long long>(workspace_bytes),
                      static_cast<long long>(p.bytes));
-  switch (latent_width(lat_pad)) {
-    case 128: return p.rows == 16 ? launch_latent<128, 1>(a, rot_pad, p, workspace, s) : launch_latent<128, 2>(a, rot_pad, p, workspace, s);
-    case 256: return p.rows == 16 ? launch_latent<256, 1>(a, rot_pad, p, workspace, s) : launch_latent<256, 2>(a, rot_pad, p, workspace, s);
-    default: return p.rows == 16 ? launch_latent<512, 1>(a, rot_pad, p, workspace, s) : launch_latent<512, 2>(a, rot_pad, p, workspace, s);
-  }
+  return p.rows == 16 ? launch_latent<16>(ctx, a, cache_slots, q_rows * heads, rot_pad, p, workspace, s)
+                      : launch_latent<32>(ctx, a, cache_slots, q_rows * heads, rot_pad, p, workspace, s);
 }
 
 int b2_expanded_attention(const void* q, int64_t ldq, void* out, int64_t ldo, const void* kv, int64_t ld_kv, const void* rot, int64_t ld_rot,

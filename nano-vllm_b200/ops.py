@@ -516,18 +516,18 @@ def latent_attention(q: torch.Tensor, heads: int, cache: torch.Tensor, lat_pad: 
                      max_kv: int, scale: float, sink, form: int = 0) -> torch.Tensor:
     """Absorbed attention of q [M, heads * row] over cached rows [blocks, block_size, 1, row]; cu_q None = decode.  Returns the
     mixed latents [M, heads * lat_pad]."""
-    row = cache.shape[-1]
+    row, block = cache.shape[-1], cache.shape[1]
     M, B = q.shape[0], kv_len.numel() if cu_q is None else cu_q.numel() - 1
-    assert q.stride(1) == 1 and q.dtype == cache.dtype and cache.is_contiguous() and q.shape[1] >= heads * row
+    assert q.is_contiguous() and q.shape[1] == heads * row and q.dtype == cache.dtype and cache.is_contiguous()
     assert block_tables.dtype == torch.int32 and kv_len.dtype == torch.int32 and (sink is None or sink.dtype == torch.float32)
     out = torch.empty(M, heads * lat_pad, dtype=q.dtype, device=q.device)
-    max_kv = min(max_kv, block_tables.shape[1] * cache.shape[1])
-    nbytes = _lib.b2_latent_attention_workspace(_dt(q), B, max_q, max_kv, heads, lat_pad, row - lat_pad)
+    max_kv = min(max_kv, block_tables.shape[1] * block)
+    nbytes = _lib.b2_latent_attention_workspace(_dt(q), B, max_q, max_kv, block, heads, lat_pad, row - lat_pad)
     ws = _workspace("latent_attention", nbytes, q.device)
-    _abi.check(_lib.b2_latent_attention(_dt(q), q.data_ptr(), q.stride(0), out.data_ptr(), out.stride(0), cache.data_ptr(), block_tables.data_ptr(),
-                                        block_tables.stride(0), cache.shape[1], _ptr(cu_q), kv_len.data_ptr(), B, max_q, max_kv, heads, lat_pad,
-                                        row - lat_pad, float(scale), _ptr(sink), _ptr(ws), ws.numel() if ws is not None else 0, form, _stream()),
-               "b2_latent_attention")
+    _abi.check(_lib.b2_latent_attention(get_runtime().ctx, _dt(q), q.data_ptr(), M, out.data_ptr(), out.stride(0), cache.data_ptr(),
+                                        cache.shape[0] * block, block_tables.data_ptr(), block_tables.stride(0), block, _ptr(cu_q), kv_len.data_ptr(), B,
+                                        max_q, max_kv, heads, lat_pad, row - lat_pad, float(scale), _ptr(sink), _ptr(ws),
+                                        ws.numel() if ws is not None else 0, form, _stream()), "b2_latent_attention")
     return out
 
 

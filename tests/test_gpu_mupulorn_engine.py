@@ -33,7 +33,7 @@ def test_generation_in_bf16_repeats_and_samples(pkg):
     """Decode graphs, the fused and (vocabulary not a multiple of 8) the unfused sampler; every pick is near the best."""
     from nanovllm_b200.engine.llm_engine import SamplingParams
     for case in ("wide", "odd"):
-        m = U.Model(case, torch.bfloat16)
+        m = U.Model(case, torch.bfloat16, kvcache_block_size=128 if case == "wide" else 16)
         try:
             prompts = [tokens(n, m.cfg["vocab"], n) for n in (33, 2, 64)]
             got = m.llm.generate(prompts, SamplingParams(max_tokens=12))
@@ -50,7 +50,7 @@ def test_generation_in_bf16_repeats_and_samples(pkg):
 
 def test_long_decoding(pkg):
     """Some hundred decoded tokens of unequal requests through the decode graphs, teacher-forced."""
-    m = U.Model("mixed", torch.bfloat16)
+    m = U.Model("mixed", torch.bfloat16, kvcache_block_size=128)
     try:
         toks = [tokens(n, m.cfg["vocab"], 60 + n) for n in (300, 290)]
         seqs = [m.seq(), m.seq()]
@@ -67,7 +67,7 @@ def test_long_decoding(pkg):
 
 def test_resident_decoder_matches_steps(pkg):
     from nanovllm_b200.engine.model_runner import ResidentDecoder, Seq
-    m = U.Model("wide", torch.bfloat16)
+    m = U.Model("wide", torch.bfloat16, kvcache_block_size=128)
     try:
         prompts = [tokens(n, m.cfg["vocab"], n) for n in (20, 45)]
         rd = ResidentDecoder(m.runner, 2)

@@ -302,7 +302,8 @@ def run_latent(dtype, heads, L, rot, lens, q_lens, block=16, form=0, seed=0, dec
         at += n
 
 
-LATENT = [(5, 52, 12, 16), (16, 128, 64, 64), (20, 200, 34, 24), (33, 512, 64, 64), (1, 24, 2, 8), (40, 264, 40, 256)]
+# heads, latent, rotated part, block (a multiple of 128: tcgen05)
+LATENT = [(5, 52, 12, 128), (16, 128, 64, 128), (20, 200, 34, 256), (33, 512, 64, 128), (1, 24, 2, 16), (40, 264, 40, 256), (7, 72, 8, 24), (32, 448, 64, 128)]
 FORMS = [(torch.float32, 0), (torch.bfloat16, 0), (torch.bfloat16, 1)]
 
 
@@ -323,9 +324,26 @@ def test_absorbed_attention_prompts_and_portions(case, dtype, form):
 def test_absorbed_attention_split_over_many_ctas():
     """Long sequences whose key tiles go to many CTAs; repeated calls find their counters reset; a batch with a short one."""
     for rep in range(3):
-        run_latent(torch.bfloat16, 6, 256, 32, [1500 + 37 * rep], [1], 64, seed=rep, decode=True)
-    run_latent(torch.bfloat16, 18, 136, 64, [900, 5], [1, 1], 64, decode=True)
-    run_latent(torch.bfloat16, 3, 512, 64, [700], [5], 32)
+        run_latent(torch.bfloat16, 6, 256, 32, [1500 + 37 * rep], [1], 128, seed=rep, decode=True)
+    run_latent(torch.bfloat16, 18, 136, 64, [900, 5], [1, 1], 256, decode=True)
+    run_latent(torch.bfloat16, 3, 512, 64, [700], [5], 128)
+    run_latent(torch.bfloat16, 2, 64, 8, [9000], [1], 128, decode=True)
+
+
+def test_absorbed_attention_when_the_running_maximum_keeps_rising():
+    """Scores that grow from tile to tile by more and by less than the amount after which outputs are rescaled."""
+    from nanovllm_b200 import ops
+    heads, L, rot, n, scale = 5, 128, 8, 900, 0.1
+    q = rnd(0, 1, heads, L + rot).bfloat16()
+    for rise in (0.004, 0.05, 0.3):
+        ramp = torch.arange(1024).view(8, 128, 1, 1) * rise
+        unit = q[0].float().mean(0) / q[0].float().mean(0).pow(2).sum()
+        c = (0.3 * rnd(1, 8, 128, 1, L + rot) + ramp * unit).bfloat16()
+        kn = c.view(1024, L + rot)[:n, :L].double().unsqueeze(1).expand(-1, heads, -1)
+        want = P.attend(q[:, :, :L].double(), q[:, :, L:].double(), kn, c.view(1024, L + rot)[:n, L:].double(), kn, scale, torch.zeros(heads).double(), n - 1)
+        got = ops.latent_attention(q.view(1, -1).to(DEV), heads, c.to(DEV), L, torch.arange(8, dtype=torch.int32, device=DEV).view(1, 8), None, i32([n]), 1, 1024,
+                                   scale, torch.zeros(heads, device=DEV))
+        close(got.view(1, heads, L), want, torch.bfloat16, f"rise {rise}")
 
 
 def test_absorbed_attention_of_wide_latents_runs_on_the_general_kernel():
@@ -336,9 +354,9 @@ def test_absorbed_attention_of_wide_latents_runs_on_the_general_kernel():
 def test_padded_decode_rows_give_zeros():
     from nanovllm_b200 import ops
     for dtype in DTYPES:
-        cache = torch.randn(2, 16, 1, 80, device=DEV).to(dtype)
+        cache = torch.randn(2, 128, 1, 80, device=DEV).to(dtype)
         out = ops.latent_attention(torch.randn(3, 160, device=DEV).to(dtype), 2, cache, 64, torch.zeros(3, 1, dtype=torch.int32, device=DEV), None,
-                                   i32([4, 0, 0]), 1, 16, 0.1, torch.zeros(2, device=DEV))
+                                   i32([4, 0, 0]), 1, 128, 0.1, torch.zeros(2, device=DEV))
         assert out[0].abs().sum() > 0 and out[1:].abs().sum() == 0
 
 

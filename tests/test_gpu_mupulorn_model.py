@@ -8,25 +8,22 @@ from tests import mupulorn_util as U
 pytestmark = pytest.mark.gpu
 
 
-@pytest.fixture(scope="module", params=[(c, d) for c in U.CASES for d in (torch.float32, torch.bfloat16)], ids=lambda p: f"{p[0]}-{str(p[1])[6:]}")
+# how prompts attend: chosen by cost (None), or always one way; decoding is always absorbed
+RUNS = [(c, torch.float32, None) for c in U.CASES] + [(c, torch.bfloat16, f) for c in U.CASES for f in (None, "absorbed", "expanded", "any")]
+
+
+@pytest.fixture(scope="module", params=RUNS, ids=lambda p: f"{p[0]}-{str(p[1])[6:]}-{p[2]}")
 def model(request, pkg):
-    m = U.Model(*request.param)
+    """Pages of 128 tokens, except for one case (pages of another size take the kernel for any size)."""
+    from nanovllm_b200.layers.latent_attention import LatentAttention
+    case, dtype, LatentAttention.form = request.param
+    m = U.Model(case, dtype, kvcache_block_size=16 if case == "odd" else 128)
     yield m
     m.llm.exit()
-
-
-@pytest.fixture(params=[None, "absorbed", "expanded", "any"])
-def form(request, pkg, model):
-    """How prompts attend: chosen by cost, or always one way (decoding is always absorbed)."""
-    from nanovllm_b200.layers.latent_attention import LatentAttention
-    if model.dtype == torch.float32 and request.param is not None:
-        pytest.skip("fp32 has one form")
-    LatentAttention.form = request.param
-    yield request.param
     LatentAttention.form = None
 
 
-def test_prompt_layer_by_layer(model, form):
+def test_prompt_layer_by_layer(model):
     M.layer_by_layer(model)
 
 
@@ -35,11 +32,11 @@ def test_decoding_token_by_token(model):
 
 
 @pytest.mark.parametrize("size", [2, 3, 5, 16, 33, 64, 100])
-def test_portions(model, form, size):
+def test_portions(model, size):
     M.portions(model, size)
 
 
-def test_batches_of_unequal_requests(model, form):
+def test_batches_of_unequal_requests(model):
     M.batches_of_unequal_requests(model)
 
 
