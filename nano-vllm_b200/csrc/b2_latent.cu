@@ -9,6 +9,7 @@
 //   latent_gather_kernel   cached rows of a batch as contiguous rows (a portion whose sequence has earlier tokens)
 //   heads_gemm_kernel      one small matrix product per head, with the rotation of the query part or an output gate
 //   latent_tc_kernel       absorbed attention on tcgen05: 16 or 32 (token, head) rows, 128 keys per tile
+//   latent_combine_kernel  the parts of its key ranges
 //   expanded_attn_kernel   expanded attention, 64 tokens of one head x 64 keys; rotates the queries it loads, gates its output
 #include <algorithm>
 
@@ -331,18 +332,17 @@ __global__ void __launch_bounds__(256) heads_gemm_f32_kernel(const HeadsArgs a) 
 //   scores   S^T [128 keys x NR]   = rows (K-major)           x Q^T
 //   outputs  O^T [128 dims x NR]  += latents^T (M contiguous) x P^T, one accumulator per 128 latent columns
 // from the same boxes.  Warps 0-3: softmax, a thread per key; the weights go back through shared memory as a sum of two bf16
-// numbers.  Warp 4: TMA.  Warp 5: MMA.  Key tiles are dealt to `splits` CTAs whose parts the last one to arrive combines.
+// numbers that lie side by side in the N dimension of one product.  Warp 4: TMA.  Warp 5: MMA.  Key tiles are dealt to
+// `splits` CTAs; a second kernel combines their parts.
 // ---------------------------------------------------------------------------
 constexpr int LT_KEYS = 128;                 // keys per tile
 constexpr int LT_BOX = LT_KEYS * 64 * 2;     // bytes of one box
 constexpr int LT_THREADS = 192;
 constexpr int LT_MAX_PAIRS = 4;              // latents up to 512 wide
 constexpr int LT_MAX_STAGES = 3;
-constexpr int LT_TMEM = 256;                 // S^T: NR columns, O^T: 4 NR
 constexpr int LT_MAX_SPLITS = 64;
-constexpr int LT_MAX_GROUPS = 65536;         // arrival counters at the front of the workspace
 constexpr uint64_t LT_LIMIT_NS = 1000000000ull;
-constexpr int LT_SMEM_MAX = 227 * 1024;
+constexpr int LT_SMEM_MAX = 227 * 1024, LT_SMEM_STATIC = 2048;  // per CTA, and what of it the kernel declares statically
 constexpr float LT_RESCALE = 8.0f;           // the running maximum may be exceeded by 2^8 before the outputs are rescaled
 
 struct LatentTcArgs {
@@ -357,10 +357,10 @@ struct LatentTcArgs {
   int stages, row_tiles, splits;
   float scale;
   const float* sink;
-  int* counters;
-  float* part;  // [group][split][2 NR + NR * 128 pairs]: maxima, sums, outputs by row
+  float* part;  // [group][split]: maxima [NR], sums [NR], outputs [NR / 4][128 pairs][4 rows]
   B2Status* status;
 };
+__host__ __device__ constexpr int64_t latent_part_floats(int nr, int pairs) { return 2 * nr + static_cast<int64_t>(nr) * 128 * pairs; }
 
 // v over the warp's 32 lanes, one result per column: lane l gets column l & (NR - 1).  Destroys v.
 template <int NR, typename Op>
@@ -398,17 +398,20 @@ template <int NR>
 __global__ void __launch_bounds__(LT_THREADS, 1)
 latent_tc_kernel(const __grid_constant__ CUtensorMap tm_lat, const __grid_constant__ CUtensorMap tm_rot, const __grid_constant__ CUtensorMap tm_ql,
                  const __grid_constant__ CUtensorMap tm_qr, const LatentTcArgs a) {
+  constexpr uint32_t TMEM_COLS = NR == 32 ? 512 : 256;  // S^T: NR columns, O^T: 2 NR (leading and trailing parts) per pair of boxes
   extern __shared__ unsigned char smem_raw[];
   __shared__ __align__(8) uint64_t s_bars[2 * LT_MAX_STAGES * (LT_MAX_PAIRS + 1) + 4];
-  __shared__ float s_red[4][32], s_fac[LT_MAX_SPLITS * 32];
+  __shared__ float s_red[4][32];
+  __shared__ int64_t s_out[NR];  // offset of every row's output
+  __shared__ int s_pos[NR];      // its position
   __shared__ uint32_t s_tmem;
-  __shared__ int s_abort, s_last;
+  __shared__ int s_abort;
   volatile int* abort_flag = &s_abort;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int pairs = (a.boxes + 1) >> 1, stage_bytes = (2 * pairs + a.rot) * LT_BOX;
   const uint32_t q_bytes = (a.boxes + a.rot) * NR * 128;
   const uint32_t sq = (smem_u32(smem_raw) + 1023u) & ~1023u;
-  const uint32_t sp = sq + ((q_bytes + 1023u) & ~1023u);  // P: [hi, lo][two halves of 64 keys][NR rows of 128 bytes]
+  const uint32_t sp = sq + ((q_bytes + 1023u) & ~1023u);  // P: [two halves of 64 keys][NR leading, NR trailing rows of 128 bytes]
   const uint32_t sk = sp + NR * 512;
   const uint32_t bar_full = smem_u32(s_bars), bar_empty = bar_full + LT_MAX_STAGES * (LT_MAX_PAIRS + 1) * 8;
   const uint32_t bar_q = bar_empty + LT_MAX_STAGES * (LT_MAX_PAIRS + 1) * 8, bar_s = bar_q + 8, bar_p = bar_q + 16, bar_o = bar_q + 24;
@@ -431,7 +434,7 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap tm_lat, const __grid_consta
     tma_prefetch_desc(&tm_qr);
   }
   if (warp == 5) {
-    tmem_alloc(smem_u32(&s_tmem), LT_TMEM);
+    tmem_alloc(smem_u32(&s_tmem), TMEM_COLS);
     tmem_relinquish();
   }
   tc_fence_before();
@@ -450,10 +453,6 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap tm_lat, const __grid_consta
   const int pmin = first_pos + r_base / a.heads, pmax = first_pos + (r_base + max(nrows, 1) - 1) / a.heads;
   const int total = nrows > 0 && klen > 0 ? pmax / LT_KEYS + 1 : 0, per = (total + a.splits - 1) / a.splits;
   const int t0 = split * per, t1 = min(total, t0 + per);
-  const auto out_row = [&](int r) {
-    const int gr = r_base + r, tok = gr / a.heads;
-    return a.out + (row0 + tok) * a.ldo + static_cast<int64_t>(gr - tok * a.heads) * a.v_pad;
-  };
 
   if (warp == 4) {
     // ---------------- TMA ----------------
@@ -486,7 +485,7 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap tm_lat, const __grid_consta
   } else if (warp == 5) {
     // ---------------- MMA ----------------
     if (lane == 0 && t0 < t1) {
-      constexpr uint32_t idesc_s = umma_idesc_bf16(NR), idesc_o = umma_idesc_bf16(NR) | UMMA_A_MN;
+      constexpr uint32_t idesc_s = umma_idesc_bf16(NR), idesc_o = umma_idesc_bf16(2 * NR) | UMMA_A_MN;
       int st = 0;
       uint32_t phase = 0;
       bool ok = mbar_wait(bar_q, 0, abort_flag, LT_LIMIT_NS, B2_WAIT_SMEM_FULL);
@@ -519,13 +518,11 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap tm_lat, const __grid_consta
         tc_fence_after();
         for (int p = 0; p < pairs; ++p) {
 #pragma unroll
-          for (int half = 0; half < 2; ++half)  // the weights' leading and trailing parts
-#pragma unroll
-            for (int k = 0; k < LT_KEYS / 16; ++k) {
-              const uint64_t dv = umma_smem_desc_mn(base + 2 * p * LT_BOX + k * 2048, LT_BOX);
-              const uint64_t dp = umma_smem_desc(sp + half * NR * 256 + (k >> 2) * NR * 128) + 2 * (k & 3);
-              umma_bf16(tm_o + p * NR, dv, dp, idesc_o, (t > t0 || half > 0 || k > 0) ? 1u : 0u);
-            }
+          for (int k = 0; k < LT_KEYS / 16; ++k) {
+            const uint64_t dv = umma_smem_desc_mn(base + 2 * p * LT_BOX + k * 2048, LT_BOX);
+            const uint64_t dp = umma_smem_desc(sp + (k >> 2) * NR * 256) + 2 * (k & 3);
+            umma_bf16(tm_o + p * 2 * NR, dv, dp, idesc_o, (t > t0 || k > 0) ? 1u : 0u);
+          }
           umma_commit(empty(st, p));
         }
         if (++st == a.stages) { st = 0; phase ^= 1; }
@@ -537,6 +534,12 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap tm_lat, const __grid_consta
     const uint32_t lanes = static_cast<uint32_t>(warp * 32) << 16;
     const int col = lane & (NR - 1);  // the row whose maximum, sum and factors this lane keeps
     const float scale = a.scale * LOG2E;
+    if (threadIdx.x < NR) {
+      const int gr = r_base + min(static_cast<int>(threadIdx.x), max(nrows, 1) - 1), tok = gr / a.heads;
+      s_pos[threadIdx.x] = first_pos + tok;
+      s_out[threadIdx.x] = (row0 + tok) * a.ldo + static_cast<int64_t>(gr - tok * a.heads) * a.v_pad;
+    }
+    softmax_meet(true);
     float m_col = -INFINITY;
     float l[NR];
 #pragma unroll
@@ -549,16 +552,17 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap tm_lat, const __grid_consta
       uint32_t raw[NR];
       tmem_load<NR>(tm_s + lanes, raw);
       float v[NR], w[NR];
-      const int j = t * LT_KEYS + threadIdx.x;
-      const bool masked = t * LT_KEYS + LT_KEYS - 1 > pmin;
 #pragma unroll
-      for (int r = 0; r < NR; ++r) {
-        v[r] = __uint_as_float(raw[r]) * scale;
-        if (masked && j > first_pos + (r_base + min(r, nrows - 1)) / a.heads) v[r] = -INFINITY;
-        w[r] = v[r];
+      for (int r = 0; r < NR; ++r) v[r] = __uint_as_float(raw[r]) * scale;
+      if (t * LT_KEYS + LT_KEYS - 1 > pmin) {
+        const int j = t * LT_KEYS + threadIdx.x;
+#pragma unroll
+        for (int r = 0; r < NR; ++r)
+          if (j > s_pos[r]) v[r] = -INFINITY;
       }
-      const float mx = reduce_columns<NR>(w, lane, [](float x, float y) { return fmaxf(x, y); });
-      s_red[warp][lane] = mx;
+#pragma unroll
+      for (int r = 0; r < NR; ++r) w[r] = v[r];
+      s_red[warp][lane] = reduce_columns<NR>(w, lane, [](float x, float y) { return fmaxf(x, y); });
       if (!(ok = softmax_meet(ok))) break;
       const float m_tile = fmaxf(fmaxf(s_red[0][col], s_red[1][col]), fmaxf(s_red[2][col], s_red[3][col]));
       const bool grow = m_tile > m_col + LT_RESCALE || m_col == -INFINITY;
@@ -567,7 +571,7 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap tm_lat, const __grid_consta
       if (__any_sync(0xffffffffu, corr != 1.0f)) {  // the same in all four warps; never in the first tile
 #pragma unroll
         for (int r = 0; r < NR; ++r) l[r] *= __shfl_sync(0xffffffffu, corr, r);
-        for (int p = 0; p < pairs; ++p) {
+        for (int p = 0; p < 2 * pairs; ++p) {
           tmem_load<NR>(tm_o + p * NR + lanes, raw);
 #pragma unroll
           for (int r = 0; r < NR; ++r) raw[r] = __float_as_uint(__uint_as_float(raw[r]) * __shfl_sync(0xffffffffu, corr, r));
@@ -588,18 +592,18 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap tm_lat, const __grid_consta
         v[r] = fast_exp2(v[r] - __shfl_sync(0xffffffffu, ref, r));
         l[r] += v[r];
       }
-      // neighbours exchange: an even lane stores rows r of keys (lane, lane + 1), an odd one rows r + 1
+      // neighbours exchange: an even lane stores row r of keys (lane, lane + 1), an odd one row r + 1
       const int odd = lane & 1, key2 = (warp & 1) * 32 + (lane & ~1);  // first of the two keys inside the half tile
-      const uint32_t at = sp + (warp >> 1) * NR * 128 + (key2 & 7) * 2;
+      const uint32_t at = sp + (warp >> 1) * NR * 256 + (key2 & 7) * 2;
 #pragma unroll
       for (int r = 0; r < NR; r += 2) {
         const float other = __shfl_xor_sync(0xffffffffu, odd ? v[r] : v[r + 1], 1);
         const int rr = r + odd;
         uint32_t hi, lo;
         split_bf16(odd ? other : v[r], odd ? v[r + 1] : other, hi, lo);
-        const uint32_t dst = at + rr * 128 + (((key2 >> 3) ^ (rr & 7)) << 4);
+        const uint32_t dst = at + rr * 128 + (((key2 >> 3) ^ (rr & 7)) << 4);  // NR is a multiple of 8: the same for both parts
         asm volatile("st.shared.u32 [%0], %1;" ::"r"(dst), "r"(hi) : "memory");
-        asm volatile("st.shared.u32 [%0], %1;" ::"r"(dst + NR * 256), "r"(lo) : "memory");
+        asm volatile("st.shared.u32 [%0], %1;" ::"r"(dst + NR * 128), "r"(lo) : "memory");
       }
       fence_proxy_async();
       tc_fence_before();
@@ -609,83 +613,42 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap tm_lat, const __grid_consta
     if (ok && t0 < t1) ok = mbar_wait(bar_o, 0, abort_flag, LT_LIMIT_NS, B2_WAIT_TMEM_FULL);
     __syncwarp();
     tc_fence_after();
-    const float lw = reduce_columns<NR>(l, lane, [](float x, float y) { return x + y; });
-    s_red[warp][lane] = lw;
+    s_red[warp][lane] = reduce_columns<NR>(l, lane, [](float x, float y) { return x + y; });
     ok = softmax_meet(ok);
     if (ok && nrows > 0) {
       const float l_col = s_red[0][col] + s_red[1][col] + s_red[2][col] + s_red[3][col];
-      const int group = b * a.row_tiles + blockIdx.y;
-      const int64_t part_floats = 2 * NR + static_cast<int64_t>(NR) * 128 * pairs;
-      float* my = a.part + (static_cast<int64_t>(group) * a.splits + split) * part_floats;
-      if (klen <= 0) {  // padded row of a decode graph
-        if (split == 0)
-          for (int i = threadIdx.x; i < nrows * a.v_pad; i += 128) out_row(i / a.v_pad)[i % a.v_pad] = 0;
-      } else {
-        float f = 1.0f;
-        if (a.splits == 1) {
-          float sum = l_col;
-          if (a.sink != nullptr) {
-            const float sk_ = a.sink[(r_base + col) % a.heads] * LOG2E, m_new = fmaxf(m_col, sk_);
-            f = fast_exp2(m_col - m_new);
-            sum = sum * f + fast_exp2(sk_ - m_new);
-          }
-          f /= sum;
-        } else if (warp == 0 && lane < nrows && lane < NR) {
+      float* my = a.part + (static_cast<int64_t>(b * a.row_tiles + blockIdx.y) * a.splits + split) * latent_part_floats(NR, pairs);
+      float f = 0.f;
+      if (a.splits > 1) {
+        if (warp == 0 && lane < NR) {
           my[lane] = m_col;
           my[NR + lane] = l_col;
         }
-        if (t0 < t1) {
-          for (int p = 0; p < pairs; ++p) {
-            uint32_t raw[NR];
-            tmem_load<NR>(tm_o + p * NR + lanes, raw);
-            const int dim = p * 128 + threadIdx.x;
+      } else if (klen > 0) {
+        const float sk_ = a.sink != nullptr ? a.sink[(r_base + col) % a.heads] * LOG2E : -INFINITY, m_new = fmaxf(m_col, sk_);
+        f = fast_exp2(m_col - m_new);
+        f /= l_col * f + fast_exp2(sk_ - m_new);
+      }
+      if (t0 < t1 || a.splits == 1) {
+        for (int p = 0; p < pairs; ++p) {
+          uint32_t raw[NR], low[NR];
+          float o[NR];
+          if (t0 < t1) {
+            tmem_load<NR>(tm_o + p * 2 * NR + lanes, raw);
+            tmem_load<NR>(tm_o + p * 2 * NR + NR + lanes, low);
+          }
+#pragma unroll
+          for (int r = 0; r < NR; ++r) o[r] = t0 < t1 ? __uint_as_float(raw[r]) + __uint_as_float(low[r]) : 0.f;  // nothing seen: a padded row
+          const int dim = p * 128 + threadIdx.x;
+          if (a.splits > 1) {
+#pragma unroll
+            for (int r = 0; r < NR; r += 4)
+              *reinterpret_cast<float4*>(my + 2 * NR + ((r >> 2) * 128 * pairs + dim) * 4) = make_float4(o[r], o[r + 1], o[r + 2], o[r + 3]);
+          } else {
 #pragma unroll
             for (int r = 0; r < NR; ++r) {
-              const float fr = __shfl_sync(0xffffffffu, f, r);
-              if (r < nrows) {
-                if (a.splits > 1) my[2 * NR + r * 128 * pairs + dim] = __uint_as_float(raw[r]);
-                else if (dim < a.v_pad) out_row(r)[dim] = from_float<uint16_t>(__uint_as_float(raw[r]) * fr);
-              }
-            }
-          }
-        }
-        if (a.splits > 1) {
-          __threadfence();
-          softmax_meet(true);
-          if (threadIdx.x == 0) s_last = atomicAdd(a.counters + group, 1) == a.splits - 1;
-          softmax_meet(true);
-          if (s_last) {
-            if (threadIdx.x == 0) a.counters[group] = 0;
-            __threadfence();
-            const float* all = a.part + static_cast<int64_t>(group) * a.splits * part_floats;
-            if (static_cast<int>(threadIdx.x) < nrows) {
-              const int r = threadIdx.x;
-              const float sk_ = a.sink != nullptr ? a.sink[(r_base + r) % a.heads] * LOG2E : -INFINITY;
-              float mt = sk_;
-              for (int s = 0; s < a.splits; ++s) mt = fmaxf(mt, ld_cg_f32(all + s * part_floats + r));
-              float lt = fast_exp2(sk_ - mt);
-              for (int s = 0; s < a.splits; ++s) {
-                const float ms = ld_cg_f32(all + s * part_floats + r);
-                const float fs = ms > -INFINITY ? fast_exp2(ms - mt) : 0.f;
-                s_fac[s * NR + r] = fs;
-                if (fs > 0.f) lt += fs * ld_cg_f32(all + s * part_floats + NR + r);
-              }
-              for (int s = 0; s < a.splits; ++s) s_fac[s * NR + r] /= lt;
-            }
-            softmax_meet(true);
-            const int vecs = a.v_pad >> 2;
-            for (int i = threadIdx.x; i < nrows * vecs; i += 128) {
-              const int r = i / vecs, c = (i - r * vecs) * 4;
-              float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
-#pragma unroll 4
-              for (int s = 0; s < a.splits; ++s) {
-                const float fs = s_fac[s * NR + r];
-                if (fs == 0.f) continue;  // a split without keys for this row may hold anything
-                const uint4 q = ld_cg_v4(all + s * part_floats + 2 * NR + r * 128 * pairs + c);
-                acc.x += fs * __uint_as_float(q.x); acc.y += fs * __uint_as_float(q.y);
-                acc.z += fs * __uint_as_float(q.z); acc.w += fs * __uint_as_float(q.w);
-              }
-              *reinterpret_cast<uint2*>(out_row(r) + c) = make_uint2(pack_bf16(acc.x, acc.y), pack_bf16(acc.z, acc.w));
+              const float x = o[r] * __shfl_sync(0xffffffffu, f, r);
+              if (r < nrows && dim < a.v_pad) a.out[s_out[r] + dim] = from_float<uint16_t>(x);
             }
           }
         }
@@ -700,7 +663,62 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap tm_lat, const __grid_consta
     for (int i = 0; i < 100; ++i) __nanosleep(2000);
     if (threadIdx.x == 0) report_timeout(a.status, s_abort);
   }
-  if (warp == 5) tmem_dealloc(s_tmem, LT_TMEM);
+  if (warp == 5) tmem_dealloc(s_tmem, TMEM_COLS);
+}
+
+// The splits' parts of 4 rows -> their outputs.  One thread per latent column.
+template <int NR>
+__global__ void __launch_bounds__(512) latent_combine_kernel(const LatentTcArgs a) {
+  __shared__ float s_fac[4][LT_MAX_SPLITS];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int b = blockIdx.z, r_base = blockIdx.y * NR, r4 = blockIdx.x;
+  const int row0 = a.cu_q ? a.cu_q[b] : b;
+  const int rows = (a.cu_q ? a.cu_q[b + 1] - row0 : 1) * a.heads;
+  if (r_base + r4 * 4 >= rows) return;
+  const int pairs = (a.boxes + 1) >> 1, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int64_t floats = latent_part_floats(NR, pairs);
+  const float* all = a.part + static_cast<int64_t>(b * a.row_tiles + blockIdx.y) * a.splits * floats;
+  const bool live = a.kv_len[b] > 0;
+  if (warp < 4) {  // a warp per row: the factors of its parts
+    const int r = r4 * 4 + warp;
+    const float sk = a.sink != nullptr ? a.sink[(r_base + r) % a.heads] * LOG2E : -INFINITY;
+    float ms[LT_MAX_SPLITS / 32], ls[LT_MAX_SPLITS / 32], top = sk, sum = 0.f;
+#pragma unroll
+    for (int i = 0; i < LT_MAX_SPLITS / 32; ++i) {
+      const int s = lane + 32 * i;
+      ms[i] = s < a.splits && live ? all[s * floats + r] : -INFINITY;
+      ls[i] = s < a.splits && live ? all[s * floats + NR + r] : 0.f;
+      top = fmaxf(top, ms[i]);
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, o));
+#pragma unroll
+    for (int i = 0; i < LT_MAX_SPLITS / 32; ++i) {
+      ms[i] = ms[i] > -INFINITY ? fast_exp2(ms[i] - top) : 0.f;
+      sum += ms[i] * ls[i];
+    }
+    sum = group_sum(sum) + (sk > -INFINITY ? fast_exp2(sk - top) : 0.f);
+#pragma unroll
+    for (int i = 0; i < LT_MAX_SPLITS / 32; ++i)
+      if (lane + 32 * i < a.splits) s_fac[warp][lane + 32 * i] = sum > 0.f ? ms[i] / sum : 0.f;
+  }
+  __syncthreads();
+  const int dim = threadIdx.x;
+  if (dim >= a.v_pad) return;
+  float o[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll 4
+  for (int s = 0; s < a.splits; ++s) {
+    const float f[4] = {s_fac[0][s], s_fac[1][s], s_fac[2][s], s_fac[3][s]};
+    if (f[0] == 0.f && f[1] == 0.f && f[2] == 0.f && f[3] == 0.f) continue;  // a part without keys may hold anything
+    const float4 x = *reinterpret_cast<const float4*>(all + s * floats + 2 * NR + (static_cast<int64_t>(r4) * 128 * pairs + dim) * 4);
+    o[0] += f[0] * x.x; o[1] += f[1] * x.y; o[2] += f[2] * x.z; o[3] += f[3] * x.w;
+  }
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const int gr = r_base + r4 * 4 + i, tok = gr / a.heads;
+    if (gr < rows) a.out[(row0 + tok) * a.ldo + static_cast<int64_t>(gr - tok * a.heads) * a.v_pad + dim] = from_float<uint16_t>(o[i]);
+  }
 }
 
 struct LatentPlan {
@@ -711,7 +729,7 @@ bool latent_tiled(int dtype, int block_size, int lat_pad, int rot_pad) {
   return dtype == B2_DT_BF16 && lat_pad <= 128 * LT_MAX_PAIRS && rot_pad <= 64 && block_size % LT_KEYS == 0;
 }
 // Rows per CTA, tiles in shared memory, and how many CTAs share a group's key tiles: as few rounds of one CTA per SM as
-// possible, where a CTA's start and end cost about three tiles and a combine one more.
+// possible, where a CTA's start and end cost about two tiles and a combine one more.
 LatentPlan latent_plan(int B, int max_q, int max_kv, int heads, int lat_pad, int rot_pad) {
   LatentPlan p{};
   const int64_t all = static_cast<int64_t>(max_q) * heads;
@@ -720,30 +738,30 @@ LatentPlan latent_plan(int B, int max_q, int max_kv, int heads, int lat_pad, int
   p.boxes = (lat_pad + 63) / 64;
   p.rot = rot_pad > 0;
   p.pairs = (p.boxes + 1) / 2;
-  const int fixed = 1024 + (((p.boxes + p.rot) * p.rows * 128 + 1023) & ~1023) + p.rows * 512 + 12 * 1024 /* static */;
+  const int fixed = 1024 + (((p.boxes + p.rot) * p.rows * 128 + 1023) & ~1023) + p.rows * 512 + LT_SMEM_STATIC;
   const int stage = (2 * p.pairs + p.rot) * LT_BOX;
   p.stages = std::max(1, std::min(LT_MAX_STAGES, (LT_SMEM_MAX - fixed) / stage));
-  p.smem = fixed - 12 * 1024 + p.stages * stage;
+  p.smem = fixed - LT_SMEM_STATIC + p.stages * stage;
   p.groups = static_cast<int64_t>(B) * p.row_tiles;
   const int64_t tiles = std::max<int64_t>(1, (static_cast<int64_t>(max_kv) + LT_KEYS - 1) / LT_KEYS);
   p.splits = 1;
-  if (p.groups <= LT_MAX_GROUPS && p.groups < 4 * 148) {
+  if (p.groups < 4 * 148) {
     int64_t best = INT64_MAX;
     for (int s = 1; s <= std::min<int64_t>(LT_MAX_SPLITS, tiles); ++s) {
-      const int64_t cost = ((p.groups * s + 147) / 148) * (8 * ((tiles + s - 1) / s) + 24 + (s > 1 ? 8 : 0)) + s;
+      const int64_t cost = ((p.groups * s + 147) / 148) * (8 * ((tiles + s - 1) / s) + 16) + (s > 1 ? 8 : 0) + s / 2;
       if (cost < best) {
         best = cost;
         p.splits = s;
       }
     }
   }
-  p.bytes = p.splits > 1 ? LT_MAX_GROUPS * 4ll + p.groups * p.splits * p.rows * (2ll + 128 * p.pairs) * 4 : 0;
+  p.bytes = p.splits > 1 ? p.groups * p.splits * latent_part_floats(p.rows, p.pairs) * 4 : 0;
   return p;
 }
 
 template <int NR>
 int launch_latent(const b2_ctx* ctx, const AttnArgs& a, int64_t slots, int64_t q_rows, int rot_pad, const LatentPlan& p, void* ws, cudaStream_t s) {
-  static const cudaError_t set = cudaFuncSetAttribute(latent_tc_kernel<NR>, cudaFuncAttributeMaxDynamicSharedMemorySize, LT_SMEM_MAX - 12 * 1024);
+  static const cudaError_t set = cudaFuncSetAttribute(latent_tc_kernel<NR>, cudaFuncAttributeMaxDynamicSharedMemorySize, LT_SMEM_MAX - LT_SMEM_STATIC);
   B2_CUDA(set);
   CUtensorMap maps[4];
   const uint16_t* cache = static_cast<const uint16_t*>(a.k_cache);
@@ -761,10 +779,11 @@ int launch_latent(const b2_ctx* ctx, const AttnArgs& a, int64_t slots, int64_t q
   t.out = static_cast<uint16_t*>(a.out); t.ldo = a.ldo; t.block_tables = a.block_tables; t.bt_stride = a.bt_stride; t.block_size = a.block_size;
   t.cu_q = a.cu_q; t.kv_len = a.kv_len; t.heads = a.nq; t.v_pad = a.v_pad; t.boxes = p.boxes; t.rot = p.rot; t.stages = p.stages;
   t.row_tiles = p.row_tiles; t.splits = p.splits; t.scale = a.scale; t.sink = a.sink;
-  t.counters = static_cast<int*>(ws);
-  t.part = ws != nullptr ? reinterpret_cast<float*>(static_cast<unsigned char*>(ws) + LT_MAX_GROUPS * 4ll) : nullptr;
+  t.part = static_cast<float*>(ws);
   t.status = ctx->status_dev;
   B2_CUDA(b2_launch(latent_tc_kernel<NR>, dim3(p.splits, p.row_tiles, a.B), dim3(LT_THREADS), p.smem, s, maps[0], maps[1], maps[2], maps[3], t));
+  if (p.splits > 1)
+    B2_CUDA(b2_launch(latent_combine_kernel<NR>, dim3(NR / 4, p.row_tiles, a.B), dim3(std::max(128, (a.v_pad + 31) / 32 * 32)), 0, s, t));
   return B2_OK;
 }
 
