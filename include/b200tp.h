@@ -555,15 +555,18 @@ int b2_latent_attention(b2_ctx* ctx, int dtype, const void* q, int64_t q_rows, v
                         int rot_pad, float scale, const float* sink, void* workspace, int64_t workspace_bytes, int form,
                         void* stream);
 
-/* Expanded attention (bf16; dim_pad + rot_pad <= 192, v_pad <= 128): rows of kv hold
- * [dim_pad key | v_pad value] per head, rows of rot the shared rotated key part;
- * position j of sequence b is row cu_k[b] + j of both.  q heads are
- * [dim_pad | rot_pad], not yet rotated.  out [M][heads][v_pad] is multiplied by
- * sigmoid(gate) when gate ([M][heads][v_pad], row stride ldg) is given. */
-int b2_expanded_attention(const void* q, int64_t ldq, void* out, int64_t ldo, const void* kv, int64_t ld_kv, const void* rot,
-                          int64_t ld_rot, const int32_t* cu_q, const int32_t* cu_k, int B, int max_q, int heads, int dim_pad,
-                          int rot_pad, int v_pad, float scale, const float* sink, const float* cos_sin, int max_pos,
-                          const void* gate, int64_t ldg, void* stream);
+/* Expanded attention on tcgen05 (bf16; dim_pad <= 128, rot_pad <= 64, v_pad <= 128,
+ * scale > 0): rows of kv ([k_rows]) hold [dim_pad key | v_pad value] per head, rows
+ * of rot the shared rotated key part; position j of sequence b is row cu_k[b] + j
+ * of both.  q heads ([q_rows]) are [dim_pad | rot_pad], not yet rotated.  Causal;
+ * out [q_rows][heads][v_pad] is multiplied by sigmoid(gate) when gate
+ * ([q_rows][heads][v_pad], row stride ldg) is given.  A bounded wait that expires
+ * shows in b2_status. */
+int b2_expanded_attention(b2_ctx* ctx, const void* q, int64_t ldq, int64_t q_rows, void* out, int64_t ldo, const void* kv,
+                          int64_t ld_kv, const void* rot, int64_t ld_rot, int64_t k_rows, const int32_t* cu_q,
+                          const int32_t* cu_k, int B, int max_q, int heads, int dim_pad, int rot_pad, int v_pad,
+                          float scale, const float* sink, const float* cos_sin, int max_pos, const void* gate,
+                          int64_t ldg, void* stream);
 
 /* Greedy pick: out[i] = argmax_j logits[i, j] (first index on ties), int64.
  * The reference's Sampler (nanovllm/layers/sampler.py:7-12) at temperature -> 0. */

@@ -75,7 +75,7 @@ SIGNATURES = {
     "b2_latent_gather": [_i, _p, _p, _i64, _i, _p, _i, _i, _i, _p, _p],
     "b2_heads_gemm": [_i, _p, _i64, _i, _p, _i64, _i64, _i, _p, _i64, _i, _i, _i, _i, _i, _p, _i64, _i, _i, _p, _p, _i, _p],
     "b2_latent_attention": [_p, _i, _p, _i64, _p, _i64, _p, _i64, _p, _i64, _i, _p, _p, _i, _i, _i, _i, _i, _i, _f, _p, _p, _i64, _i, _p],
-    "b2_expanded_attention": [_p, _i64, _p, _i64, _p, _i64, _p, _i64, _p, _p, _i, _i, _i, _i, _i, _i, _f, _p, _p, _i, _p, _i64, _p],
+    "b2_expanded_attention": [_p, _p, _i64, _i64, _p, _i64, _p, _i64, _p, _i64, _i64, _p, _p, _i, _i, _i, _i, _i, _i, _f, _p, _p, _i, _p, _i64, _p],
     "b2_gemm_static_scratch": [_p, _i64, _p, _i64, _p, _p, _i64, _i, _i, _i, _p],
     "b2_rowpar_fused": [_p, _p, _i64, _p, _i64, _p, _i, _i, _i, _p, _p, _f, _p, _p, _p],
     "b2_ctx_set_option": [_p, _i, _i64],

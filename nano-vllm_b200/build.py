@@ -15,7 +15,7 @@ CSRC = os.path.join(HERE, "csrc")
 LIBDIR = os.path.join(HERE, "lib")
 LIB = os.path.join(LIBDIR, "libb200tp.so")
 SOURCES = ["b2_ctx.cu", "b2_elementwise.cu", "b2_gemm.cu", "b2_gemm_f32.cu", "b2_streams.cu", "b2_attention.cu", "b2_linear_attn.cu",
-           "b2_sandwich.cu", "b2_latent.cu"]
+           "b2_sandwich.cu", "b2_latent.cu", "b2_expanded.cu"]
 HEADERS = ["b2_common.cuh", "b2_vec.cuh", "b2_mma.cuh", "b2_attn.cuh", os.path.join("..", "..", "include", "b200tp.h")]
 NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17"]
 

@@ -70,6 +70,50 @@ __global__ void __launch_bounds__(256) qk_norm_store_kernel(T* qkv, int64_t ld, 
   }
 }
 
+// ---------------------------------------------------------------------------
+// Tensor-core kernels, bf16, head sizes up to 128.  The query heads that share a key/value head are rows of one tile
+// (row = token * rep + head), so K and V are read once per group.  Scores, softmax and weights are fp32; the weights
+// enter the product with V as a sum of two bf16 numbers.
+// ---------------------------------------------------------------------------
+constexpr int BN = 64;  // keys per tile
+
+// The key tiles a range of positions [pmin, pmax] looks at: those of the kept first tokens, then those of the window.
+struct KeyTiles {
+  int n_first, win0, total;
+  __device__ __forceinline__ KeyTiles(int pmin, int pmax, int window, int keep_first) {
+    const int lo = pmin - window + 1;
+    win0 = (lo > 0 ? lo : 0) / BN;
+    const int kept = min(keep_first, pmax + 1);
+    n_first = min((kept + BN - 1) / BN, win0);
+    total = n_first + pmax / BN - win0 + 1;
+  }
+  __device__ __forceinline__ int at(int i) const { return i < n_first ? i : win0 + (i - n_first); }
+};
+
+// Scores in units of log2: t = log2(e) * softcap(scale * s).  The three forms of the cap:
+enum { CAP_NONE = 0, CAP_SHORT = 1, CAP_FULL = 2 };
+struct ScoreScale {
+  float a, b, c;  // NONE: t = a s.  SHORT: t = c - b / (1 + 2^(a s)).  FULL: see score()
+};
+__host__ __device__ inline ScoreScale score_scale(int cap_form, float scale, float cap) {
+  constexpr float L = 1.4426950408889634f;
+  if (cap_form == CAP_NONE) return {scale * L, 0.f, 0.f};
+  return {2.0f * L * scale / cap, 2.0f * cap * L, cap * L};
+}
+// tanh(x) = 1 - 2 / (1 + e^2x) has an absolute error of about 1e-7, so the capped score is off by 1e-7 cap: below fp32
+// rounding of the scores themselves for caps up to a few hundred (SHORT).  FULL adds the Taylor series where the
+// difference would cancel, for any cap.
+template <int CAP>
+__device__ __forceinline__ float score(float s, const ScoreScale& k) {
+  if (CAP == CAP_NONE) return s * k.a;
+  const float z = s * k.a;  // 2 log2(e) x
+  const float t = fmaf(-k.b, __fdividef(1.0f, 1.0f + fast_exp2(fminf(z, 120.0f))), k.c);
+  if (CAP == CAP_SHORT) return t;
+  const float x = z * 0.34657359027997264f, x2 = x * x;
+  const float series = k.c * x * fmaf(x2, fmaf(x2, 0.13333333333f, -0.33333333333f), 1.0f);
+  return fabsf(x) < 0.125f ? series : t;
+}
+
 // The slot of key j of a sequence
 __device__ __forceinline__ int64_t slot_of(const AttnArgs& a, const int32_t* bt, int j) {
   const int blk = j / a.block_size;
@@ -109,6 +153,57 @@ __device__ __forceinline__ void load_kv_tile(const AttnArgs& a, const int32_t* b
   load_rows<DV>(a, static_cast<const uint16_t*>(a.v_cache), bt, whole, slot0, g, a.v_pad, tile, last, sv);
 }
 
+// One tile's scores of a warp: NT 8-key column tiles starting at key j0.  Scales, caps, masks (when `masked`), folds
+// into the running maximum m and sum l, and leaves the weights in s.  Returns the factors for the old outputs.
+template <int NT, int CAP>
+__device__ __forceinline__ void softmax_tile(const AttnArgs& a, const ScoreScale& k, float (&s)[NT][4], int j0, const int (&pos)[2], bool masked,
+                                             float (&m)[2], float (&l)[2], float (&corr)[2], int lane) {
+  float mx[2] = {-INFINITY, -INFINITY};
+#pragma unroll
+  for (int n = 0; n < NT; ++n)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) s[n][e] = score<CAP>(s[n][e], k);
+  if (masked) {
+#pragma unroll
+    for (int n = 0; n < NT; ++n)
+#pragma unroll
+      for (int e = 0; e < 4; ++e)
+        if (!visible(pos[e >> 1], j0 + n * 8 + (lane & 3) * 2 + (e & 1), a.window, a.keep_first)) s[n][e] = -INFINITY;
+  }
+#pragma unroll
+  for (int n = 0; n < NT; ++n)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) mx[e >> 1] = fmaxf(mx[e >> 1], s[n][e]);
+  float base[2];
+#pragma unroll
+  for (int h = 0; h < 2; ++h) {
+    mx[h] = fmaxf(mx[h], __shfl_xor_sync(0xffffffffu, mx[h], 1));
+    mx[h] = fmaxf(mx[h], __shfl_xor_sync(0xffffffffu, mx[h], 2));
+    const float m_new = fmaxf(m[h], mx[h]);
+    base[h] = m_new == -INFINITY ? 0.f : m_new;  // nothing visible yet: every weight is 2^-inf = 0
+    corr[h] = fast_exp2(m[h] - base[h]);
+    m[h] = m_new;
+  }
+  float sum[2] = {0.f, 0.f};
+#pragma unroll
+  for (int n = 0; n < NT; ++n)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const float p = fast_exp2(s[n][e] - base[e >> 1]);
+      s[n][e] = p;
+      sum[e >> 1] += p;
+    }
+#pragma unroll
+  for (int h = 0; h < 2; ++h) l[h] = fmaf(l[h], corr[h], sum[h]);  // this lane's part; summed over the row's four lanes at the end
+}
+
+template <int DQ, int DV>
+struct CfgTile {
+  static constexpr int STAGE = BN * (DQ + DV) * 2;
+  static constexpr int SMEM_PREFILL = 64 * DQ * 2 + 2 * STAGE + 128;
+  static constexpr int DEC_STAGES = 3;
+  static constexpr int SMEM_DECODE = 16 * DQ * 2 + DEC_STAGES * STAGE + 128;
+};
 
 // Prefill: 64 rows (token, head of the group) per CTA, 16 per warp; the four warps share the key tiles.
 template <int DQ, int DV, int CAP>
@@ -130,6 +225,7 @@ __global__ void __launch_bounds__(128, 2) attn_prefill_kernel(const AttnArgs a, 
   const int32_t* bt = a.block_tables + b * a.bt_stride;
   const int pmin = first_pos + tile0 / rep, pmax = first_pos + min(tile0 + 63, rows - 1) / rep;
   const KeyTiles tiles(pmin, pmax, a.window, a.keep_first);
+  const ScoreScale sscale = score_scale(CAP, a.scale, a.softcap);
   const uint16_t* q = static_cast<const uint16_t*>(a.q);
 #pragma unroll
   for (int i = 0; i < 64 * (DQ / 8) / 128; ++i) {
@@ -139,9 +235,71 @@ __global__ void __launch_bounds__(128, 2) attn_prefill_kernel(const AttnArgs a, 
     const int tok = ok ? gr / rep : 0, hh = ok ? gr - tok * rep : 0;
     b2::cp_async16(b2::tile_addr<DQ>(sq, r, p), q + (row0 + tok) * a.ldq + static_cast<int64_t>(g * rep + hh) * a.qk_pad + (ok ? p * 8 : 0), ok);
   }
-  auto load = [&](int tile, uint32_t sk, uint32_t sv) { load_kv_tile<DQ, DV>(a, bt, whole, g, tile, pmax, sk, sv); };
-  float m[2], l[2], o[DV / 8][4];
-  prefill_tiles<DQ, DV, CAP>(a, first_pos, tile0, rows, rep, tiles, sq, skv, load, [] {}, m, l, o);
+  load_kv_tile<DQ, DV>(a, bt, whole, g, tiles.at(0), pmax, skv, skv + BN * DQ * 2);
+  b2::cp_async_commit();
+  int pos[2];
+#pragma unroll
+  for (int h = 0; h < 2; ++h) pos[h] = first_pos + min(tile0 + warp * 16 + (lane >> 2) + h * 8, rows - 1) / rep;
+  const int wpmin = first_pos + min(tile0 + warp * 16, rows - 1) / rep;
+  const int wpmax = first_pos + min(tile0 + warp * 16 + 15, rows - 1) / rep;
+  float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
+  float o[DV / 8][4];
+#pragma unroll
+  for (int n = 0; n < DV / 8; ++n)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) o[n][e] = 0.f;
+  for (int it = 0; it < tiles.total; ++it) {
+    const uint32_t sk = skv + (it & 1) * CfgTile<DQ, DV>::STAGE, sv = sk + BN * DQ * 2;
+    b2::cp_async_wait<0>();
+    __syncthreads();  // this tile has landed for everyone, and everyone has left the stage that is filled next
+    if (it + 1 < tiles.total) {
+      const uint32_t nk = skv + ((it + 1) & 1) * CfgTile<DQ, DV>::STAGE;
+      load_kv_tile<DQ, DV>(a, bt, whole, g, tiles.at(it + 1), pmax, nk, nk + BN * DQ * 2);
+    }
+    b2::cp_async_commit();
+    const int j0 = tiles.at(it) * BN;
+    float s[BN / 8][4];
+#pragma unroll
+    for (int n = 0; n < BN / 8; ++n)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) s[n][e] = 0.f;
+#pragma unroll
+    for (int k = 0; k < DQ / 16; ++k) {
+      uint32_t qa[4];
+      b2::frag_a<DQ>(sq, warp * 16, k * 16, lane, qa);
+#pragma unroll
+      for (int n = 0; n < BN / 16; ++n) {
+        uint32_t kb[4];
+        b2::frag_b<DQ>(sk, n * 16, k * 16, lane, kb);
+        b2::mma16816(s[2 * n], qa, kb[0], kb[1]);
+        b2::mma16816(s[2 * n + 1], qa, kb[2], kb[3]);
+      }
+    }
+    const bool all_seen = j0 + BN - 1 <= wpmin && (wpmax - j0 < a.window || j0 + BN - 1 < a.keep_first);
+    float corr[2];
+    softmax_tile<BN / 8, CAP>(a, sscale, s, j0, pos, !all_seen, m, l, corr, lane);
+#pragma unroll
+    for (int n = 0; n < DV / 8; ++n) {
+      o[n][0] *= corr[0]; o[n][1] *= corr[0]; o[n][2] *= corr[1]; o[n][3] *= corr[1];
+    }
+#pragma unroll
+    for (int k = 0; k < BN / 16; ++k) {
+      uint32_t hi[4], lo[4];
+      b2::split_bf16(s[2 * k][0], s[2 * k][1], hi[0], lo[0]);
+      b2::split_bf16(s[2 * k][2], s[2 * k][3], hi[1], lo[1]);
+      b2::split_bf16(s[2 * k + 1][0], s[2 * k + 1][1], hi[2], lo[2]);
+      b2::split_bf16(s[2 * k + 1][2], s[2 * k + 1][3], hi[3], lo[3]);
+#pragma unroll
+      for (int n = 0; n < DV / 16; ++n) {
+        uint32_t vb[4];
+        b2::frag_b_t<DV>(sv, n * 16, k * 16, lane, vb);
+        b2::mma16816(o[2 * n], hi, vb[0], vb[1]);
+        b2::mma16816(o[2 * n + 1], hi, vb[2], vb[3]);
+        b2::mma16816(o[2 * n], lo, vb[0], vb[1]);
+        b2::mma16816(o[2 * n + 1], lo, vb[2], vb[3]);
+      }
+    }
+  }
   uint16_t* out = static_cast<uint16_t*>(a.out);
 #pragma unroll
   for (int h = 0; h < 2; ++h) {

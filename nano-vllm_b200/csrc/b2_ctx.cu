@@ -52,8 +52,7 @@ bool pdl_enabled() {
 }
 void count_launch() { g_launches.fetch_add(1, std::memory_order_relaxed); }
 
-int encode_tmap_2d(CUtensorMap* out, const void* base, uint64_t inner, uint64_t rows, uint64_t ld_elems,
-                   uint32_t box_inner, uint32_t box_rows) {
+static int encode_tmap(CUtensorMap* out, const void* base, int rank, const cuuint64_t* dims, const cuuint64_t* strides, const cuuint32_t* box) {
   if (g_encode == nullptr) {
     void* fn = nullptr;
     cudaDriverEntryPointQueryResult q;
@@ -65,21 +64,32 @@ int encode_tmap_2d(CUtensorMap* out, const void* base, uint64_t inner, uint64_t 
     }
     g_encode = reinterpret_cast<EncodeTiledFn>(fn);
   }
-  cuuint64_t dims[2] = {inner, rows};
-  cuuint64_t strides[1] = {ld_elems * 2};  // bytes between rows
-  cuuint32_t box[2] = {box_inner, box_rows};
-  cuuint32_t estr[2] = {1, 1};
-  CUresult r = g_encode(out, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(base), dims, strides, box, estr,
+  cuuint32_t estr[3] = {1, 1, 1};
+  CUresult r = g_encode(out, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, rank, const_cast<void*>(base), dims, strides, box, estr,
                         CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
                         CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
   if (r != CUDA_SUCCESS) {
     snprintf(g_last_error, sizeof(g_last_error),
-             "cuTensorMapEncodeTiled failed (%d): base=%p inner=%llu rows=%llu ld=%llu box=%ux%u", static_cast<int>(r), base,
-             static_cast<unsigned long long>(inner), static_cast<unsigned long long>(rows),
-             static_cast<unsigned long long>(ld_elems), box_inner, box_rows);
+             "cuTensorMapEncodeTiled failed (%d): base=%p rank=%d inner=%llu rows=%llu row bytes=%llu box=%ux%u", static_cast<int>(r), base, rank,
+             static_cast<unsigned long long>(dims[0]), static_cast<unsigned long long>(dims[rank - 1]),
+             static_cast<unsigned long long>(strides[rank - 2]), box[0], box[rank - 1]);
     return B2_ERR_CUDA;
   }
   return B2_OK;
+}
+
+int encode_tmap_2d(CUtensorMap* out, const void* base, uint64_t inner, uint64_t rows, uint64_t ld_elems,
+                   uint32_t box_inner, uint32_t box_rows) {
+  const cuuint64_t dims[2] = {inner, rows}, strides[1] = {ld_elems * 2};  // bytes between rows
+  const cuuint32_t box[2] = {box_inner, box_rows};
+  return encode_tmap(out, base, 2, dims, strides, box);
+}
+
+int encode_tmap_heads(CUtensorMap* out, const void* base, uint64_t inner, uint64_t heads, uint64_t head_elems, uint64_t rows, uint64_t ld_elems,
+                      uint32_t box_inner, uint32_t box_rows) {
+  const cuuint64_t dims[3] = {inner, heads, rows}, strides[2] = {head_elems * 2, ld_elems * 2};
+  const cuuint32_t box[3] = {box_inner, 1, box_rows};
+  return encode_tmap(out, base, 3, dims, strides, box);
 }
 }  // namespace b2
 

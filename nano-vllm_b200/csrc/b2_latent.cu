@@ -10,7 +10,7 @@
 //   heads_gemm_kernel      one small matrix product per head, with the rotation of the query part or an output gate
 //   latent_tc_kernel       absorbed attention on tcgen05: 16 or 32 (token, head) rows, 128 keys per tile
 //   latent_combine_kernel  the parts of its key ranges
-//   expanded_attn_kernel   expanded attention, 64 tokens of one head x 64 keys; rotates the queries it loads, gates its output
+// (The expanded form is in b2_expanded.cu.)
 #include <algorithm>
 
 #include "b2_attn.cuh"
@@ -18,22 +18,6 @@
 namespace {
 
 using namespace b2;
-
-// cos/sin of one rotated pair: table [max_pos][rot_pad / 2] of (cos, sin)
-__device__ __forceinline__ float2 rot_at(const float2* cs, int max_pos, int half, int64_t pos, int pair) {
-  const int64_t p = pos < 0 ? 0 : pos >= max_pos ? max_pos - 1 : pos;
-  return __ldg(cs + p * half + pair);
-}
-// (u, v) -> (u cos - v sin, v cos + u sin) on the four pairs of 8 elements
-__device__ __forceinline__ void rotate8(float (&f)[8], const float2* cs, int max_pos, int half, int64_t pos, int pair0) {
-#pragma unroll
-  for (int i = 0; i < 4; ++i) {
-    const float2 r = rot_at(cs, max_pos, half, pos, pair0 + i);
-    const float u = f[2 * i], v = f[2 * i + 1];
-    f[2 * i] = u * r.x - v * r.y;
-    f[2 * i + 1] = v * r.x + u * r.y;
-  }
-}
 
 // ---------------------------------------------------------------------------
 // Rows [q latent | latent | rotated part | ...] in place; [latent | rotated part] also to the cache.  One warp per
@@ -159,17 +143,16 @@ __device__ __forceinline__ void rotate_rows(const HeadsArgs& a, int m0, int h) {
   }
 }
 
-// Output tiles of 64 x NT, K in steps of 64 of which HEADS_STAGES - 1 are in flight
-constexpr int HEADS_STAGES = 4;
-template <bool KN>
+// Output tiles of 64 x NT; K in steps of 64, STAGES of them in flight
+template <bool KN, int STAGES>
 struct CfgHeads {
   static constexpr int NT = KN ? 64 : 32;
   static constexpr int A_BYTES = 64 * 64 * 2, STAGE = A_BYTES + 64 * NT * 2;
-  static constexpr int SMEM = HEADS_STAGES * STAGE + 128;
+  static constexpr int SMEM = STAGES * STAGE + 128;
 };
-template <bool KN>
+template <bool KN, int STAGES>
 __global__ void __launch_bounds__(128) heads_gemm_kernel(const HeadsArgs a) {
-  using C = CfgHeads<KN>;
+  using C = CfgHeads<KN, STAGES>;
   constexpr int NT = C::NT;
   extern __shared__ unsigned char smem_raw[];
   const uint32_t base = (smem_u32(smem_raw) + 127) & ~127u;
@@ -200,14 +183,13 @@ __global__ void __launch_bounds__(128) heads_gemm_kernel(const HeadsArgs a) {
   const bool product = n0 < a.N;
   // weights do not depend on an earlier kernel: the first ones are fetched before the wait
   if (product)
-    for (int i = 0; i < HEADS_STAGES - 1; ++i)
-      if (i * 64 < a.K) load_w(i, i * 64);
+    for (int i = 0; i < STAGES && i * 64 < a.K; ++i) load_w(i, i * 64);
   pdl_wait();
   if (!product) {
     rotate_rows<uint16_t>(a, m0, h);
     return;
   }
-  for (int i = 0; i < HEADS_STAGES - 1; ++i) {
+  for (int i = 0; i < STAGES; ++i) {
     if (i * 64 < a.K) load_x(i, i * 64);
     cp_async_commit();
   }
@@ -216,16 +198,10 @@ __global__ void __launch_bounds__(128) heads_gemm_kernel(const HeadsArgs a) {
   for (int n = 0; n < NT / 8; ++n)
 #pragma unroll
     for (int e = 0; e < 4; ++e) acc[n][e] = 0.f;
-  for (int k0 = 0, it = 0; k0 < a.K; k0 += 64, ++it) {
-    cp_async_wait<HEADS_STAGES - 2>();
-    __syncthreads();  // this step has landed, and everyone has left the stage that is filled next
-    const int ahead = k0 + 64 * (HEADS_STAGES - 1);
-    if (ahead < a.K) {
-      load_w((it + HEADS_STAGES - 1) % HEADS_STAGES, ahead);
-      load_x((it + HEADS_STAGES - 1) % HEADS_STAGES, ahead);
-    }
-    cp_async_commit();
-    const uint32_t sa = base + (it % HEADS_STAGES) * C::STAGE, sw = sa + C::A_BYTES;
+  for (int k0 = 0, st = 0; k0 < a.K; k0 += 64, st = st + 1 == STAGES ? 0 : st + 1) {
+    cp_async_wait<STAGES - 1>();
+    __syncthreads();  // this step has landed for everyone
+    const uint32_t sa = base + st * C::STAGE, sw = sa + C::A_BYTES;
 #pragma unroll
     for (int k = 0; k < 4; ++k) {
       uint32_t qa[4];
@@ -239,6 +215,12 @@ __global__ void __launch_bounds__(128) heads_gemm_kernel(const HeadsArgs a) {
         mma16816(acc[2 * n + 1], qa, kb[2], kb[3]);
       }
     }
+    if (k0 + 64 * STAGES < a.K) {
+      __syncthreads();  // everyone has left the stage
+      load_w(st, k0 + 64 * STAGES);
+      load_x(st, k0 + 64 * STAGES);
+    }
+    cp_async_commit();
   }
 #pragma unroll
   for (int e = 0; e < 2; ++e) {
@@ -261,11 +243,13 @@ __global__ void __launch_bounds__(128) heads_gemm_kernel(const HeadsArgs a) {
   }
 }
 
-template <bool KN>
-int launch_heads(const HeadsArgs& a, dim3 grid, cudaStream_t s) {
-  static const cudaError_t set = cudaFuncSetAttribute(heads_gemm_kernel<KN>, cudaFuncAttributeMaxDynamicSharedMemorySize, CfgHeads<KN>::SMEM);
+template <bool KN, int STAGES>
+int launch_heads(const HeadsArgs& a, int heads, cudaStream_t s) {
+  using C = CfgHeads<KN, STAGES>;
+  static const cudaError_t set = cudaFuncSetAttribute(heads_gemm_kernel<KN, STAGES>, cudaFuncAttributeMaxDynamicSharedMemorySize, C::SMEM);
   B2_CUDA(set);
-  B2_CUDA(b2_launch(heads_gemm_kernel<KN>, grid, dim3(128), CfgHeads<KN>::SMEM, s, a));
+  const dim3 grid((a.N + C::NT - 1) / C::NT + (a.rot_pad > 0 ? 1 : 0), (a.M + 63) / 64, heads);
+  B2_CUDA(b2_launch(heads_gemm_kernel<KN, STAGES>, grid, dim3(128), C::SMEM, s, a));
   return B2_OK;
 }
 
@@ -787,118 +771,6 @@ int launch_latent(const b2_ctx* ctx, const AttnArgs& a, int64_t slots, int64_t q
   return B2_OK;
 }
 
-// ---------------------------------------------------------------------------
-// Expanded attention
-// ---------------------------------------------------------------------------
-struct ExpandedArgs {
-  const uint16_t* kv;  // rows [heads][dim_pad key | v_pad value], row cu_k[b] + j = position j
-  int64_t ld_kv;
-  const uint16_t* rot;  // rotated key parts of the same rows
-  int64_t ld_rot;
-  const int32_t* cu_k;
-  int dim_pad, rot_pad;
-  const float2* cs;
-  int max_pos;
-  const uint16_t* gate;  // [M][heads][v_pad] or null
-  int64_t ldg;
-};
-
-template <int DQ, int DV>
-__global__ void __launch_bounds__(128, 2) expanded_attn_kernel(const AttnArgs a, const ExpandedArgs e) {
-  extern __shared__ unsigned char smem_raw[];
-  const uint32_t base = (smem_u32(smem_raw) + 127) & ~127u;
-  const uint32_t sq = base, skv = base + 64 * DQ * 2;
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  pdl_launch_dependents();
-  pdl_wait();
-  const int b = blockIdx.z, h = blockIdx.y;
-  const int row0 = a.cu_q[b], rows = a.cu_q[b + 1] - row0;
-  const int tile0 = (static_cast<int>(gridDim.x) - 1 - static_cast<int>(blockIdx.x)) * 64;  // the longest rows first
-  if (tile0 >= rows) return;
-  const int key0 = e.cu_k[b], first_pos = e.cu_k[b + 1] - key0 - rows;
-  const int pmin = first_pos + tile0, pmax = first_pos + min(tile0 + 63, rows - 1);
-  const KeyTiles tiles(pmin, pmax, a.window, a.keep_first);
-  constexpr int PQ = DQ / 8, PV = DV / 8;
-  const uint16_t* q = static_cast<const uint16_t*>(a.q) + row0 * a.ldq + static_cast<int64_t>(h) * a.qk_pad;
-#pragma unroll 4
-  for (int i = 0; i < 64 * PQ / 128; ++i) {
-    const int idx = threadIdx.x + i * 128, r = idx / PQ, p = idx % PQ;
-    const bool ok = tile0 + r < rows && p * 8 < a.qk_pad;
-    cp_async16(tile_addr<DQ>(sq, r, p), ok ? q + (tile0 + r) * a.ldq + p * 8 : q, ok);
-  }
-  const int dim8 = e.dim_pad >> 3, all8 = dim8 + (e.rot_pad >> 3), v8 = a.v_pad >> 3;
-  const uint16_t* kvh = e.kv + key0 * e.ld_kv + static_cast<int64_t>(h) * (e.dim_pad + a.v_pad);
-  const uint16_t* rot = e.rot + key0 * e.ld_rot;
-  auto load = [&](int tile, uint32_t sk, uint32_t sv) {
-#pragma unroll 4
-    for (int i = 0; i < 64 * PQ / 128; ++i) {
-      const int idx = threadIdx.x + i * 128, r = idx / PQ, p = idx % PQ, j = tile * BN + r;
-      const bool ok = p < all8 && j <= pmax;
-      const uint16_t* src = p < dim8 ? kvh + j * e.ld_kv + p * 8 : rot + j * e.ld_rot + (p - dim8) * 8;
-      cp_async16(tile_addr<DQ>(sk, r, p), ok ? src : kvh, ok);
-    }
-#pragma unroll 4
-    for (int i = 0; i < 64 * PV / 128; ++i) {
-      const int idx = threadIdx.x + i * 128, r = idx / PV, p = idx % PV, j = tile * BN + r;
-      const bool ok = p < v8 && j <= pmax;
-      cp_async16(tile_addr<DV>(sv, r, p), ok ? kvh + j * e.ld_kv + e.dim_pad + p * 8 : kvh, ok);
-    }
-  };
-  auto rotate_q = [&] {
-    cp_async_wait<0>();
-    __syncthreads();
-    const int rot8 = e.rot_pad >> 3;
-    for (int idx = threadIdx.x; idx < 64 * rot8; idx += 128) {
-      const int r = idx / rot8, p = idx % rot8;
-      uint16_t* at = reinterpret_cast<uint16_t*>(smem_raw + (tile_addr<DQ>(sq, r, dim8 + p) - smem_u32(smem_raw)));
-      float f[8];
-      load8<uint16_t>(at, f);
-      rotate8(f, e.cs, e.max_pos, e.rot_pad >> 1, first_pos + tile0 + r, p * 4);
-      store8<uint16_t>(at, f);
-    }
-  };
-  float m[2], l[2], o[DV / 8][4];
-  prefill_tiles<DQ, DV, CAP_NONE>(a, first_pos, tile0, rows, 1, tiles, sq, skv, load, rotate_q, m, l, o);
-  uint16_t* out = static_cast<uint16_t*>(a.out) + static_cast<int64_t>(h) * a.v_pad;
-#pragma unroll
-  for (int i = 0; i < 2; ++i) {
-    l[i] += __shfl_xor_sync(0xffffffffu, l[i], 1);
-    l[i] += __shfl_xor_sync(0xffffffffu, l[i], 2);
-    const int r = tile0 + warp * 16 + (lane >> 2) + i * 8;
-    if (r >= rows) continue;
-    float f = 1.0f;
-    if (a.sink != nullptr) {
-      const float sk = a.sink[h] * LOG2E, m_new = fmaxf(m[i], sk);
-      f = fast_exp2(m[i] - m_new);
-      l[i] = l[i] * f + fast_exp2(sk - m_new);
-    }
-    f /= l[i];
-    uint16_t* dst = out + (row0 + r) * a.ldo;
-    const uint16_t* g = e.gate != nullptr ? e.gate + (row0 + r) * e.ldg + static_cast<int64_t>(h) * a.v_pad : nullptr;
-#pragma unroll
-    for (int n = 0; n < DV / 8; ++n) {
-      const int c = n * 8 + (lane & 3) * 2;
-      if (c >= a.v_pad) continue;
-      float u = o[n][2 * i] * f, v = o[n][2 * i + 1] * f;
-      if (g != nullptr) {
-        const uint32_t gv = *reinterpret_cast<const uint32_t*>(g + c);
-        u *= sigmoid_fast(bf16_lo(gv));
-        v *= sigmoid_fast(bf16_hi(gv));
-      }
-      *reinterpret_cast<uint32_t*>(dst + c) = pack_bf16(u, v);
-    }
-  }
-}
-
-template <int DQ, int DV>
-int launch_expanded(const AttnArgs& a, const ExpandedArgs& e, int max_q, cudaStream_t s) {
-  constexpr int SMEM = CfgTile<DQ, DV>::SMEM_PREFILL;
-  static const cudaError_t set = cudaFuncSetAttribute(expanded_attn_kernel<DQ, DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM);
-  B2_CUDA(set);
-  B2_CUDA(b2_launch(expanded_attn_kernel<DQ, DV>, dim3((max_q + 63) / 64, a.nq, a.B), dim3(128), SMEM, s, a, e));
-  return B2_OK;
-}
-
 bool bad_dtype(int dtype) { return dtype != B2_DT_BF16 && dtype != B2_DT_F32; }
 
 }  // namespace
@@ -954,12 +826,12 @@ int b2_heads_gemm(int dtype, const void* x, int64_t ldx, int x_head, const void*
   a.M = M; a.N = N; a.K = K; a.gate = gate; a.ldg = ldg; a.gate_hs = gate_head; a.rot_pad = rot_pad; a.positions = positions;
   a.cs = reinterpret_cast<const float2*>(cos_sin); a.max_pos = max_pos;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  const int nt = dtype == B2_DT_BF16 && !w_is_kn ? CfgHeads<false>::NT : 64;
-  const dim3 grid((N + nt - 1) / nt + (rot_pad > 0 ? 1 : 0), (M + 63) / 64, heads);
   if (dtype == B2_DT_BF16) {
-    if (w_is_kn) return launch_heads<true>(a, grid, s);
-    return launch_heads<false>(a, grid, s);
-  } else {
+    if (K <= 128) return w_is_kn ? launch_heads<true, 2>(a, heads, s) : launch_heads<false, 2>(a, heads, s);
+    return w_is_kn ? launch_heads<true, 8>(a, heads, s) : launch_heads<false, 8>(a, heads, s);
+  }
+  {
+    const dim3 grid((N + 63) / 64 + (rot_pad > 0 ? 1 : 0), (M + 63) / 64, heads);
     if (w_is_kn) B2_CUDA(b2_launch(heads_gemm_f32_kernel<true>, grid, dim3(256), 0, s, a));
     else B2_CUDA(b2_launch(heads_gemm_f32_kernel<false>, grid, dim3(256), 0, s, a));
   }
@@ -997,31 +869,6 @@ int b2_latent_attention(b2_ctx* ctx, int dtype, const void* q, int64_t q_rows, v
                      static_cast<long long>(p.bytes));
   return p.rows == 16 ? launch_latent<16>(ctx, a, cache_slots, q_rows * heads, rot_pad, p, workspace, s)
                       : launch_latent<32>(ctx, a, cache_slots, q_rows * heads, rot_pad, p, workspace, s);
-}
-
-int b2_expanded_attention(const void* q, int64_t ldq, void* out, int64_t ldo, const void* kv, int64_t ld_kv, const void* rot, int64_t ld_rot,
-                          const int32_t* cu_q, const int32_t* cu_k, int B, int max_q, int heads, int dim_pad, int rot_pad, int v_pad, float scale,
-                          const float* sink, const float* cos_sin, int max_pos, const void* gate, int64_t ldg, void* stream) {
-  if (B < 0 || max_q < 0 || heads <= 0 || dim_pad < 0 || rot_pad < 0 || v_pad <= 0 || dim_pad % 8 != 0 || rot_pad % 8 != 0 || v_pad % 8 != 0) return B2_ERR_ARG;
-  if (dim_pad + rot_pad <= 0) return B2_ERR_ARG;
-  if (B == 0 || max_q == 0) return B2_OK;
-  if (!q || !out || !kv || !cu_q || !cu_k || !aligned16(q) || !aligned16(out) || !aligned16(kv)) return B2_ERR_ARG;
-  if (ldq % 8 != 0 || ldo % 8 != 0 || ld_kv % 8 != 0 || ld_rot % 8 != 0) return B2_ERR_ARG;
-  if (rot_pad > 0 && (!rot || !aligned16(rot) || !cos_sin || max_pos <= 0)) return B2_ERR_ARG;
-  if (gate != nullptr && (!aligned16(gate) || ldg % 8 != 0)) return B2_ERR_ARG;
-  if (dim_pad + rot_pad > 192 || v_pad > 128 || B > 65535 || heads > 65535) return B2_ERR_SHAPE;
-  AttnArgs a{};
-  a.q = q; a.ldq = ldq; a.out = out; a.ldo = ldo; a.cu_q = cu_q; a.B = B; a.nq = heads; a.nkv = heads;
-  a.qk_pad = dim_pad + rot_pad; a.v_pad = v_pad; a.window = INT_MAX; a.scale = scale; a.sink = sink;
-  ExpandedArgs e{};
-  e.kv = static_cast<const uint16_t*>(kv); e.ld_kv = ld_kv;
-  e.rot = rot_pad > 0 ? static_cast<const uint16_t*>(rot) : e.kv; e.ld_rot = ld_rot;
-  e.cu_k = cu_k; e.dim_pad = dim_pad; e.rot_pad = rot_pad; e.cs = reinterpret_cast<const float2*>(cos_sin); e.max_pos = max_pos;
-  e.gate = static_cast<const uint16_t*>(gate); e.ldg = ldg;
-  cudaStream_t s = static_cast<cudaStream_t>(stream);
-  const int dq = dim_pad + rot_pad;
-  if (v_pad <= 64) return dq <= 64 ? launch_expanded<64, 64>(a, e, max_q, s) : dq <= 128 ? launch_expanded<128, 64>(a, e, max_q, s) : launch_expanded<192, 64>(a, e, max_q, s);
-  return dq <= 64 ? launch_expanded<64, 128>(a, e, max_q, s) : dq <= 128 ? launch_expanded<128, 128>(a, e, max_q, s) : launch_expanded<192, 128>(a, e, max_q, s);
 }
 
 }  // extern "C"

@@ -79,4 +79,20 @@ __device__ __forceinline__ float sigmoid(float x) { return 1.0f / (1.0f + expf(-
 // a few units in the last place of fp32: for values that are rounded to bf16
 __device__ __forceinline__ float sigmoid_fast(float x) { return __fdividef(1.0f, 1.0f + __expf(-x)); }
 
+// cos/sin of one rotated pair: table [max_pos][rot_pad / 2] of (cos, sin)
+__device__ __forceinline__ float2 rot_at(const float2* cs, int max_pos, int half, int64_t pos, int pair) {
+  const int64_t p = pos < 0 ? 0 : pos >= max_pos ? max_pos - 1 : pos;
+  return __ldg(cs + p * half + pair);
+}
+// (u, v) -> (u cos - v sin, v cos + u sin) on the four pairs of 8 elements
+__device__ __forceinline__ void rotate8(float (&f)[8], const float2* cs, int max_pos, int half, int64_t pos, int pair0) {
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const float2 r = rot_at(cs, max_pos, half, pos, pair0 + i);
+    const float u = f[2 * i], v = f[2 * i + 1];
+    f[2 * i] = u * r.x - v * r.y;
+    f[2 * i + 1] = v * r.x + u * r.y;
+  }
+}
+
 }  // namespace b2

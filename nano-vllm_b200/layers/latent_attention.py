@@ -103,7 +103,9 @@ class LatentAttention(nn.Module):
         return self.o_proj(attend(q, p[:, l0:g0], gate, positions, cache, ctx))
 
     def _expands(self, x: torch.Tensor, ctx) -> bool:
-        if not ctx.is_prefill or x.dtype != torch.bfloat16 or self.dim_pad + self.rot_pad > 192 or self.v_pad > 128 or self.form in ("absorbed", "any"):
+        if not ctx.is_prefill or x.dtype != torch.bfloat16 or self.form in ("absorbed", "any"):
+            return False
+        if self.dim_pad > 128 or self.rot_pad > 64 or self.v_pad > 128 or self.scale <= 0:  # the kernel's tiles
             return False
         if self.form == "expanded":
             return True

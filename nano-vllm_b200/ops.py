@@ -536,13 +536,13 @@ def expanded_attention(q: torch.Tensor, heads: int, kv: torch.Tensor, rot: torch
     """Attention of the unrotated q [M, heads * (dim_pad + rot_pad)] over contiguous rows kv [keys, heads * (dim_pad + v_pad)]
     and rot [keys, rot_pad]; the output is multiplied by sigmoid(gate)."""
     M = q.shape[0]
-    assert q.dtype == kv.dtype == rot.dtype == torch.bfloat16 and q.stride(1) == kv.stride(1) == rot.stride(1) == 1
+    assert q.dtype == kv.dtype == rot.dtype == torch.bfloat16 and q.stride(1) == kv.stride(1) == rot.stride(1) == 1 and rot.shape[0] == kv.shape[0]
     assert cu_q.dtype == cu_k.dtype == torch.int32 and cos_sin.is_contiguous() and (sink is None or sink.dtype == torch.float32)
     assert gate is None or (gate.dtype == q.dtype and gate.stride(1) == 1)
     out = torch.empty(M, heads * v_pad, dtype=q.dtype, device=q.device)
-    _abi.check(_lib.b2_expanded_attention(q.data_ptr(), q.stride(0), out.data_ptr(), out.stride(0), kv.data_ptr(), kv.stride(0), rot.data_ptr(),
-                                          rot.stride(0), cu_q.data_ptr(), cu_k.data_ptr(), cu_q.numel() - 1, max_q, heads, dim_pad, rot_pad, v_pad,
-                                          float(scale), _ptr(sink), cos_sin.data_ptr(), cos_sin.shape[0], _ptr(gate),
+    _abi.check(_lib.b2_expanded_attention(get_runtime().ctx, q.data_ptr(), q.stride(0), M, out.data_ptr(), out.stride(0), kv.data_ptr(), kv.stride(0),
+                                          rot.data_ptr(), rot.stride(0), kv.shape[0], cu_q.data_ptr(), cu_k.data_ptr(), cu_q.numel() - 1, max_q, heads,
+                                          dim_pad, rot_pad, v_pad, float(scale), _ptr(sink), cos_sin.data_ptr(), cos_sin.shape[0], _ptr(gate),
                                           gate.stride(0) if gate is not None else 0, _stream()), "b2_expanded_attention")
     return out
 

@@ -392,8 +392,15 @@ def run_expanded(heads, d, rot, dv, lens, q_lens, seed=0, scale=0.12, gated=True
         at += n
 
 
-@pytest.mark.parametrize("heads,d,rot,dv", [(3, 20, 12, 28), (2, 40, 20, 72), (4, 64, 64, 64), (2, 128, 64, 128), (1, 72, 2, 16), (2, 160, 32, 40)])
+@pytest.mark.parametrize("heads,d,rot,dv", [(3, 20, 12, 28), (2, 40, 20, 72), (4, 64, 64, 64), (2, 128, 64, 128), (1, 72, 2, 16), (2, 120, 40, 100), (5, 8, 8, 8)])
 def test_expanded_attention(heads, d, rot, dv):
     run_expanded(heads, d, rot, dv, [1, 70, 150, 129, 66], [1, 70, 21, 1, 2])
     run_expanded(heads, d, rot, dv, [130, 64, 65], [130, 64, 63], seed=1, gated=False)
     run_expanded(heads, d, rot, dv, [300, 257, 40], [300, 130, 40], seed=2)
+
+
+def test_expanded_attention_over_many_tiles():
+    """Longer sequences: every slot of the rings is used again, both query tiles and one of them alone, a late short portion."""
+    run_expanded(2, 128, 64, 128, [900, 1100, 513], [900, 600, 129], seed=3)
+    run_expanded(1, 64, 32, 64, [1500, 700], [300, 3], seed=4)
+    run_expanded(3, 72, 8, 104, [640, 641], [640, 257], seed=5, scale=0.4)  # sharp scores: outputs are rescaled on the way
