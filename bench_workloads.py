@@ -265,7 +265,7 @@ def _model_throughput(torch, cfg: dict, vocab: int, batch: int, prompt: int, ste
 
 class KernelTable:
     """Rows (kernel, microseconds, fraction of the roofline) beside the like kernel of another model.  Rooflines: the measured
-    copy bandwidth or burst bf16 throughput, or (bound "sum") seconds the caller has added up from both."""
+    copy bandwidth or burst bf16 throughput, or (bound "sum") seconds the caller has worked out from both."""
 
     def __init__(self, peaks: dict):
         self.peaks, self.rows = peaks, []
@@ -543,21 +543,21 @@ def _mupulorn_kernels(torch, z: dict, peaks: dict, batch: int, ctx_len: int) -> 
             ws = [rnd(N, K, k=0.02) for _ in range(max(2, min(24, int(3e8 / (N * K * 2)) + 1)))]
             x = rnd(M, K)
             return time_in_graph(lambda i: ops.gemm(x, ws[i]), len(ws), 4 * len(ws))
-        work = lambda N, K: 2.0 * M * N * K if M > 1000 else 2.0 * (N * K + M * K + M * N)
-        bound = "tensor" if M > 1000 else "hbm"
+        # seconds at the slower of the two rooflines (a short K makes even a product of many tokens bound by its output)
+        work = lambda N, K: max(2.0 * M * N * K / tensor, 2.0 * (N * K + M * K + M * N) / hbm)
         Nq = (H + 2 * G) * d
         qkv_us = gemm_us(Nq, W)
         for nm, N, K in (("in_proj", Q + row + H * d, W), ("q_proj", H * qh, Q), ("up_proj", ff, W)) + ((("kv_proj", H * 2 * d, L),) if M > 1000 else ()):
-            add(f"{nm} M={M}", "qkv projection GEMM", work(N, K), gemm_us(N, K), work(Nq, W), qkv_us, bound)
+            add(f"{nm} M={M}", "qkv projection GEMM", work(N, K), gemm_us(N, K), work(Nq, W), qkv_us, "sum")
         if M == batch:  # per-head products of the absorbed form
             ws = [rnd(H, 2 * d, L, k=0.05) for _ in range(max(2, min(48, int(3e8 / (H * 2 * d * L * 2)) + 1)))]
             q, o, gate = rnd(M, H * qh), rnd(M, H * L), rnd(M, H * d)
             nb = 2.0 * (H * d * L + M * H * (qh + row))
             us = time_in_graph(lambda i: ops.heads_gemm(q, qh, ws[i][:, :d], True, row, rotate=(rot, pos, rope.table)), len(ws), 4 * len(ws))
-            add(f"heads_gemm q Wk + rotation M={M}", "qkv projection GEMM", nb, us, work(Nq, W), qkv_us, "hbm")
+            add(f"heads_gemm q Wk + rotation M={M}", "qkv projection GEMM", nb / hbm, us, work(Nq, W), qkv_us, "sum")
             nb = 2.0 * (H * d * L + M * H * (L + 2 * d))
             us = time_in_graph(lambda i: ops.heads_gemm(o, L, ws[i][:, d:], False, d, gate=gate, gate_head=d), len(ws), 4 * len(ws))
-            add(f"heads_gemm Wv + gate M={M}", "qkv projection GEMM", nb, us, work(Nq, W), qkv_us, "hbm")
+            add(f"heads_gemm Wv + gate M={M}", "qkv projection GEMM", nb / hbm, us, work(Nq, W), qkv_us, "sum")
             del ws
     sink = torch.zeros(H, device=dev)
     # prompts: 4 sequences of 2048, full causal
