@@ -20,6 +20,10 @@ cases:
   linear_prefill  decayed linear attention, 4 prompts of 2048, 32 heads of 128 x 128
   linear_decode   the same for 64 sequences, one row each, 4 layers' states
   stream_step     residual streams (4) between two sublayers, 8192 x 4096
+  latent_decode   absorbed latent attention (tcgen05), 64 sequences of 1024 tokens, 32 heads, latent 512 + 64, 4 layers' caches
+  latent_prefill  expanded latent attention (tcgen05), 4 prompts of 2048, 32 heads of 128 + 64 / 128, gate
+  sandwich_step   residual, two norms and a 4-tap convolution between two sublayers, 4 prompts of 2048 x 4096
+  poly_norm       PolyNorm of 8192 rows of 18432
   embed           embedding lookup, 16384 ids into a [151936, 4096] table (one rank)
 """
 from __future__ import annotations
@@ -114,6 +118,29 @@ def main():
         x, y = torch.randn(8192, 4, 4096, device=dev), rnd(8192, 4096)
         mix, one, nw = torch.eye(4, device=dev), torch.ones(4, device=dev), torch.ones(4096, device=dev)
         call = lambda i: ops.stream_step(x, y, mix, one, 0.1, one / 4, nw, 1e-6, 4096)
+    elif a.case == "latent_decode":
+        heads, lat, rot, seqs, length, layers = 32, 512, 64, 64, 1024, 4
+        caches = [rnd(seqs * length // 256, 256, 1, lat + rot) for _ in range(layers)]
+        bt = torch.randperm(seqs * length // 256, device=dev, generator=g).int().view(seqs, -1).contiguous()
+        kl, q, sink = torch.full((seqs,), length, dtype=torch.int32, device=dev), rnd(seqs, heads * (lat + rot)), torch.zeros(heads, device=dev)
+        call = lambda i: ops.latent_attention(q, heads, caches[i % layers], lat, bt, None, kl, 1, length, 0.05, sink)
+    elif a.case == "latent_prefill":
+        heads, d, rot, seqs, length = 32, 128, 64, 4, 2048
+        rows = seqs * length
+        cu = torch.arange(0, rows + 1, length, device=dev, dtype=torch.int32)
+        q, kv, kr, gate = rnd(rows, heads * (d + rot)), rnd(rows, heads * 2 * d), rnd(rows, rot), rnd(rows, heads * d)
+        table, sink = torch.ones(length, rot // 2, 2, device=dev), torch.zeros(heads, device=dev)
+        call = lambda i: ops.expanded_attention(q, heads, kv, kr, cu, cu, length, d, rot, d, 0.07, sink, table, gate)
+    elif a.case == "sandwich_step":
+        rows, w, taps, seqs = 8192, 4096, 4, 4
+        cu = torch.arange(0, rows + 1, rows // seqs, device=dev, dtype=torch.int32)
+        batch = (cu, torch.full((seqs,), rows // seqs, dtype=torch.int32, device=dev), torch.arange(seqs, device=dev, dtype=torch.int32), rows // seqs)
+        x, y, one = torch.randn(rows, w, device=dev), rnd(rows, w), torch.ones(1, device=dev)
+        conv, state = rnd(taps, w, scale=0.1), rnd(seqs, taps - 1, w)
+        call = lambda i: ops.sandwich_step(x, y, one, one, 1e-6, w, batch, conv, state)
+    elif a.case == "poly_norm":
+        z, coef = rnd(8192, 18432), torch.full((4,), 0.3, device=dev)
+        call = lambda i: ops.poly_norm(z, coef, 1e-6, 18432)
     elif a.case == "embed":
         w = rnd(151936, 4096)
         ids = [torch.randint(0, 151936, (16384,), device=dev, generator=g) for _ in range(2)]
