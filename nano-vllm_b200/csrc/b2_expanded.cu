@@ -7,7 +7,8 @@
 //     O += P V        P in tensor memory where S was, as a leading and a trailing bf16 part; V rows are used as they lie
 // While one tile's softmax runs, the tensor cores work for the other tile: P0 V, S0 of the next keys, P1 V, S1 ...
 // Copies land in boxes of 128 rows x 64 columns (16 KB).  Key and value boxes share a ring of three pairs (keys of tile t,
-// values of t, keys of t + 1, ...); the rotated key part has two boxes of its own.
+// values of t, keys of t + 1, ...); the rotated key part has two boxes of its own, copied together with the keys: the slot that
+// keys of tile t go to held the values of tile t - 2, whose last use comes after the last use of the keys of tile t - 2.
 #include <algorithm>
 
 #include "b2_attn.cuh"
@@ -41,23 +42,23 @@ __global__ void __launch_bounds__(EX_THREADS, 1)
 expanded_attn_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_qr, const __grid_constant__ CUtensorMap tm_k,
                      const __grid_constant__ CUtensorMap tm_kr, const __grid_constant__ CUtensorMap tm_v, const ExpandedArgs a) {
   extern __shared__ unsigned char smem_raw[];
-  __shared__ __align__(8) uint64_t s_bars[20];
+  __shared__ __align__(8) uint64_t s_bars[16];
   __shared__ uint32_t s_tmem;
   __shared__ int s_abort;
   volatile int* abort_flag = &s_abort;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const uint32_t sq = (smem_u32(smem_raw) + 1023u) & ~1023u, s_pair = sq + 6 * EX_BOX, s_one = s_pair + 6 * EX_BOX;
   const uint32_t bars = smem_u32(s_bars);
-  // pair slots 0..2 and single slots 3, 4: full and empty; per query tile: copied, rotated, scores, weights, outputs
+  // per pair slot: full, empty; per query tile: copied, rotated, scores, weights, outputs
   const auto full = [&](int i) { return bars + i * 8; };
-  const auto empty = [&](int i) { return bars + (5 + i) * 8; };
-  const auto q_full = [&](int g) { return bars + (10 + g) * 8; };
-  const auto q_ready = [&](int g) { return bars + (12 + g) * 8; };
-  const auto s_full = [&](int g) { return bars + (14 + g) * 8; };
-  const auto p_full = [&](int g) { return bars + (16 + g) * 8; };
-  const auto o_full = [&](int g) { return bars + (18 + g) * 8; };
+  const auto empty = [&](int i) { return bars + (3 + i) * 8; };
+  const auto q_full = [&](int g) { return bars + (6 + g) * 8; };
+  const auto q_ready = [&](int g) { return bars + (8 + g) * 8; };
+  const auto s_full = [&](int g) { return bars + (10 + g) * 8; };
+  const auto p_full = [&](int g) { return bars + (12 + g) * 8; };
+  const auto o_full = [&](int g) { return bars + (14 + g) * 8; };
   if (threadIdx.x == 0) {
-    for (int i = 0; i < 20; ++i) mbar_init(bars + i * 8, (i == 12 || i == 13 || i == 16 || i == 17) ? 4 : 1);
+    for (int i = 0; i < 16; ++i) mbar_init(bars + i * 8, (i == 8 || i == 9 || i == 12 || i == 13) ? 4 : 1);  // softmax: a lane per warp arrives
     s_abort = 0;
     mbar_fence_init();
     tma_prefetch_desc(&tm_q);
@@ -75,10 +76,10 @@ expanded_attn_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
   pdl_launch_dependents();     // only now: a later kernel must not take the tensor memory that a CTA of this one still needs
   pdl_wait();
 
-  const int b = blockIdx.z, h = blockIdx.y;
+  const int b = blockIdx.y, h = blockIdx.x;
   const int row0 = a.cu_q[b], rows = a.cu_q[b + 1] - row0;
   const int key0 = a.cu_k[b], first_pos = a.cu_k[b + 1] - key0 - rows;
-  const int tile0 = (static_cast<int>(gridDim.x) - 1 - static_cast<int>(blockIdx.x)) * 256;  // the longest rows first
+  const int tile0 = (static_cast<int>(gridDim.z) - 1 - static_cast<int>(blockIdx.z)) * 256;  // the longest rows first
   int nr[2], nt[2];  // rows and key tiles of the two query tiles
 #pragma unroll
   for (int g = 0; g < 2; ++g) {
@@ -102,14 +103,11 @@ expanded_attn_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
         for (int half = 0; half < 2; ++half) {  // keys, then values
           const int u = 2 * t + half, slot = u % 3, n = half ? a.nv : a.nd;
           if (!(ok = mbar_wait(empty(slot), ((u / 3) & 1) ^ 1, abort_flag, EX_LIMIT_NS, B2_WAIT_SMEM_EMPTY))) break;
-          mbar_arrive_expect_tx(full(slot), n * EX_BOX);
+          const bool r = half == 0 && a.rot > 0;
+          mbar_arrive_expect_tx(full(slot), (n + r) * EX_BOX);
           for (int i = 0; i < n; ++i)
             tma_load_3d(s_pair + (2 * slot + i) * EX_BOX, half ? &tm_v : &tm_k, full(slot), 64 * i, h, key, kEvictNormal);
-          if (half == 0 && a.rot > 0) {
-            if (!(ok = mbar_wait(empty(3 + (t & 1)), ((t >> 1) & 1) ^ 1, abort_flag, EX_LIMIT_NS, B2_WAIT_SMEM_EMPTY))) break;
-            mbar_arrive_expect_tx(full(3 + (t & 1)), EX_BOX);
-            tma_load_2d(s_one + (t & 1) * EX_BOX, &tm_kr, full(3 + (t & 1)), 0, key, kEvictNormal);
-          }
+          if (r) tma_load_2d(s_one + (t & 1) * EX_BOX, &tm_kr, full(slot), 0, key, kEvictNormal);
         }
       }
     }
@@ -136,10 +134,9 @@ expanded_attn_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
             if (t == nt[g]) umma_commit(o_full(g));
           }
           if (t < nt[g]) {  // S_g = Q_g K^T of tile t, over the weights that have just been used
-            const int u = 2 * t, slot = u % 3, one = 3 + (t & 1);
+            const int u = 2 * t, slot = u % 3;
             if (t == 0 && !(ok = mbar_wait(q_ready(g), 0, abort_flag, EX_LIMIT_NS, B2_WAIT_SMEM_FULL))) break;
             if (!(ok = mbar_wait(full(slot), (u / 3) & 1, abort_flag, EX_LIMIT_NS, B2_WAIT_SMEM_FULL))) break;
-            if (a.rot > 0 && !(ok = mbar_wait(full(one), (t >> 1) & 1, abort_flag, EX_LIMIT_NS, B2_WAIT_SMEM_FULL))) break;
             tc_fence_after();
             for (int i = 0; i < a.nd + (a.rot > 0); ++i) {
               const bool r = i == a.nd;
@@ -148,11 +145,8 @@ expanded_attn_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
 #pragma unroll
               for (int k = 0; k < 4; ++k) umma_bf16(tm + 128 * g, dq + 2 * k, dk + 2 * k, idesc_s, (i > 0 || k > 0) ? 1u : 0u);
             }
-            if (g == last) {
-              umma_commit(empty(slot));
-              if (a.rot > 0) umma_commit(empty(one));
-            }
             umma_commit(s_full(g));  // also says that this tile's outputs so far are complete
+            if (g == last) umma_commit(empty(slot));
           }
         }
       }
@@ -166,15 +160,30 @@ expanded_attn_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
     const float scale = a.scale * LOG2E;
     bool ok = true;
     if (tiles_g > 0) {
+      // the row's angles are on their way while the queries are copied
+      float4 cs[16];
+      const int64_t at_pos = min(pos, a.max_pos - 1);
+#pragma unroll
+      for (int i = 0; i < 16; ++i)
+        if (4 * i < a.rot) cs[i] = __ldg(reinterpret_cast<const float4*>(a.cs + at_pos * (a.rot >> 1)) + i);  // two pairs
       ok = mbar_wait(q_full(g), 0, abort_flag, EX_LIMIT_NS, B2_WAIT_SMEM_FULL);
       if (ok && a.rot > 0) {
         unsigned char* box = smem_raw + (sq - smem_u32(smem_raw)) + (3 * g + 2) * EX_BOX + r * 128;
-        for (int c = 0; c < a.rot >> 3; ++c) {
+#pragma unroll
+        for (int c = 0; c < 8; ++c) {
+          if (c * 8 >= a.rot) break;
           uint16_t* at = reinterpret_cast<uint16_t*>(box + ((c ^ (r & 7)) << 4));
-          float f[8];
+          float f[8], o[8];
           load8<uint16_t>(at, f);
-          rotate8(f, a.cs, a.max_pos, a.rot >> 1, pos, c * 4);
-          store8<uint16_t>(at, f);
+#pragma unroll
+          for (int i = 0; i < 2; ++i) {
+            const float4 w = cs[2 * c + i];
+            o[4 * i] = f[4 * i] * w.x - f[4 * i + 1] * w.y;
+            o[4 * i + 1] = f[4 * i + 1] * w.x + f[4 * i] * w.y;
+            o[4 * i + 2] = f[4 * i + 2] * w.z - f[4 * i + 3] * w.w;
+            o[4 * i + 3] = f[4 * i + 3] * w.z + f[4 * i + 2] * w.w;
+          }
+          store8<uint16_t>(at, o);
         }
       }
       fence_proxy_async();
@@ -244,6 +253,15 @@ expanded_attn_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
       __syncwarp();
       if (lane == 0) mbar_arrive(p_full(g));
     }
+    const bool write = ok && r < nr[g];
+    const int64_t row = row0 + tile0 + 128 * g + r;
+    uint4 gate[16];  // the row's gates are on their way while the last product runs
+    if (a.gate != nullptr && write) {
+      const uint16_t* src = a.gate + row * a.ldg + static_cast<int64_t>(h) * a.v_pad;
+#pragma unroll
+      for (int i = 0; i < 16; ++i)
+        if (8 * i < a.v_pad) gate[i] = *reinterpret_cast<const uint4*>(src + 8 * i);
+    }
     if (ok && tiles_g > 0) ok = mbar_wait(o_full(g), 0, abort_flag, EX_LIMIT_NS, B2_WAIT_TMEM_FULL);
     if (__all_sync(0xffffffffu, ok) && tiles_g > 0) {
       tc_fence_after();
@@ -254,29 +272,27 @@ expanded_attn_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
         l = l * f + fast_exp2(sk - m_new);
       }
       f /= l;
-      const int64_t row = row0 + tile0 + 128 * g + r;
       uint16_t* dst = a.out + row * a.ldo + static_cast<int64_t>(h) * a.v_pad;
-      const uint16_t* gate = a.gate != nullptr ? a.gate + row * a.ldg + static_cast<int64_t>(h) * a.v_pad : nullptr;
-#pragma unroll 1
-      for (int c = 0; c < 2 * a.nv; ++c) {
+#pragma unroll
+      for (int c = 0; c < 4; ++c) {
+        if (32 * c >= a.v_pad) break;
         uint32_t o[32];
         tmem_ld_32x32(to + 32 * c, o);
         tc_wait_ld();
-        if (r >= nr[g]) continue;
+        if (!write) continue;
 #pragma unroll
-        for (int i = 0; i < 32; i += 8) {
-          const int col = 32 * c + i;
-          if (col >= a.v_pad) break;
+        for (int i = 0; i < 4; ++i) {
+          if (32 * c + 8 * i >= a.v_pad) break;
           float x[8];
 #pragma unroll
-          for (int e = 0; e < 8; ++e) x[e] = __uint_as_float(o[i + e]) * f;
-          if (gate != nullptr) {
-            float s[8];
-            load8<uint16_t>(gate + col, s);
+          for (int e = 0; e < 8; ++e) x[e] = __uint_as_float(o[8 * i + e]) * f;
+          if (a.gate != nullptr) {
+            const uint4 s = gate[4 * c + i];
+            const float y[8] = {bf16_lo(s.x), bf16_hi(s.x), bf16_lo(s.y), bf16_hi(s.y), bf16_lo(s.z), bf16_hi(s.z), bf16_lo(s.w), bf16_hi(s.w)};
 #pragma unroll
-            for (int e = 0; e < 8; ++e) x[e] *= sigmoid_fast(s[e]);
+            for (int e = 0; e < 8; ++e) x[e] *= sigmoid_fast(y[e]);
           }
-          store8<uint16_t>(dst + col, x);
+          store8<uint16_t>(dst + 32 * c + 8 * i, x);
         }
       }
     }
@@ -306,9 +322,9 @@ int b2_expanded_attention(b2_ctx* ctx, const void* q, int64_t ldq, int64_t q_row
   if (!q || !out || !kv || !cu_q || !cu_k || !aligned16(q) || !aligned16(out) || !aligned16(kv)) return B2_ERR_ARG;
   if (ldq % 8 != 0 || ldo % 8 != 0 || ld_kv % 8 != 0 || ld_rot % 8 != 0) return B2_ERR_ARG;
   if (ldq < static_cast<int64_t>(heads) * (dim_pad + rot_pad) || ld_kv < static_cast<int64_t>(heads) * (dim_pad + v_pad)) return B2_ERR_ARG;
-  if (rot_pad > 0 && (!rot || !aligned16(rot) || ld_rot < rot_pad || !cos_sin || max_pos <= 0)) return B2_ERR_ARG;
+  if (rot_pad > 0 && (!rot || !aligned16(rot) || ld_rot < rot_pad || !cos_sin || !aligned16(cos_sin) || max_pos <= 0)) return B2_ERR_ARG;
   if (gate != nullptr && (!aligned16(gate) || ldg % 8 != 0)) return B2_ERR_ARG;
-  if (dim_pad > 128 || rot_pad > 64 || v_pad > 128 || B > 65535 || heads > 65535 || q_rows > INT_MAX || k_rows > INT_MAX) return B2_ERR_SHAPE;
+  if (dim_pad > 128 || rot_pad > 64 || v_pad > 128 || B > 65535 || (max_q + 255) / 256 > 65535 || q_rows > INT_MAX || k_rows > INT_MAX) return B2_ERR_SHAPE;
   static const cudaError_t set = cudaFuncSetAttribute(expanded_attn_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, EX_SMEM);
   B2_CUDA(set);
   const uint16_t* qp = static_cast<const uint16_t*>(q);
@@ -330,7 +346,7 @@ int b2_expanded_attention(b2_ctx* ctx, const void* q, int64_t ldq, int64_t q_row
   a.out = static_cast<uint16_t*>(out); a.ldo = ldo; a.cu_q = cu_q; a.cu_k = cu_k; a.nd = (dim_pad + 63) / 64; a.nv = (v_pad + 63) / 64;
   a.rot = rot_pad; a.v_pad = v_pad; a.scale = scale; a.sink = sink; a.cs = reinterpret_cast<const float2*>(cos_sin); a.max_pos = max_pos;
   a.gate = static_cast<const uint16_t*>(gate); a.ldg = ldg; a.status = ctx->status_dev;
-  B2_CUDA(b2_launch(expanded_attn_kernel, dim3((max_q + 255) / 256, heads, B), dim3(EX_THREADS), EX_SMEM, static_cast<cudaStream_t>(stream), m[0], m[1],
+  B2_CUDA(b2_launch(expanded_attn_kernel, dim3(heads, B, (max_q + 255) / 256), dim3(EX_THREADS), EX_SMEM, static_cast<cudaStream_t>(stream), m[0], m[1],
                     m[2], m[3], m[4], a));
   return B2_OK;
 }

@@ -724,15 +724,18 @@ LatentPlan latent_plan(int B, int max_q, int max_kv, int heads, int lat_pad, int
   p.pairs = (p.boxes + 1) / 2;
   const int fixed = 1024 + (((p.boxes + p.rot) * p.rows * 128 + 1023) & ~1023) + p.rows * 512 + LT_SMEM_STATIC;
   const int stage = (2 * p.pairs + p.rot) * LT_BOX;
-  p.stages = std::max(1, std::min(LT_MAX_STAGES, (LT_SMEM_MAX - fixed) / stage));
+  // two CTAs on an SM with one tile each hide each other's waits better than one with several tiles
+  const int per_sm = p.rows == 16 && 2 * (fixed + stage + 1024) <= LT_SMEM_MAX + 1024 ? 2 : 1;
+  p.stages = per_sm == 2 ? 1 : std::max(1, std::min(LT_MAX_STAGES, (LT_SMEM_MAX - fixed) / stage));
   p.smem = fixed - LT_SMEM_STATIC + p.stages * stage;
   p.groups = static_cast<int64_t>(B) * p.row_tiles;
   const int64_t tiles = std::max<int64_t>(1, (static_cast<int64_t>(max_kv) + LT_KEYS - 1) / LT_KEYS);
   p.splits = 1;
-  if (p.groups < 4 * 148) {
+  const int64_t at_once = 148 * per_sm;
+  if (p.groups < 4 * at_once) {
     int64_t best = INT64_MAX;
     for (int s = 1; s <= std::min<int64_t>(LT_MAX_SPLITS, tiles); ++s) {
-      const int64_t cost = ((p.groups * s + 147) / 148) * (8 * ((tiles + s - 1) / s) + 16) + (s > 1 ? 8 : 0) + s / 2;
+      const int64_t cost = ((p.groups * s + at_once - 1) / at_once) * (8 * ((tiles + s - 1) / s) + 16) + (s > 1 ? 8 : 0) + s / 2;
       if (cost < best) {
         best = cost;
         p.splits = s;
