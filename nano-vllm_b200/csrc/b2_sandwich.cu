@@ -76,7 +76,7 @@ struct Vec8<float> {
 // TAPS > 0: that many taps, history and weights in registers; 0: no convolution; -1: a.taps, history in shared memory.
 // NV vectors of 8 channels per thread; RB tokens at a time, so that their loads are in flight together and share barriers.
 template <typename T, int NV, int TAPS, int RB>
-__global__ void __launch_bounds__(512) sandwich_step_kernel(const SandwichArgs a) {
+__global__ void __launch_bounds__(512, RB == 2 && sizeof(T) == 2 ? 2 : 1) sandwich_step_kernel(const SandwichArgs a) {
   extern __shared__ __align__(16) unsigned char hist_smem[];  // TAPS < 0: [taps - 1][dim_pad], a ring by row
   __shared__ __align__(16) float red[2][16][RB];
   constexpr bool CONV = TAPS != 0, REG = TAPS > 0;
@@ -96,9 +96,10 @@ __global__ void __launch_bounds__(512) sandwich_step_kernel(const SandwichArgs a
     nv[i] = c < a.dim_pad ? c : -1;
   }
   T* ring = reinterpret_cast<T*>(hist_smem);
-  Vec8<T> hist[HIST][NV], w[REG ? TAPS : 1][NV];
+  constexpr bool KEEP_W = REG && RB == 1;  // else the weights come from the L1 cache for every token
+  Vec8<T> hist[HIST][NV], w[KEEP_W ? TAPS : 1][NV];
   int head = 0;  // the ring's oldest row
-  if constexpr (REG) {
+  if constexpr (KEEP_W) {
     const T* cw = static_cast<const T*>(a.conv_w);
 #pragma unroll
     for (int j = 0; j < TAPS; ++j)
@@ -241,18 +242,18 @@ __global__ void __launch_bounds__(512) sandwich_step_kernel(const SandwichArgs a
           if (t0 + r >= emit) {
             float acc[8], hf[8], wf[8];
             h.get(hf);
-            if constexpr (REG) w[TAPS - 1][i].get(wf);
+            if constexpr (KEEP_W) w[TAPS - 1][i].get(wf);
             else b2::load8<T>(static_cast<const T*>(a.conv_w) + static_cast<int64_t>(taps - 1) * a.dim_pad + nv[i], wf);
 #pragma unroll
             for (int e = 0; e < 8; ++e) acc[e] = fmaf(wf[e], hf[e], hf[e]);
 #pragma unroll
             for (int j = 0; j < (REG ? TAPS - 1 : taps - 1); ++j) {
               float f[8];
+              if constexpr (KEEP_W) w[j][i].get(wf);
+              else b2::load8<T>(static_cast<const T*>(a.conv_w) + static_cast<int64_t>(j) * a.dim_pad + nv[i], wf);
               if constexpr (REG) {
-                w[j][i].get(wf);
                 hist[j][i].get(f);
               } else {
-                b2::load8<T>(static_cast<const T*>(a.conv_w) + static_cast<int64_t>(j) * a.dim_pad + nv[i], wf);
                 b2::load8<T>(ring + static_cast<int64_t>((head + j) % (taps - 1)) * a.dim_pad + nv[i], f);
               }
 #pragma unroll
@@ -328,7 +329,7 @@ int launch(SandwichArgs a, int B, int max_q, int run, int threads, size_t smem, 
 }
 template <typename T, int NV>
 int dispatch_taps(const SandwichArgs& a, int B, int max_q, int run, int threads, cudaStream_t s) {
-#define B2_STEP(TAPS) return max_q > 1 ? launch<T, NV, TAPS, 4>(a, B, max_q, run, threads, 0, s) : launch<T, NV, TAPS, 1>(a, B, max_q, run, threads, 0, s)
+#define B2_STEP(TAPS) return max_q > 1 ? launch<T, NV, TAPS, 2>(a, B, max_q, run, threads, 0, s) : launch<T, NV, TAPS, 1>(a, B, max_q, run, threads, 0, s)
   if (a.taps == 0) return launch<T, NV, 0, 1>(a, B, max_q, run, threads, 0, s);
   if constexpr (NV == 1) {
     switch (a.taps) {
@@ -352,15 +353,15 @@ int dispatch(const SandwichArgs& a, int B, int max_q, int run, cudaStream_t s) {
 }
 
 // out = a N(z) + b N(z^2) + c N(z^3) + e, N dividing by the root mean square over the row's `dim` elements
-template <typename T>
-__global__ void __launch_bounds__(512) poly_norm_kernel(const T* z, int64_t ldz, const float* coef, float eps, int dim, int dim_pad, T* out, int64_t ldo) {
+// KEEP vectors of 8 per thread stay in registers, longer rows are read again: many for few rows, few where many rows share an SM
+template <typename T, int KEEP>
+__global__ void __launch_bounds__(512, KEEP <= 3 ? 3 : 1) poly_norm_kernel(const T* z, int64_t ldz, const float* coef, float eps, int dim, int dim_pad, T* out, int64_t ldo) {
   __shared__ float red[3][32];
   b2::pdl_launch_dependents();
   b2::pdl_wait();
   const int64_t row = blockIdx.x;
   const T* zr = z + row * ldz;
-  constexpr int KEEP = 4;  // vectors a thread keeps in registers; longer rows are read again
-  float kept[KEEP][8];
+  Vec8<T> kept[KEEP];
   float s1 = 0.f, s2 = 0.f, s3 = 0.f;
   auto add = [&](const float (&f)[8]) {
 #pragma unroll
@@ -374,12 +375,15 @@ __global__ void __launch_bounds__(512) poly_norm_kernel(const T* z, int64_t ldz,
 #pragma unroll
   for (int i = 0; i < KEEP; ++i) {
     const int c = (threadIdx.x + i * blockDim.x) * 8;
-#pragma unroll
-    for (int e = 0; e < 8; ++e) kept[i][e] = 0.f;
-    if (c < dim_pad) b2::load8<T>(zr + c, kept[i]);
+    kept[i].zero();
+    if (c < dim_pad) kept[i].load(zr + c);
   }
 #pragma unroll
-  for (int i = 0; i < KEEP; ++i) add(kept[i]);
+  for (int i = 0; i < KEEP; ++i) {
+    float f[8];
+    kept[i].get(f);
+    add(f);
+  }
   for (int c = (threadIdx.x + KEEP * blockDim.x) * 8; c < dim_pad; c += blockDim.x * 8) {
     float f[8];
     b2::load8<T>(zr + c, f);
@@ -411,7 +415,10 @@ __global__ void __launch_bounds__(512) poly_norm_kernel(const T* z, int64_t ldz,
 #pragma unroll
   for (int i = 0; i < KEEP; ++i) {
     const int c = (threadIdx.x + i * blockDim.x) * 8;
-    if (c < dim_pad) finish(c, kept[i]);
+    if (c >= dim_pad) break;
+    float f[8];
+    kept[i].get(f);
+    finish(c, f);
   }
   for (int c = (threadIdx.x + KEEP * blockDim.x) * 8; c < dim_pad; c += blockDim.x * 8) {
     float f[8];
@@ -471,14 +478,18 @@ int b2_poly_norm(int dtype, const void* z, int64_t ldz, const float* coef, float
   if (M == 0) return B2_OK;
   if (!z || !out || !coef || !aligned16(z) || !aligned16(out)) return B2_ERR_ARG;
   const int nvec = dim_pad / 8;
-  const int threads = std::min(512, std::max(32, (nvec + (M > 296 ? 3 : 0)) / (M > 296 ? 4 : 1) + 31) / 32 * 32);
+  const bool many = M > 296;
+  const int threads = std::min(512, std::max(32, (nvec + (many ? 3 : 0)) / (many ? 4 : 1) + 31) / 32 * 32);
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  if (dtype == B2_DT_BF16)
-    B2_CUDA(b2_launch(poly_norm_kernel<uint16_t>, dim3(M), dim3(threads), 0, s, static_cast<const uint16_t*>(z), ldz, coef, eps, dim, dim_pad,
-                      static_cast<uint16_t*>(out), ldo));
-  else
-    B2_CUDA(b2_launch(poly_norm_kernel<float>, dim3(M), dim3(threads), 0, s, static_cast<const float*>(z), ldz, coef, eps, dim, dim_pad,
-                      static_cast<float*>(out), ldo));
+#define B2_POLY(T, KEEP) \
+  B2_CUDA(b2_launch(poly_norm_kernel<T, KEEP>, dim3(M), dim3(threads), 0, s, static_cast<const T*>(z), ldz, coef, eps, dim, dim_pad, static_cast<T*>(out), ldo))
+  if (dtype == B2_DT_BF16) {
+    if (many) B2_POLY(uint16_t, 3);
+    else B2_POLY(uint16_t, 6);
+  } else {
+    B2_POLY(float, 4);
+  }
+#undef B2_POLY
   return B2_OK;
 }
 
