@@ -9,8 +9,8 @@ Layout mirrors the part of the reference it replaces:
     runtime.py per-process tensor-parallel context (symmetric buffers)
     ops.py     tensor-level wrappers over the C ABI
     layers/    drop-in layer classes (linear, layernorm, embed_head, attention, ...)
-    models/    Qwen3 wiring that uses the fused row-parallel entry
-    engine/    the part of the model runner that hosts the path
+    models/    Qwen3 wiring that uses the fused row-parallel entry; Vekerax, Mupulorn; the registry
+    engine/    the part of the model runner that hosts the path; cache manager, scheduler, LLM
     utils/     per-step context
 """
 from . import _abi  # noqa: F401  (fails loudly when the CUDA library is missing)

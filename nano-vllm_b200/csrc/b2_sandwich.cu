@@ -307,8 +307,12 @@ int launch(SandwichArgs a, int B, int max_q, int run, int threads, size_t smem, 
   if (max_q == 1) run = 1;
   if (run == 0) {
     // tokens per CTA: the fewest rounds of groups over all SMs, where a run also walks the tokens in front of it
-    int resident = 1;
-    B2_CUDA(cudaOccupancyMaxActiveBlocksPerMultiprocessor(&resident, kernel, threads, smem));
+    static int known_threads = -1, known = 1;  // of the last thread count asked for: a model has one
+    if (threads != known_threads) {
+      B2_CUDA(cudaOccupancyMaxActiveBlocksPerMultiprocessor(&known, kernel, threads, smem));
+      known_threads = threads;
+    }
+    const int resident = known;
     const int64_t at_once = 148ll * std::max(1, resident);
     int64_t best = INT64_MAX;
     for (int groups = 1; groups <= 16; ++groups) {
