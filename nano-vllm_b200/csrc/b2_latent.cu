@@ -833,11 +833,9 @@ int b2_heads_gemm(int dtype, const void* x, int64_t ldx, int x_head, const void*
     if (K <= 128) return w_is_kn ? launch_heads<true, 2>(a, heads, s) : launch_heads<false, 2>(a, heads, s);
     return w_is_kn ? launch_heads<true, 8>(a, heads, s) : launch_heads<false, 8>(a, heads, s);
   }
-  {
-    const dim3 grid((N + 63) / 64 + (rot_pad > 0 ? 1 : 0), (M + 63) / 64, heads);
-    if (w_is_kn) B2_CUDA(b2_launch(heads_gemm_f32_kernel<true>, grid, dim3(256), 0, s, a));
-    else B2_CUDA(b2_launch(heads_gemm_f32_kernel<false>, grid, dim3(256), 0, s, a));
-  }
+  const dim3 grid((N + 63) / 64 + (rot_pad > 0 ? 1 : 0), (M + 63) / 64, heads);
+  if (w_is_kn) B2_CUDA(b2_launch(heads_gemm_f32_kernel<true>, grid, dim3(256), 0, s, a));
+  else B2_CUDA(b2_launch(heads_gemm_f32_kernel<false>, grid, dim3(256), 0, s, a));
   return B2_OK;
 }
 
